@@ -227,10 +227,11 @@ class PreNormBlockSpec:
 
 @dataclass(frozen=True)
 class EmbeddingSpec:
-    """x[t] = table[id_t], no scaling (model.py:95)."""
+    """x[t] = scale * table[id_t] in float32; the reference scales by nothing (model.py:95)."""
     vocab_size: int
     hidden_size: int
     weight: str
+    scale: float = 1.0
 
     def tensors(self) -> Mapping[str, TensorSpec]:
         return {self.weight: TensorSpec((self.vocab_size, self.hidden_size))}
@@ -249,6 +250,7 @@ class LMHeadSpec:
     tied: bool
     stored_as: Optional[str] = None
     softcap: Optional[float] = None       # c: logits <- c * tanh(logits / c)
+    scale: float = 1.0                    # logits <- scale * logits, before the soft cap
 
     def tensors(self) -> Mapping[str, TensorSpec]:
         if self.tied:
@@ -599,7 +601,13 @@ class RotaryValueAttentionSpec:
     -i.  Causal, optional window, plain softmax; key and value heads may differ in width.  ``v_proj`` None: the
     values are the keys as projected, before their rotation, and the model has no v matrix.  ``weight_terms``: on the
     tensor-core routes a softmax weight, formed in float32, enters the weighted sum as one bfloat16 number or as two
-    (its rounding and what the rounding left out: 16 bits of the float32 weight, two products)."""
+    (its rounding and what the rounding left out: 16 bits of the float32 weight, two products).
+
+    ``q_bias`` / ``k_bias`` / ``v_bias``: vectors added in the projections.  ``softcap`` c: a scaled score s becomes
+    c * tanh(s / c) before the mask and the softmax.  ``sink_score`` z: exp(z) joins the softmax's denominator, with no key
+    and no value (0: one is added to it).  ``reads_cache``: the mixer has queries only (no k and v tensors) and attends over
+    the keys and values that another layer's mixer stores; its layer call names that layer's cache entry with ``store``
+    False.  ``position`` then turns the queries only."""
     hidden_size: int
     num_heads: int
     num_kv_heads: int
@@ -608,7 +616,7 @@ class RotaryValueAttentionSpec:
     scale: float
     eps: float
     q_proj: str
-    k_proj: str
+    k_proj: Optional[str]
     v_proj: Optional[str]
     o_proj: str
     position: Optional[RotarySpec] = None
@@ -616,14 +624,24 @@ class RotaryValueAttentionSpec:
     value_position: Optional[RotarySpec] = None
     window: Optional[int] = None
     weight_terms: int = 1
+    q_bias: Optional[str] = None
+    k_bias: Optional[str] = None
+    v_bias: Optional[str] = None
+    softcap: Optional[float] = None
+    sink_score: Optional[float] = None
+    reads_cache: bool = False
 
     def tensors(self) -> Mapping[str, TensorSpec]:
         W = self.hidden_size
-        t = {self.q_proj: TensorSpec((self.num_heads * self.head_dim, W)),
-             self.k_proj: TensorSpec((self.num_kv_heads * self.head_dim, W)),
-             self.o_proj: TensorSpec((W, self.num_heads * self.value_head_dim))}
-        if self.v_proj is not None:
-            t[self.v_proj] = TensorSpec((self.num_kv_heads * self.value_head_dim, W))
+        widths = ((self.q_proj, self.q_bias, self.num_heads * self.head_dim),
+                  (self.k_proj, self.k_bias, self.num_kv_heads * self.head_dim),
+                  (self.v_proj, self.v_bias, self.num_kv_heads * self.value_head_dim))
+        t = {self.o_proj: TensorSpec((W, self.num_heads * self.value_head_dim))}
+        for proj, bias, width in widths:
+            if proj is not None:
+                t[proj] = TensorSpec((width, W))
+            if bias is not None:
+                t[bias] = TensorSpec((width,), init=(0.0, 0.3))
         return t
 
     def cache_need(self):
@@ -650,8 +668,10 @@ class ParallelMixerSpec:
 
 @dataclass(frozen=True)
 class RoutedExpertsSpec:
-    """A mixture of gated feed-forwards without biases.  Router logits z = R h in 32-bit; an expert is
-    down(act(gate h) * (up h)).  ``experts`` names each expert's (gate, up, down) tensors.
+    """A mixture of feed-forwards without biases.  Router logits z = R h in 32-bit; an expert is
+    down(act(gate h) * (up h)).  ``experts`` names each expert's (gate, up, down) tensors; where they name two (up, down), an
+    expert has no gate: down(act(up h)).  ``activation``: "silu" with a gate, "relu2" (the square of relu), "silu" or
+    "gelu_tanh" without.
 
     ``scoring`` "chosen" (the default): each token runs the ``top`` experts with the largest logits, weighted by the
     softmax over those logits only.  ``scoring`` "all": the scores are the softmax over all experts, the ``top`` largest
@@ -659,29 +679,43 @@ class RoutedExpertsSpec:
     the scores are sigmoid(z) per expert, chosen and weighted like "all".  ``weight_on`` "output" (the default): the
     weight multiplies the expert's result; "input": it multiplies what the expert reads, and the results are summed as
     they are (the two differ because an expert is not linear).  ``groups`` =
-    (count, keep): the experts form ``count`` equal groups of neighbours, a group's score is its largest score, and only
-    experts of the ``keep`` best groups can be chosen (None: no such limit).  ``shared``: a gated feed-forward that
+    (count, keep): the experts form ``count`` equal groups of neighbours, a group's score is the sum of its ``group_best``
+    largest scores (1, the default: its largest; a group with fewer experts sums those it has), and only experts of the
+    ``keep`` best groups can be chosen (None: no such limit).  ``shared``: a feed-forward that
     every token runs, added to the sum; with ``shared_gate`` (a tensor [1, hidden]) it is first multiplied by
-    sigmoid(shared_gate . h), one number per token."""
+    sigmoid(shared_gate . h), one number per token.
+
+    With ``scoring`` "sigmoid": ``correction`` names a vector [experts] that is added to the scores for the choice (of the
+    groups and of the experts) and not for the weights; ``normalise``: the chosen scores are divided by their sum + 1e-20
+    (then times ``weight_scale``)."""
     hidden_size: int
     intermediate_size: int
     top: int
     activation: str
     router: str
-    experts: Tuple[Tuple[str, str, str], ...]
+    experts: Tuple[Tuple[str, ...], ...]
     scoring: str = "chosen"
     weight_scale: float = 1.0
     groups: Optional[Tuple[int, int]] = None
-    shared: Optional[GatedMLPSpec] = None
+    shared: Optional[object] = None            # a GatedMLPSpec or a DenseMLPSpec
     shared_gate: Optional[str] = None
     weight_on: str = "output"
+    correction: Optional[str] = None
+    normalise: bool = False
+    group_best: int = 1
+
+    @property
+    def gated(self) -> bool:
+        return len(self.experts[0]) == 3
 
     def tensors(self) -> Mapping[str, TensorSpec]:
         t = {self.router: TensorSpec((len(self.experts), self.hidden_size), init=(0.0, 0.3))}
-        for gate, up, down in self.experts:
-            t[gate] = TensorSpec((self.intermediate_size, self.hidden_size))
-            t[up] = TensorSpec((self.intermediate_size, self.hidden_size))
-            t[down] = TensorSpec((self.hidden_size, self.intermediate_size))
+        for names in self.experts:
+            for name in names[:-1]:
+                t[name] = TensorSpec((self.intermediate_size, self.hidden_size))
+            t[names[-1]] = TensorSpec((self.hidden_size, self.intermediate_size))
+        if self.correction is not None:
+            t[self.correction] = TensorSpec((len(self.experts),), init=(0.0, 0.1))
         if self.shared is not None:
             t.update(self.shared.tensors())
         if self.shared_gate is not None:
@@ -865,6 +899,26 @@ class DepthAverageBlockSpec:
         """Entry 0: the mixer's; entries 1 and 2: the states of the two convolutions (None where there is none)."""
         return (self.mixer.cache_need(), self.mixer_conv.cache_need() if self.mixer_conv is not None else None,
                 self.ffn_conv.cache_need() if self.ffn_conv is not None and self.ffn is not None else None)
+
+
+# --------------------------------------------------------------------------- parts of parallel-sublayer decoders
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """h = norm(x); x += mixer(h) + ffn(h): one norm, whose output both sublayers read, and one addition (``ffn`` None: the
+    mixer alone)."""
+    norm: object
+    mixer: object
+    ffn: Optional[object] = None
+
+    def tensors(self) -> Mapping[str, TensorSpec]:
+        t = {}
+        for part in (self.norm, self.mixer, self.ffn):
+            if part is not None:
+                t.update(part.tensors())
+        return t
+
+    def cache_need(self):
+        return self.mixer.cache_need()
 
 
 # --------------------------------------------------------------------------- the order

@@ -1,5 +1,6 @@
 // Attention over the paged cache on tensor cores (bfloat16 operands, float32 accumulation and
-// softmax), compiled for one head size: -DHEAD_DIM=<multiple of 16, at most 256>.
+// softmax), compiled for one head size: -DHEAD_DIM=<multiple of 16, at most 256>; -DVALUE_DIM=<likewise> where values are
+// narrower or wider than keys.
 //
 // Two kernels share the tile code and split a step's requests between them by the number of
 // score rows a request brings, rows = query tokens x (query heads per key/value head):
@@ -16,10 +17,16 @@
 // Both read every key, this step's own included, from the pages named by the request's block
 // table: the query at position p sees positions max(0, p-window+1) .. p.  Keys outside what a
 // CTA needs are not fetched (block-table entries of pages that a window has passed are stale).
+// Keys and values are two page streams: a stream's page p begins `page_stride` elements after page p - 1 and holds
+// [kv_heads][page_size][width] (keys and values in one tensor [pages][2][...] are two such streams with a common stride).
+// More than 16 query heads per key/value head are worked on as several groups that read the same head (`share`).
+//
+// -DSOFTCAP=1: a scaled score s becomes c tanh(s / c) before mask and softmax.  A sink z (an argument; -inf: none) joins the
+// denominator as exp(z) where a row's sums are finished.
 //
 // How a tile of keys and values reaches shared memory.  With head sizes that are multiples of 64 and
-// pages of 16, 32 or 64 tokens, TMA brings it: the page pool is described by one tensor map as a
-// matrix [pages * 2 * kv_heads * page_size, head_dim], a page's keys (or values) of one head are one
+// pages of 16, 32 or 64 tokens, TMA brings it: each stream is described by a tensor map as a
+// matrix of rows of its width, a page's keys (or values) of one head are one
 // box per 64 columns, written in the 128-byte swizzle, which ldmatrix then reads without bank
 // conflicts.  Sixteen lanes of warp 0 issue a tile's boxes; a stage's mbarrier counts the bytes.  A
 // page that lies outside the keys a CTA needs is fetched from a row beyond the tensor (zeros).  Waits
@@ -37,17 +44,27 @@
 #if HEAD_DIM % 16 != 0 || HEAD_DIM < 16 || HEAD_DIM > 256
 #error "HEAD_DIM must be a multiple of 16 between 16 and 256"
 #endif
+#ifndef VALUE_DIM
+#define VALUE_DIM HEAD_DIM
+#endif
+#if VALUE_DIM % 16 != 0 || VALUE_DIM < 16 || VALUE_DIM > 256
+#error "VALUE_DIM must be a multiple of 16 between 16 and 256"
+#endif
+#ifndef SOFTCAP
+#define SOFTCAP 0
+#endif
 
 typedef __nv_bfloat16 bf16;
-constexpr int D = HEAD_DIM;
-constexpr int DP = D + 8;          // shared-memory row length: the 16-byte pad keeps ldmatrix conflict-free
+constexpr int D = HEAD_DIM, VD = VALUE_DIM;
+constexpr int DP = D + 8, VDP = VD + 8;      // shared-memory row lengths: the 16-byte pad keeps ldmatrix conflict-free
 constexpr int BN = 64;             // keys per tile
 constexpr int THREADS = 128;
-constexpr int KCH = D / 8;         // 16-byte pieces of a row
-constexpr int KB = D / 16;         // k-blocks of a q.k product, n-block pairs of a p.v product
+constexpr int KCH = D / 8;         // 16-byte pieces of a query row
+constexpr int KB = D / 16;         // k-blocks of a q.k product
+constexpr int VB = VD / 16;        // n-block pairs of a p.v product
 constexpr int SQ_STAGES = 3;       // tile buffers of the small-q kernel: two tiles are in flight while one is used
-constexpr bool TMA_D = (D % 64 == 0);            // head sizes the TMA path takes
-constexpr int HALVES = TMA_D ? D / 64 : 1;       // 64-column (128-byte) boxes per row
+constexpr bool TMA_D = (D % 64 == 0 && VD % 64 == 0);       // head sizes the TMA path takes
+constexpr int KHALVES = TMA_D ? D / 64 : 1, VHALVES = TMA_D ? VD / 64 : 1;      // 64-column (128-byte) boxes per row
 constexpr uint32_t ATT_SPIN_LIMIT = 1u << 22;
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -77,6 +94,22 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+// What stands between a product q . k and the exponent of its weight: SOFTCAP 0: `a` = scale * log2(e), s * a.  SOFTCAP 1:
+// the capped score c tanh(scale s / c) in the base-2 domain, `a` = c log2(e), `b` = 2 scale log2(e) / c:
+// a (1 - 2 / (1 + 2^(b s))), whose absolute error is a few 2^-23 of a (exact at both ends: 2^(b s) may be 0 or infinite).
+struct AttScale { float a, b; };
+__device__ __forceinline__ float att_score(float s, const AttScale& sc) {
+#if SOFTCAP
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.f + fast_exp2(s * sc.b)));
+  return fmaf(-2.f * sc.a, r, sc.a);
+#else
+  return s * sc.a;
+#endif
+}
+// Where the rows of a key/value stream lie: element (page, head, offset, col) at page * page_stride + (head * page_size +
+// offset) * width + col.
+struct AttStream { const bf16* base; long long page_stride; };
 // WEIGHT_TERMS 2 (a library variant of its own): a softmax weight enters the P V product as the sum of two bfloat16 numbers,
 // its rounding and what the rounding left out (16 bits of the float32 weight), and the product takes two instructions.
 #ifndef WEIGHT_TERMS
@@ -121,58 +154,65 @@ __device__ __forceinline__ void att_tma_load_2d(void* smem, const CUtensorMap* m
                ::"r"(smem_u32(smem)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y) : "memory");
 }
 
-// Address of 8 elements (key, col .. col+7) of a K or V tile.  Padded layout: [BN][DP].  Swizzled layout (what
-// TMA wrote): [HALVES][BN][64], the 16-byte piece c of a row stored at c ^ (row & 7); the tile is 1024-byte aligned.
-template <bool SWZ>
+// Address of 8 elements (key, col .. col+7) of a K or V tile.  Padded layout: [BN][PITCH].  Swizzled layout (what
+// TMA wrote): [halves][BN][64], the 16-byte piece c of a row stored at c ^ (row & 7); the tile is 1024-byte aligned.
+template <bool SWZ, int PITCH>
 __device__ __forceinline__ const bf16* kv_at(const bf16* tile, int key, int col) {
   if (SWZ) return tile + (col >> 6) * (BN * 64) + key * 64 + ((((col & 63) >> 3) ^ (key & 7)) << 3);
-  return tile + key * DP + col;
+  return tile + key * PITCH + col;
 }
 
+// The two streams as matrices of rows: how many rows a page spans and how many rows there are.
+struct AttRows { int k_page, v_page, k_total, v_total; };
+
 // One tile by TMA, issued by warp 0 (all 32 lanes call): K to `stage`, V to `stage + BN*D`.  Pages that do not
-// overlap the keys [k_lo, k_hi] are read from beyond the tensor's last row, which gives zeros.
-__device__ __forceinline__ void tma_issue_tile(const CUtensorMap* map, bf16* stage, uint64_t* bar, const int* __restrict__ bt,
-                                               int tile_key0, int k_lo, int k_hi, int kvh, int nkv, int page_size,
-                                               int ps_shift, int total_rows, int lane) {
+// overlap the keys [k_lo, k_hi] are read from beyond the tensor's last row, which gives zeros.  head: of the keys/values.
+__device__ __forceinline__ void tma_issue_tile(const CUtensorMap* k_map, const CUtensorMap* v_map, bf16* stage, uint64_t* bar,
+                                               const int* __restrict__ bt, int tile_key0, int k_lo, int k_hi, int head,
+                                               int page_size, int ps_shift, const AttRows& rows, int lane) {
   const int ppt = BN >> ps_shift;                    // pages per tile
-  const int n_ops = ppt * HALVES * 2;                // at most 4 * 4 * 2 = 32
-  if (lane == 0) att_mbar_expect_tx(bar, 2u * BN * D * sizeof(bf16));
+  const int n_k = ppt * KHALVES, n_ops = n_k + ppt * VHALVES;      // at most 4 * 4 + 4 * 4 = 32
+  if (lane == 0) att_mbar_expect_tx(bar, (uint32_t)(BN * (D + VD)) * (uint32_t)sizeof(bf16));
   __syncwarp();
   if (lane < n_ops) {
-    const int kv = lane / (ppt * HALVES), rem = lane % (ppt * HALVES), pg = rem / HALVES, half = rem % HALVES;
+    const bool is_v = lane >= n_k;
+    const int rem = is_v ? lane - n_k : lane, halves = is_v ? VHALVES : KHALVES, pg = rem / halves, half = rem % halves;
     const int key0 = tile_key0 + pg * page_size;
-    int y = total_rows;
-    if (key0 <= k_hi && key0 + page_size - 1 >= k_lo) y = ((bt[key0 >> ps_shift] * 2 + kv) * nkv + kvh) * page_size;
-    att_tma_load_2d(stage + kv * (BN * D) + half * (BN * 64) + pg * page_size * 64, map, bar, half * 64, y);
+    int y = is_v ? rows.v_total : rows.k_total;
+    if (key0 <= k_hi && key0 + page_size - 1 >= k_lo) y = bt[key0 >> ps_shift] * (is_v ? rows.v_page : rows.k_page) + head * page_size;
+    att_tma_load_2d(stage + (is_v ? BN * D : 0) + half * (BN * 64) + pg * page_size * 64, is_v ? v_map : k_map, bar, half * 64, y);
   }
 }
 
-// Keys key0 .. key0+BN-1 of one key/value head into Ks and Vs ([BN][DP]); keys outside [lo, hi] are zeros.
+// Keys key0 .. key0+BN-1 of one key/value head into Ks ([BN][DP]) and Vs ([BN][VDP]); keys outside [lo, hi] are zeros.
 // Consecutive threads copy consecutive 16-byte pieces of a row, so a warp's copy instruction covers whole
 // 128-byte lines (a piece per thread at scattered rows would cost a memory request each).
-__device__ __forceinline__ void load_kv_tile(bf16* Ks, bf16* Vs, const bf16* __restrict__ pages,
-                                             const int* __restrict__ bt, int key0, int lo, int hi, int kvh, int nkv,
-                                             int page_size, int tid) {
-  const size_t head_stride = (size_t)page_size * D, page_stride = 2 * (size_t)nkv * head_stride;
+template <int W, int PITCH>
+__device__ __forceinline__ void load_stream_tile(bf16* dst, const AttStream& st, const int* __restrict__ bt, int key0, int lo, int hi,
+                                                 int head, int page_size, int tid) {
+  constexpr int CH = W / 8, PASSES = (BN * CH + THREADS - 1) / THREADS;
   const int ps_shift = (page_size & (page_size - 1)) == 0 ? __ffs(page_size) - 1 : -1;   // power of two: shift, else divide
-  constexpr int PASSES = (BN * KCH + THREADS - 1) / THREADS;
 #pragma unroll
   for (int ps = 0; ps < PASSES; ++ps) {
     const int c = tid + ps * THREADS;
-    if ((BN * KCH) % THREADS != 0 && c >= BN * KCH) break;
-    const int row = c / KCH, ch = c % KCH;
+    if ((BN * CH) % THREADS != 0 && c >= BN * CH) break;
+    const int row = c / CH, ch = c % CH;
     const int key = key0 + row;
     const bool valid = key >= lo && key <= hi;
-    const bf16* src = pages;
+    const bf16* src = st.base;
     if (valid) {
       int pi, off;
       if (ps_shift >= 0) { pi = key >> ps_shift; off = key & (page_size - 1); }
       else { pi = key / page_size; off = key - pi * page_size; }
-      src = pages + (size_t)bt[pi] * page_stride + (size_t)kvh * head_stride + (size_t)off * D + ch * 8;
+      src = st.base + (size_t)bt[pi] * st.page_stride + ((size_t)head * page_size + off) * W + ch * 8;
     }
-    cp_async16(Ks + row * DP + ch * 8, src, valid);
-    cp_async16(Vs + row * DP + ch * 8, valid ? src + (size_t)nkv * head_stride : pages, valid);
+    cp_async16(dst + row * PITCH + ch * 8, src, valid);
   }
+}
+__device__ __forceinline__ void load_kv_tile(bf16* Ks, bf16* Vs, const AttStream& ks, const AttStream& vs, const int* __restrict__ bt,
+                                             int key0, int lo, int hi, int head, int page_size, int tid) {
+  load_stream_tile<D, DP>(Ks, ks, bt, key0, lo, hi, head, page_size, tid);
+  load_stream_tile<VD, VDP>(Vs, vs, bt, key0, lo, hi, head, page_size, tid);
 }
 
 // One warp: scores of its 16 query rows (fragments qf) against keys [kbeg, kbeg + 8*NB) of the tile in
@@ -180,8 +220,8 @@ __device__ __forceinline__ void load_kv_tile(bf16* Ks, bf16* Vs, const bf16* __r
 // pA/pB: position of the row's query (-1000000000: the row does not exist); wlo: window (0: none).
 template <int NB, bool MASK, bool SWZ>
 __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[KB][4], const bf16* Ks, const bf16* Vs, int kbeg,
-                                          int key0, int klo, int khi, int pA, int pB, int window, float scale_log2,
-                                          float (&m)[2], float (&l)[2], float (&o)[D / 8][4], int lane) {
+                                          int key0, int klo, int khi, int pA, int pB, int window, const AttScale& sc,
+                                          float (&m)[2], float (&l)[2], float (&o)[VD / 8][4], int lane) {
   float s[NB][4];
 #pragma unroll
   for (int j = 0; j < NB; ++j) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
@@ -192,7 +232,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[KB][4], const bf1
       uint32_t b[4];
       const int key = kbeg + j * 8 + (lane & 7) + ((lane >> 4) << 3);
       const int col = kb * 16 + (((lane >> 3) & 1) << 3);
-      ldmatrix_x4(b, kv_at<SWZ>(Ks, key, col));
+      ldmatrix_x4(b, kv_at<SWZ, DP>(Ks, key, col));
       mma_bf16(s[j], qf[kb], b[0], b[1]);
       mma_bf16(s[j + 1], qf[kb], b[2], b[3]);
     }
@@ -211,8 +251,8 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[KB][4], const bf1
         va = in && key <= pA && key >= loA;
         vb = in && key <= pB && key >= loB;
       }
-      s[j][e] = va ? s[j][e] * scale_log2 : -INFINITY;
-      s[j][2 + e] = vb ? s[j][2 + e] * scale_log2 : -INFINITY;
+      s[j][e] = va ? att_score(s[j][e], sc) : -INFINITY;
+      s[j][2 + e] = vb ? att_score(s[j][2 + e], sc) : -INFINITY;
       mxA = fmaxf(mxA, s[j][e]);
       mxB = fmaxf(mxB, s[j][2 + e]);
     }
@@ -241,7 +281,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[KB][4], const bf1
   l[1] = l[1] * cB + sumB;
   if (__any_sync(0xffffffffu, moved)) {                     // else both factors are exactly 1 for every lane
 #pragma unroll
-    for (int n = 0; n < D / 8; ++n) { o[n][0] *= cA; o[n][1] *= cA; o[n][2] *= cB; o[n][3] *= cB; }
+    for (int n = 0; n < VD / 8; ++n) { o[n][0] *= cA; o[n][1] *= cA; o[n][2] *= cB; o[n][3] *= cB; }
   }
   // o += p v
 #pragma unroll
@@ -259,11 +299,11 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[KB][4], const bf1
     a2[3] = pack_bf16_rest(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #endif
 #pragma unroll
-    for (int n2 = 0; n2 < KB; ++n2) {
+    for (int n2 = 0; n2 < VB; ++n2) {
       uint32_t b[4];
       const int key = kbeg + kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
       const int col = n2 * 16 + ((lane >> 4) << 3);
-      ldmatrix_x4_trans(b, kv_at<SWZ>(Vs, key, col));
+      ldmatrix_x4_trans(b, kv_at<SWZ, VDP>(Vs, key, col));
       mma_bf16(o[2 * n2], a, b[0], b[1]);
       mma_bf16(o[2 * n2 + 1], a, b[2], b[3]);
 #if WEIGHT_TERMS == 2
@@ -286,18 +326,19 @@ __device__ __forceinline__ void load_q_frags(uint32_t (&qf)[KB][4], const bf16* 
 constexpr int NO_ROW = -1000000000;
 
 // The end of a small-q CTA: its four consumer warps' (m, l, o) are merged through shared memory (`scratch`, at least
-// 4*16*D + 128 floats, free by now); then the output row is written, or with several splits the partial sums go to
+// 4*16*VD + 128 floats, free by now); then the output row is written, or with several splits the partial sums go to
 // global memory and the CTA that arrives last for its (request, key/value head) merges the splits in split order.
+// The sink (base-2 score; -inf: none) joins the denominator where it is last summed.
 // Every thread of the CTA calls this (threads of warps above 3 only keep the barriers company).
-__device__ __forceinline__ void small_q_finish(float* scratch, float (&m)[2], float (&l)[2], float (&o)[D / 8][4], int rows,
+__device__ __forceinline__ void small_q_finish(float* scratch, float (&m)[2], float (&l)[2], float (&o)[VD / 8][4], int rows,
                                                int G, int q0, int kvh, int r, int split, int num_splits, int nq, int nkv,
                                                bf16* __restrict__ out, float* __restrict__ part_o,
-                                               float* __restrict__ part_ml, int* __restrict__ counters, int* is_last_p) {
+                                               float* __restrict__ part_ml, int* __restrict__ counters, int* is_last_p, float sink) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int nthreads = blockDim.x;
   const int rowA = lane >> 2, rowB = rowA + 8;
-  float* sm_o = scratch;                                     // [4][16][D]
-  float* sm_m = sm_o + 4 * 16 * D;                           // [4][16]
+  float* sm_o = scratch;                                     // [4][16][VD]
+  float* sm_m = sm_o + 4 * 16 * VD;                          // [4][16]
   float* sm_l = sm_m + 64;                                   // [4][16]
   if (warp < 4) {
 #pragma unroll
@@ -310,17 +351,17 @@ __device__ __forceinline__ void small_q_finish(float* scratch, float (&m)[2], fl
       sm_l[warp * 16 + rowA] = l[0]; sm_l[warp * 16 + rowB] = l[1];
     }
 #pragma unroll
-    for (int n = 0; n < D / 8; ++n) {
+    for (int n = 0; n < VD / 8; ++n) {
       const int col = n * 8 + ((lane & 3) << 1);
-      float* pa = sm_o + ((size_t)warp * 16 + rowA) * D + col;
-      float* pb = sm_o + ((size_t)warp * 16 + rowB) * D + col;
+      float* pa = sm_o + ((size_t)warp * 16 + rowA) * VD + col;
+      float* pb = sm_o + ((size_t)warp * 16 + rowB) * VD + col;
       pa[0] = o[n][0]; pa[1] = o[n][1]; pb[0] = o[n][2]; pb[1] = o[n][3];
     }
   }
   __syncthreads();
-  for (int idx = tid; idx < rows * D; idx += nthreads) {
-    const int row = idx / D, dim = idx % D;
-    float M = -INFINITY;
+  for (int idx = tid; idx < rows * VD; idx += nthreads) {
+    const int row = idx / VD, dim = idx % VD;
+    float M = num_splits == 1 ? sink : -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) M = fmaxf(M, sm_m[w * 16 + row]);
     const float U = M == -INFINITY ? 0.f : M;
@@ -329,14 +370,15 @@ __device__ __forceinline__ void small_q_finish(float* scratch, float (&m)[2], fl
     for (int w = 0; w < 4; ++w) {
       const float f = exp2f(sm_m[w * 16 + row] - U);
       den += sm_l[w * 16 + row] * f;
-      acc += sm_o[((size_t)w * 16 + row) * D + dim] * f;
+      acc += sm_o[((size_t)w * 16 + row) * VD + dim] * f;
     }
     const int tok = q0 + row / G, head = kvh * G + row % G;
     if (num_splits == 1) {
-      out[((size_t)tok * nq + head) * D + dim] = __float2bfloat16_rn(den > 0.f ? acc / den : 0.f);
+      den += exp2f(sink - U);
+      out[((size_t)tok * nq + head) * VD + dim] = __float2bfloat16_rn(den > 0.f ? acc / den : 0.f);
     } else {
       const size_t base = ((size_t)tok * nq + head) * num_splits + split;
-      part_o[base * D + dim] = acc;
+      part_o[base * VD + dim] = acc;
       if (dim == 0) { part_ml[base * 2] = M; part_ml[base * 2 + 1] = den; }
     }
   }
@@ -350,20 +392,20 @@ __device__ __forceinline__ void small_q_finish(float* scratch, float (&m)[2], fl
   __syncthreads();
   if (!*is_last_p) return;
   __threadfence();
-  for (int idx = tid; idx < rows * D; idx += nthreads) {
-    const int row = idx / D, dim = idx % D;
+  for (int idx = tid; idx < rows * VD; idx += nthreads) {
+    const int row = idx / VD, dim = idx % VD;
     const int tok = q0 + row / G, head = kvh * G + row % G;
     const size_t base = ((size_t)tok * nq + head) * num_splits;
-    float M = -INFINITY;
+    float M = sink;
     for (int sp = 0; sp < num_splits; ++sp) M = fmaxf(M, part_ml[(base + sp) * 2]);
     const float U = M == -INFINITY ? 0.f : M;
-    float den = 0.f, acc = 0.f;
+    float den = exp2f(sink - U), acc = 0.f;
     for (int sp = 0; sp < num_splits; ++sp) {
       const float f = exp2f(part_ml[(base + sp) * 2] - U);
       den += part_ml[(base + sp) * 2 + 1] * f;
-      acc += part_o[(base + sp) * D + dim] * f;
+      acc += part_o[(base + sp) * VD + dim] * f;
     }
-    out[((size_t)tok * nq + head) * D + dim] = __float2bfloat16_rn(den > 0.f ? acc / den : 0.f);
+    out[((size_t)tok * nq + head) * VD + dim] = __float2bfloat16_rn(den > 0.f ? acc / den : 0.f);
   }
   if (tid == 0) counters[r * nkv + kvh] = 0;       // ready for the next launch
 }
@@ -373,18 +415,18 @@ __device__ __forceinline__ void small_q_finish(float* scratch, float (&m)[2], fl
 // --------------------------------------------------------------------------------------------
 template <bool TMA>
 __global__ void __launch_bounds__(THREADS)
-attn_small_q_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, int* __restrict__ err,
-                    const bf16* __restrict__ qkv, int row_stride, const bf16* __restrict__ pages,
+attn_small_q_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, AttRows mrows,
+                    int* __restrict__ err, const bf16* __restrict__ qkv, int row_stride, AttStream kst, AttStream vst,
                     const int* __restrict__ block_tables, int bt_stride, const int* __restrict__ cu_q,
                     const int* __restrict__ seq_lens, bf16* __restrict__ out, float* __restrict__ part_o,
-                    float* __restrict__ part_ml, int* __restrict__ counters, int nq, int nkv, int page_size,
-                    float scale_log2, int window, int num_splits) {
+                    float* __restrict__ part_ml, int* __restrict__ counters, int nq, int nkv, int share, int page_size,
+                    AttScale sc, float sink, int window, int num_splits) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ int is_last;
   __shared__ uint64_t full_bar[SQ_STAGES];
   __shared__ int abort_word;
   volatile int* abort_flag = &abort_word;
-  constexpr int STAGE = TMA ? 2 * BN * D : 2 * BN * DP;       // elements of one stage: K tile then V tile
+  constexpr int KT = TMA ? BN * D : BN * DP, STAGE = KT + (TMA ? BN * VD : BN * VDP);   // elements of a K tile, of one stage
   // the stages first (TMA wants them 1024-byte aligned), then the 16 query rows
   const uint32_t raw = smem_u32(smem_raw);
   bf16* KV = reinterpret_cast<bf16*>(smem_raw + (TMA ? ((raw + 1023u) & ~1023u) - raw : 0u));
@@ -433,19 +475,19 @@ attn_small_q_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, 
       bf16* Kn = KV + st * STAGE;
       if (TMA) {
         if (warp == 0)
-          tma_issue_tile(&kv_map, Kn, &full_bar[st], bt, T0 + st * BN, k_begin, k_end - 1, kvh, nkv, page_size, ps_shift,
-                         total_rows, lane);
+          tma_issue_tile(&k_map, &v_map, Kn, &full_bar[st], bt, T0 + st * BN, k_begin, k_end - 1, kvh / share, page_size, ps_shift,
+                         mrows, lane);
       } else {
-        load_kv_tile(Kn, Kn + BN * DP, pages, bt, T0 + st * BN, k_begin, k_end - 1, kvh, nkv, page_size, tid);
+        load_kv_tile(Kn, Kn + KT, kst, vst, bt, T0 + st * BN, k_begin, k_end - 1, kvh / share, page_size, tid);
       }
     }
     if (!TMA) cp_async_commit();
   }
 
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  float o[D / 8][4];
+  float o[VD / 8][4];
 #pragma unroll
-  for (int n = 0; n < D / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
+  for (int n = 0; n < VD / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
   const int rowA = lane >> 2, rowB = rowA + 8;
   const int pA = rowA < rows ? p_first + rowA / G : NO_ROW, pB = rowB < rows ? p_first + rowB / G : NO_ROW;
   uint32_t qf[KB][4];
@@ -453,7 +495,7 @@ attn_small_q_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, 
   for (int t = 0; t < n_tiles; ++t) {
     const int stage = t % SQ_STAGES;
     bf16* Ks = KV + stage * STAGE;
-    bf16* Vs = Ks + (TMA ? BN * D : BN * DP);
+    bf16* Vs = Ks + KT;
     if (TMA) {
       if (t == 0) cp_async_wait<0>();        // the query rows
       ok = att_mbar_wait(&full_bar[stage], (t / SQ_STAGES) & 1, abort_flag, err, 1);
@@ -467,10 +509,10 @@ attn_small_q_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, 
       bf16* Kn = KV + (nt % SQ_STAGES) * STAGE;
       if (TMA) {
         if (warp == 0)
-          tma_issue_tile(&kv_map, Kn, &full_bar[nt % SQ_STAGES], bt, T0 + nt * BN, k_begin, k_end - 1, kvh, nkv, page_size,
-                         ps_shift, total_rows, lane);
+          tma_issue_tile(&k_map, &v_map, Kn, &full_bar[nt % SQ_STAGES], bt, T0 + nt * BN, k_begin, k_end - 1, kvh / share, page_size,
+                         ps_shift, mrows, lane);
       } else {
-        load_kv_tile(Kn, Kn + BN * DP, pages, bt, T0 + nt * BN, k_begin, k_end - 1, kvh, nkv, page_size, tid);
+        load_kv_tile(Kn, Kn + KT, kst, vst, bt, T0 + nt * BN, k_begin, k_end - 1, kvh / share, page_size, tid);
       }
     }
     if (!TMA) cp_async_commit();
@@ -480,9 +522,9 @@ attn_small_q_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, 
     const int tile0 = T0 + t * BN;
     const bool interior = tile0 >= k_begin && tile0 + BN - 1 <= min(p_first, k_end - 1) && (window == 0 || tile0 >= L - window);
     if (interior)
-      warp_tile<2, false, TMA>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, scale_log2, m, l, o, lane);
+      warp_tile<2, false, TMA>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, sc, m, l, o, lane);
     else
-      warp_tile<2, true, TMA>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, scale_log2, m, l, o, lane);
+      warp_tile<2, true, TMA>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, sc, m, l, o, lane);
   }
   cp_async_wait<0>();
   if (TMA && !ok) {                          // a wait gave up: let copies in flight land, then leave
@@ -491,7 +533,7 @@ attn_small_q_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, 
   }
   __syncthreads();
   small_q_finish(reinterpret_cast<float*>(KV), m, l, o, rows, G, q0, kvh, r, split, num_splits, nq, nkv, out, part_o, part_ml,
-                 counters, &is_last);
+                 counters, &is_last, sink);
 }
 
 // --------------------------------------------------------------------------------------------
@@ -507,17 +549,18 @@ __device__ __forceinline__ void att_mbar_arrive(uint64_t* bar) {
 }
 
 __global__ void __launch_bounds__(WS_THREADS)
-attn_small_q_ws_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, int* __restrict__ err,
+attn_small_q_ws_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, AttRows mrows,
+                       int* __restrict__ err,
                        const bf16* __restrict__ qkv, int row_stride, const int* __restrict__ block_tables, int bt_stride,
                        const int* __restrict__ cu_q, const int* __restrict__ seq_lens, bf16* __restrict__ out,
                        float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int nq,
-                       int nkv, int page_size, float scale_log2, int window, int num_splits) {
+                       int nkv, int share, int page_size, AttScale sc, float sink, int window, int num_splits) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ int is_last;
   __shared__ uint64_t full_bar[SQ_STAGES], empty_bar[SQ_STAGES];
   __shared__ int abort_word;
   volatile int* abort_flag = &abort_word;
-  constexpr int STAGE = 2 * BN * D;
+  constexpr int STAGE = BN * (D + VD);
   const uint32_t raw = smem_u32(smem_raw);
   bf16* KV = reinterpret_cast<bf16*>(smem_raw + (((raw + 1023u) & ~1023u) - raw));
   bf16* Qs = KV + SQ_STAGES * STAGE;                          // [16][DP]
@@ -553,9 +596,9 @@ attn_small_q_ws_kernel(const __grid_constant__ CUtensorMap kv_map, int total_row
   __syncthreads();
 
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  float o[D / 8][4];
+  float o[VD / 8][4];
 #pragma unroll
-  for (int n = 0; n < D / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
+  for (int n = 0; n < VD / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
   bool ok = true;
   if (warp == 4) {
     // ---- producer: tile t goes to stage t % S once the consumers have released that stage's previous tile.
@@ -571,8 +614,8 @@ attn_small_q_ws_kernel(const __grid_constant__ CUtensorMap kv_map, int total_row
       }
       if (t >= SQ_STAGES) ok = att_mbar_wait(&empty_bar[stage], ((t / SQ_STAGES) - 1) & 1, abort_flag, err, 3);
       if (!ok) break;
-      tma_issue_tile(&kv_map, KV + stage * STAGE, &full_bar[stage], bt, T0 + t * BN, k_begin, k_end - 1, kvh, nkv, page_size,
-                     ps_shift, total_rows, lane);
+      tma_issue_tile(&k_map, &v_map, KV + stage * STAGE, &full_bar[stage], bt, T0 + t * BN, k_begin, k_end - 1, kvh / share, page_size,
+                     ps_shift, mrows, lane);
     }
   } else {
     // ---- consumers: the query rows (row = token * G + head-in-group), then the tiles
@@ -600,9 +643,9 @@ attn_small_q_ws_kernel(const __grid_constant__ CUtensorMap kv_map, int total_row
       const int tile0 = T0 + t * BN;
       const bool interior = tile0 >= k_begin && tile0 + BN - 1 <= min(p_first, k_end - 1) && (window == 0 || tile0 >= L - window);
       if (interior)
-        warp_tile<2, false, true>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, scale_log2, m, l, o, lane);
+        warp_tile<2, false, true>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, sc, m, l, o, lane);
       else
-        warp_tile<2, true, true>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, scale_log2, m, l, o, lane);
+        warp_tile<2, true, true>(qf, Ks, Vs, warp * 16, tile0, k_begin, k_end - 1, pA, pB, window, sc, m, l, o, lane);
       __syncwarp();
       if (lane == 0) att_mbar_arrive(&empty_bar[stage]);        // this warp is done with the stage
     }
@@ -613,24 +656,24 @@ attn_small_q_ws_kernel(const __grid_constant__ CUtensorMap kv_map, int total_row
     return;
   }
   small_q_finish(reinterpret_cast<float*>(KV), m, l, o, rows, G, q0, kvh, r, split, num_splits, nq, nkv, out, part_o, part_ml,
-                 counters, &is_last);
+                 counters, &is_last, sink);
 }
 
 // --------------------------------------------------------------------------------------------
 // tile kernel: grid (query tiles, kv heads, requests); a warp keeps floor(16/G) tokens x G heads
 // --------------------------------------------------------------------------------------------
 template <bool TMA>
-__global__ void __launch_bounds__(THREADS, D <= 128 ? 3 : 1)      // three CTAs per SM where the accumulators allow
-attn_tile_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, int* __restrict__ err,
-                 const bf16* __restrict__ qkv, int row_stride, const bf16* __restrict__ pages,
+__global__ void __launch_bounds__(THREADS, D <= 128 && VD <= 128 ? 3 : 1)      // three CTAs per SM where the accumulators allow
+attn_tile_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, AttRows mrows,
+                 int* __restrict__ err, const bf16* __restrict__ qkv, int row_stride, AttStream kst, AttStream vst,
                  const int* __restrict__ block_tables, int bt_stride, const int* __restrict__ cu_q,
-                 const int* __restrict__ seq_lens, bf16* __restrict__ out, int nq, int nkv, int page_size,
-                 float scale_log2, int window) {
+                 const int* __restrict__ seq_lens, bf16* __restrict__ out, int nq, int nkv, int share, int page_size,
+                 AttScale sc, float sink, int window) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ uint64_t full_bar[2];
   __shared__ int abort_word;
   volatile int* abort_flag = &abort_word;
-  constexpr int STAGE = TMA ? 2 * BN * D : 2 * BN * DP;
+  constexpr int KT = TMA ? BN * D : BN * DP, STAGE = KT + (TMA ? BN * VD : BN * VDP);
   const uint32_t raw = smem_u32(smem_raw);
   bf16* KV = reinterpret_cast<bf16*>(smem_raw + (TMA ? ((raw + 1023u) & ~1023u) - raw : 0u));
   ifb_pdl_wait();
@@ -663,16 +706,17 @@ attn_tile_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, int
   }
   if (n_tiles > 0) {
     if (TMA) {
-      if (warp == 0) tma_issue_tile(&kv_map, KV, &full_bar[0], bt, T0, lo, hi, kvh, nkv, page_size, ps_shift, total_rows, lane);
+      if (warp == 0)
+        tma_issue_tile(&k_map, &v_map, KV, &full_bar[0], bt, T0, lo, hi, kvh / share, page_size, ps_shift, mrows, lane);
     } else {
-      load_kv_tile(KV, KV + BN * DP, pages, bt, T0, lo, hi, kvh, nkv, page_size, tid);
+      load_kv_tile(KV, KV + KT, kst, vst, bt, T0, lo, hi, kvh / share, page_size, tid);
     }
   }
   if (!TMA) cp_async_commit();
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  float o[D / 8][4];
+  float o[VD / 8][4];
 #pragma unroll
-  for (int n = 0; n < D / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
+  for (int n = 0; n < VD / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
   const int rowA = lane >> 2, rowB = rowA + 8;
   const int tokA = t0 + warp * tpw + rowA / G, tokB = t0 + warp * tpw + rowB / G;
   const int pA = (rowA < tpw * G && tokA < t1) ? p_first + tokA : NO_ROW;
@@ -695,16 +739,16 @@ attn_tile_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, int
   bool ok = true;
   for (int t = 0; t < n_tiles; ++t) {
     bf16* Ks = KV + (t & 1) * STAGE;
-    bf16* Vs = Ks + (TMA ? BN * D : BN * DP);
+    bf16* Vs = Ks + KT;
     // tile t+1 goes to the other stage, which every warp left at the barrier that ended iteration t-1
     if (t + 1 < n_tiles) {
       bf16* Kn = KV + ((t + 1) & 1) * STAGE;
       if (TMA) {
         if (warp == 0)
-          tma_issue_tile(&kv_map, Kn, &full_bar[(t + 1) & 1], bt, T0 + (t + 1) * BN, lo, hi, kvh, nkv, page_size, ps_shift,
-                         total_rows, lane);
+          tma_issue_tile(&k_map, &v_map, Kn, &full_bar[(t + 1) & 1], bt, T0 + (t + 1) * BN, lo, hi, kvh / share, page_size, ps_shift,
+                         mrows, lane);
       } else {
-        load_kv_tile(Kn, Kn + BN * DP, pages, bt, T0 + (t + 1) * BN, lo, hi, kvh, nkv, page_size, tid);
+        load_kv_tile(Kn, Kn + KT, kst, vst, bt, T0 + (t + 1) * BN, lo, hi, kvh / share, page_size, tid);
         cp_async_commit();
       }
     }
@@ -721,9 +765,9 @@ attn_tile_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, int
       const bool interior = t0 + warp * tpw < t1 && tile0 >= lo && tile0 + BN - 1 <= min(hi, p_first + t0 + warp * tpw) &&
                             (window == 0 || tile0 >= warp_hi - window + 1);
       if (interior)
-        warp_tile<8, false, TMA>(qf, Ks, Vs, 0, tile0, lo, hi, pA, pB, window, scale_log2, m, l, o, lane);
+        warp_tile<8, false, TMA>(qf, Ks, Vs, 0, tile0, lo, hi, pA, pB, window, sc, m, l, o, lane);
       else
-        warp_tile<8, true, TMA>(qf, Ks, Vs, 0, tile0, lo, hi, pA, pB, window, scale_log2, m, l, o, lane);
+        warp_tile<8, true, TMA>(qf, Ks, Vs, 0, tile0, lo, hi, pA, pB, window, sc, m, l, o, lane);
     }
     __syncthreads();
   }
@@ -736,109 +780,148 @@ attn_tile_kernel(const __grid_constant__ CUtensorMap kv_map, int total_rows, int
     l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
     l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
   }
-  const float iA = l[0] > 0.f ? 1.f / l[0] : 0.f, iB = l[1] > 0.f ? 1.f / l[1] : 0.f;
+  float iA, iB;
+  if (sink == -INFINITY) {
+    iA = l[0] > 0.f ? 1.f / l[0] : 0.f;
+    iB = l[1] > 0.f ? 1.f / l[1] : 0.f;
+  } else {                                                   // the sink joins the sums: factors against the larger maximum
+    const float MA = fmaxf(m[0], sink), MB = fmaxf(m[1], sink), fA = exp2f(m[0] - MA), fB = exp2f(m[1] - MB);
+    iA = fA / (l[0] * fA + exp2f(sink - MA));
+    iB = fB / (l[1] * fB + exp2f(sink - MB));
+  }
 #pragma unroll
-  for (int n = 0; n < D / 8; ++n) {
+  for (int n = 0; n < VD / 8; ++n) {
     const int col = n * 8 + ((lane & 3) << 1);
     if (pA != NO_ROW) {
-      bf16* dst = out + ((size_t)(q0 + tokA) * nq + kvh * G + rowA % G) * D + col;
+      bf16* dst = out + ((size_t)(q0 + tokA) * nq + kvh * G + rowA % G) * VD + col;
       *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(o[n][0] * iA, o[n][1] * iA);
     }
     if (pB != NO_ROW) {
-      bf16* dst = out + ((size_t)(q0 + tokB) * nq + kvh * G + rowB % G) * D + col;
+      bf16* dst = out + ((size_t)(q0 + tokB) * nq + kvh * G + rowB % G) * VD + col;
       *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(o[n][2] * iB, o[n][3] * iB);
     }
   }
 }
 
 // ---------------------------------------------------------------------------------------------------
+// (the merge of a small-q CTA's warps reuses the stages: 4 * 16 * VD + 128 floats)
 static size_t small_q_smem(bool tma) {
-  return tma ? (size_t)(SQ_STAGES * 2 * BN * D + 16 * DP) * sizeof(bf16) + 1024 : (size_t)(SQ_STAGES * 2 * BN * DP + 16 * DP) * sizeof(bf16);
+  const size_t stages = tma ? (size_t)(SQ_STAGES * BN * (D + VD)) * sizeof(bf16) : (size_t)(SQ_STAGES * BN * (DP + VDP)) * sizeof(bf16);
+  return stages + (size_t)16 * DP * sizeof(bf16) + (tma ? 1024 : 0);
 }
+static_assert((size_t)SQ_STAGES * BN * (D + VD) * sizeof(bf16) >= (size_t)(4 * 16 * VD + 128) * sizeof(float),
+              "the merge of the warps' sums must fit in the stages");
 static size_t tile_smem(bool tma) {
-  return tma ? (size_t)(2 * 2 * BN * D) * sizeof(bf16) + 1024 : (size_t)(2 * 2 * BN * DP) * sizeof(bf16);
+  return tma ? (size_t)(2 * BN * (D + VD)) * sizeof(bf16) + 1024 : (size_t)(2 * BN * (DP + VDP)) * sizeof(bf16);
 }
 
-// The pool [pages, 2, kv_heads, page_size, D] as a matrix [rows, D] with boxes of page_size rows x 64 columns in
-// the 128-byte swizzle.
-static int kv_tensor_map(CUtensorMap* out, const void* pages, long long rows, int page_size) {
-  const unsigned long long dims[2] = {(unsigned long long)D, (unsigned long long)rows};
-  const unsigned long long strides[1] = {(unsigned long long)D * sizeof(bf16)};
+// A stream as a matrix [rows, width] with boxes of page_size rows x 64 columns in the 128-byte swizzle.
+static int kv_tensor_map(CUtensorMap* out, const void* base, long long rows, int width, int page_size) {
+  const unsigned long long dims[2] = {(unsigned long long)width, (unsigned long long)rows};
+  const unsigned long long strides[1] = {(unsigned long long)width * sizeof(bf16)};
   const unsigned box[2] = {64, (unsigned)page_size};
-  return ifb_tensor_map_bf16(out, pages, 2, dims, strides, box);
+  return ifb_tensor_map_bf16(out, base, 2, dims, strides, box);
 }
 
 IFB_EXPORT int ifb_attention_mma_head_dim() { return D; }
 
 // Floats of scratch the small-q kernel needs for `n_tokens` tokens of `nq` heads in `num_splits` splits.
 IFB_EXPORT long long ifb_attention_mma_scratch_floats(int n_tokens, int nq, int num_splits) {
-  return num_splits > 1 ? (long long)n_tokens * nq * num_splits * (D + 2) : 0;
+  return num_splits > 1 ? (long long)n_tokens * nq * num_splits * (VD + 2) : 0;
 }
 
+struct AttArgs {
+  CUtensorMap k_map, v_map;
+  AttRows rows;
+  AttStream k, v;
+  int* err;
+  const void* qkv;
+  int row_stride;
+  const int *block_tables, *cu_q, *seq_lens;
+  int bt_stride;
+  void* out;
+  float* scratch;
+  int* counters;
+  int n_tokens, n_req, nq, nkv, share, page_size, window, max_q_len, num_splits, run_small, run_tiles;
+  AttScale sc;
+  float sink;
+};
+
 template <bool TMA>
-static int att_launch(const CUtensorMap& map, int total_rows, int* err, const void* qkv, int row_stride, const void* pages,
-                      const int* block_tables, int bt_stride, const int* cu_q, const int* seq_lens, void* out, float* scratch,
-                      int* counters, int n_tokens, int n_req, int nq, int nkv, int page_size, float scale_log2, int window,
-                      int max_q_len, int num_splits, int run_small, int run_tiles, cudaStream_t stream) {
+static int att_launch(const AttArgs& a, cudaStream_t stream) {
   if (TMA) IFB_ALLOW_SMEM(attn_small_q_ws_kernel, small_q_smem(true));
   else IFB_ALLOW_SMEM(attn_small_q_kernel<false>, small_q_smem(false));
   IFB_ALLOW_SMEM(attn_tile_kernel<TMA>, tile_smem(TMA));
-  const int G = nq / nkv;
-  if (run_small) {
-    float* part_o = scratch;
-    float* part_ml = scratch ? scratch + (size_t)n_tokens * nq * num_splits * D : nullptr;
-    dim3 grid(num_splits, nkv, n_req);
+  const int G = a.nq / a.nkv;
+  if (a.run_small) {
+    float* part_o = a.scratch;
+    float* part_ml = a.scratch ? a.scratch + (size_t)a.n_tokens * a.nq * a.num_splits * VD : nullptr;
+    dim3 grid(a.num_splits, a.nkv, a.n_req);
     int st;
     if (TMA)
-      st = ifb_launch(attn_small_q_ws_kernel, grid, dim3(WS_THREADS), small_q_smem(true), stream, map, total_rows, err,
-                      (const bf16*)qkv, row_stride, block_tables, bt_stride, cu_q, seq_lens, (bf16*)out, part_o, part_ml,
-                      counters, nq, nkv, page_size, scale_log2, window, num_splits);
+      st = ifb_launch(attn_small_q_ws_kernel, grid, dim3(WS_THREADS), small_q_smem(true), stream, a.k_map, a.v_map, a.rows, a.err,
+                      (const bf16*)a.qkv, a.row_stride, a.block_tables, a.bt_stride, a.cu_q, a.seq_lens, (bf16*)a.out, part_o, part_ml,
+                      a.counters, a.nq, a.nkv, a.share, a.page_size, a.sc, a.sink, a.window, a.num_splits);
     else
-      st = ifb_launch(attn_small_q_kernel<false>, grid, dim3(THREADS), small_q_smem(false), stream, map, total_rows, err,
-                      (const bf16*)qkv, row_stride, (const bf16*)pages, block_tables, bt_stride, cu_q, seq_lens, (bf16*)out,
-                      part_o, part_ml, counters, nq, nkv, page_size, scale_log2, window, num_splits);
+      st = ifb_launch(attn_small_q_kernel<false>, grid, dim3(THREADS), small_q_smem(false), stream, a.k_map, a.v_map, a.rows, a.err,
+                      (const bf16*)a.qkv, a.row_stride, a.k, a.v, a.block_tables, a.bt_stride, a.cu_q, a.seq_lens, (bf16*)a.out, part_o,
+                      part_ml, a.counters, a.nq, a.nkv, a.share, a.page_size, a.sc, a.sink, a.window, a.num_splits);
     if (st) return st;
   }
-  if (run_tiles) {
+  if (a.run_tiles) {
     const int tpc = 4 * (16 / G);
-    dim3 grid((max_q_len + tpc - 1) / tpc, nkv, n_req);
-    return ifb_launch(attn_tile_kernel<TMA>, grid, dim3(THREADS), tile_smem(TMA), stream, map, total_rows, err, (const bf16*)qkv,
-                      row_stride, (const bf16*)pages, block_tables, bt_stride, cu_q, seq_lens, (bf16*)out, nq, nkv, page_size,
-                      scale_log2, window);
+    dim3 grid((a.max_q_len + tpc - 1) / tpc, a.nkv, a.n_req);
+    return ifb_launch(attn_tile_kernel<TMA>, grid, dim3(THREADS), tile_smem(TMA), stream, a.k_map, a.v_map, a.rows, a.err,
+                      (const bf16*)a.qkv, a.row_stride, a.k, a.v, a.block_tables, a.bt_stride, a.cu_q, a.seq_lens, (bf16*)a.out, a.nq,
+                      a.nkv, a.share, a.page_size, a.sc, a.sink, a.window);
   }
   return IFB_OK;
 }
 
-// max_q_len: the most query tokens any request brings.  run_small / run_tiles: which of the two kernels to
-// launch; requests are routed by rows = q_len * (nq / nkv) <= 16.  num_pages: pages of the pool `pages`.
-// err: a device int that stays 0 unless a bounded wait gave up (TMA path).  use_tma 0 forces the cp.async path.
-IFB_EXPORT int ifb_attention_mma(const void* qkv, int row_stride, const void* pages, long long num_pages,
-                                 const int* block_tables, int bt_stride, const int* cu_q, const int* seq_lens, void* out,
-                                 float* scratch, int* counters, int* err, int n_tokens, int n_req, int nq, int nkv, int d,
-                                 int page_size, float scale, int window, int max_q_len, int num_splits, int run_small,
-                                 int run_tiles, int use_tma, cudaStream_t stream) {
+// qkv: the q heads are the first nq * d columns of its rows.  k_pages / v_pages: the two streams, pages k_page_stride /
+// v_page_stride elements apart, num_pages of them, each [kv heads][page_size][d or dv].  nkv: groups of query heads, `share`
+// of which read one key/value head.  max_q_len: the most query tokens any request brings.  run_small / run_tiles: which of the
+// two kernels to launch; requests are routed by rows = q_len * (nq / nkv) <= 16.  err: a device int that stays 0 unless a
+// bounded wait gave up (TMA path).  use_tma 0 forces the cp.async path.  softcap: 0 none (a library compiled with SOFTCAP
+// takes a positive one and no other takes one).  has_sink: exp(sink) joins the denominators.
+IFB_EXPORT int ifb_attention_mma(const void* qkv, int row_stride, const void* k_pages, long long k_page_stride, const void* v_pages,
+                                 long long v_page_stride, long long num_pages, const int* block_tables, int bt_stride, const int* cu_q,
+                                 const int* seq_lens, void* out, float* scratch, int* counters, int* err, int n_tokens, int n_req,
+                                 int nq, int nkv, int share, int d, int dv, int page_size, float scale, int window, float softcap,
+                                 int has_sink, float sink, int max_q_len, int num_splits, int run_small, int run_tiles, int use_tma,
+                                 cudaStream_t stream) {
   if (n_tokens <= 0 || n_req <= 0) return IFB_OK;
-  if (d != D) return IFB_ERR_SIZE;
-  if (nkv < 1 || nq % nkv || page_size < 1 || window < 0 || num_splits < 1) return IFB_ERR_ARG;
-  const int G = nq / nkv;
-  if (G > 16 && run_tiles) return IFB_ERR_SIZE;
-  if (row_stride % 8 || ((uintptr_t)qkv & 15) || ((uintptr_t)pages & 15) || ((uintptr_t)out & 3)) return IFB_ERR_ALIGN;
+  if (d != D || dv != VD) return IFB_ERR_SIZE;
+  if (nkv < 1 || nq % nkv || share < 1 || nkv % share || page_size < 1 || window < 0 || num_splits < 1 || num_pages < 1) return IFB_ERR_ARG;
+  if (SOFTCAP ? !(softcap > 0.f) : softcap != 0.f) return IFB_ERR_ARG;
+  const int G = nq / nkv, heads = nkv / share;
+  if (G > 16) return IFB_ERR_SIZE;
+  if (row_stride % 8 || (((uintptr_t)qkv | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) || ((uintptr_t)out & 3) || k_page_stride % 8 ||
+      v_page_stride % 8)
+    return IFB_ERR_ALIGN;
+  if (k_page_stride < (long long)heads * page_size * D || v_page_stride < (long long)heads * page_size * VD) return IFB_ERR_ARG;
   if (n_req > 65535 || nkv > 65535) return IFB_ERR_SIZE;
   if (run_small && num_splits > 1 && (!scratch || !counters)) return IFB_ERR_ARG;
-  const float scale_log2 = scale * 1.4426950408889634f;
-  const long long rows = num_pages * 2 * nkv * page_size;
-  const bool tma = use_tma && TMA_D && err && (page_size == 16 || page_size == 32 || page_size == 64) && rows < 0x7fffffffLL &&
-                   ((uintptr_t)pages & 127) == 0;
-  CUtensorMap map;
-  if (tma) {
-    int st = kv_tensor_map(&map, pages, rows, page_size);
-    if (st) return st;
-    return att_launch<true>(map, (int)rows, err, qkv, row_stride, pages, block_tables, bt_stride, cu_q, seq_lens, out, scratch,
-                            counters, n_tokens, n_req, nq, nkv, page_size, scale_log2, window, max_q_len, num_splits, run_small,
-                            run_tiles, stream);
-  }
-  memset(&map, 0, sizeof(map));
-  return att_launch<false>(map, 0, err, qkv, row_stride, pages, block_tables, bt_stride, cu_q, seq_lens, out, scratch, counters,
-                           n_tokens, n_req, nq, nkv, page_size, scale_log2, window, max_q_len, num_splits, run_small, run_tiles,
-                           stream);
+  constexpr float LOG2E = 1.4426950408889634f;
+  AttArgs a;
+  memset(&a, 0, sizeof(a));
+  a.k = {(const bf16*)k_pages, k_page_stride};
+  a.v = {(const bf16*)v_pages, v_page_stride};
+  a.err = err; a.qkv = qkv; a.row_stride = row_stride; a.block_tables = block_tables; a.bt_stride = bt_stride; a.cu_q = cu_q;
+  a.seq_lens = seq_lens; a.out = out; a.scratch = scratch; a.counters = counters; a.n_tokens = n_tokens; a.n_req = n_req; a.nq = nq;
+  a.nkv = nkv; a.share = share; a.page_size = page_size; a.window = window; a.max_q_len = max_q_len; a.num_splits = num_splits;
+  a.run_small = run_small; a.run_tiles = run_tiles;
+  a.sc = SOFTCAP ? AttScale{softcap * LOG2E, 2.f * scale * LOG2E / softcap} : AttScale{scale * LOG2E, 0.f};
+  a.sink = has_sink ? sink * LOG2E : -INFINITY;
+  const long long k_page = k_page_stride / D, v_page = v_page_stride / VD;
+  const long long k_rows = (num_pages - 1) * k_page + (long long)heads * page_size, v_rows = (num_pages - 1) * v_page + (long long)heads * page_size;
+  const bool tma = use_tma && TMA_D && err && (page_size == 16 || page_size == 32 || page_size == 64) && k_page_stride % D == 0 &&
+                   v_page_stride % VD == 0 && k_rows < 0x7fffffffLL && v_rows < 0x7fffffffLL;
+  if (!tma) return att_launch<false>(a, stream);
+  a.rows = {(int)k_page, (int)v_page, (int)k_rows, (int)v_rows};
+  int st = kv_tensor_map(&a.k_map, k_pages, k_rows, D, page_size);
+  if (st) return st;
+  st = kv_tensor_map(&a.v_map, v_pages, v_rows, VD, page_size);
+  if (st) return st;
+  return att_launch<true>(a, stream);
 }

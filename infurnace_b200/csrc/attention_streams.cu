@@ -9,7 +9,8 @@
 //
 // (2) paged_attention_streams: one warp per (query token, query head); float32 scores, softmax weights and sums,
 // whatever the storage.  A query at position p reads the keys at positions first .. p from the pages of its request,
-// first = max(0, p - window + 1) with a window, else 0.  After the division by the softmax sum the head's output is
+// first = max(0, p - window + 1) with a window, else 0.  With a soft cap c a scaled score s becomes c tanh(s / c); with a
+// sink z, exp(z) joins the denominator.  After the division by the softmax sum the head's output is
 // rotated BACK by the query token's angles (optional): (u, v) becomes (u c + v s, v c - u s).
 //
 // Head sizes up to 256 for keys and for values, any page size, any grouping.
@@ -127,7 +128,7 @@ paged_attention_streams_kernel(const T* __restrict__ q, const T* __restrict__ k_
                                const T* __restrict__ v_pages, long long v_page_stride, const int* __restrict__ block_tables,
                                int bt_stride, const int* __restrict__ cu_q, const int* __restrict__ seq_lens, T* __restrict__ out,
                                int n_tokens, int n_req, int H, int G, int d, int dv, int page_size, float scale, int window,
-                               const float* __restrict__ out_table, int out_interleaved) {
+                               const float* __restrict__ out_table, int out_interleaved, float softcap, float sink) {
   extern __shared__ float sm[];
   ifb_pdl_wait();
   ifb_pdl_trigger();
@@ -150,7 +151,7 @@ paged_attention_streams_kernel(const T* __restrict__ q, const T* __restrict__ k_
   for (int i = lane; i < d; i += 32) qs[i] = to_f32<T>(qp[i]);
   __syncwarp();
   const int* bt = block_tables + (size_t)r * bt_stride;
-  float m = -INFINITY, l = 0.f;
+  float m = sink, l = sink == -INFINITY ? 0.f : 1.f;      // the sink (-inf: none) stands as a key without a value
   float acc[AS_MAX_D / 32];
 #pragma unroll
   for (int c = 0; c < AS_MAX_D / 32; ++c) acc[c] = 0.f;
@@ -164,6 +165,7 @@ paged_attention_streams_kernel(const T* __restrict__ q, const T* __restrict__ k_
       float dot = 0.f;
       for (int i = 0; i < d; ++i) dot = fmaf(qs[i], to_f32<T>(kp[i]), dot);
       s = dot * scale;
+      if (softcap > 0.f) s = softcap * tanhf(s / softcap);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float pj = valid ? expf(s - m_new) : 0.f;
@@ -208,7 +210,7 @@ IFB_EXPORT int ifb_paged_attention_streams(const void* q, int dtype, const void*
                                            const void* v_pages, long long v_page_stride, const int* block_tables, int bt_stride,
                                            const int* cu_q, const int* seq_lens, void* out, int n_tokens, int n_req, int H, int G,
                                            int d, int dv, int page_size, float scale, int window, const float* out_table,
-                                           int out_interleaved, cudaStream_t stream) {
+                                           int out_interleaved, float softcap, float sink, cudaStream_t stream) {
   if (n_tokens <= 0 || n_req <= 0) return IFB_OK;
   if (d < 1 || d > AS_MAX_D || dv < 1 || dv > AS_MAX_D) return IFB_ERR_SIZE;
   if (G < 1 || H % G || page_size < 1 || window < 0 || (out_table && dv % 2)) return IFB_ERR_ARG;
@@ -219,11 +221,12 @@ IFB_EXPORT int ifb_paged_attention_streams(const void* q, int dtype, const void*
   if (dtype == IFB_F32)
     return ifb_launch(paged_attention_streams_kernel<float>, dim3(blocks), dim3(warps * 32), smem, stream, (const float*)q,
                       (const float*)k_pages, k_page_stride, (const float*)v_pages, v_page_stride, block_tables, bt_stride, cu_q,
-                      seq_lens, (float*)out, n_tokens, n_req, H, G, d, dv, page_size, scale, window, out_table, out_interleaved);
+                      seq_lens, (float*)out, n_tokens, n_req, H, G, d, dv, page_size, scale, window, out_table, out_interleaved,
+                      softcap, sink);
   if (dtype == IFB_BF16)
     return ifb_launch(paged_attention_streams_kernel<__nv_bfloat16>, dim3(blocks), dim3(warps * 32), smem, stream,
                       (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, k_page_stride, (const __nv_bfloat16*)v_pages,
                       v_page_stride, block_tables, bt_stride, cu_q, seq_lens, (__nv_bfloat16*)out, n_tokens, n_req, H, G, d, dv,
-                      page_size, scale, window, out_table, out_interleaved);
+                      page_size, scale, window, out_table, out_interleaved, softcap, sink);
   return IFB_ERR_DTYPE;
 }

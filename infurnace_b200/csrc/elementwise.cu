@@ -5,12 +5,12 @@
 #include <math.h>
 
 // ------------------------------------------------------------------------------------------
-// embed: out[n, :] = float(table[ids[n], :])
+// embed: out[n, :] = scale * float(table[ids[n], :])
 // An id outside [0, vocab) (ids may come straight from the sampling kernel of the step before, unseen by the
 // host) reads no memory: the row is written as zeros and IFB_DEV_ERR_TOKEN_ID is recorded in *err (if given).
 // ------------------------------------------------------------------------------------------
 __global__ void embed_kernel(const void* __restrict__ table, int table_dtype, const int* __restrict__ ids,
-                             float* __restrict__ out, int hidden, int vocab, int* __restrict__ err) {
+                             float* __restrict__ out, int hidden, int vocab, int* __restrict__ err, float scale) {
   ifb_pdl_wait();
   ifb_pdl_trigger();
   const int n = blockIdx.x;
@@ -22,15 +22,15 @@ __global__ void embed_kernel(const void* __restrict__ table, int table_dtype, co
   }
   const size_t row = (size_t)id * hidden;
   for (int h = threadIdx.x; h < hidden; h += blockDim.x)
-    out[(size_t)n * hidden + h] = load_as_f32(table, table_dtype, row + h);
+    out[(size_t)n * hidden + h] = load_as_f32(table, table_dtype, row + h) * scale;
 }
 
 IFB_EXPORT int ifb_embed(const void* table, int table_dtype, const int* ids, float* out, int n, int hidden, int vocab,
-                         int* err, cudaStream_t stream) {
+                         int* err, float scale, cudaStream_t stream) {
   if (n <= 0) return IFB_OK;
   if (table_dtype != IFB_F32 && table_dtype != IFB_BF16) return IFB_ERR_DTYPE;
   if (vocab < 1) return IFB_ERR_SIZE;
-  return ifb_launch(embed_kernel, dim3(n), dim3(256), 0, stream, table, table_dtype, ids, out, hidden, vocab, err);
+  return ifb_launch(embed_kernel, dim3(n), dim3(256), 0, stream, table, table_dtype, ids, out, hidden, vocab, err, scale);
 }
 
 // ------------------------------------------------------------------------------------------

@@ -157,6 +157,7 @@ struct TcFold {
   int res_g_dtype;
   float* res_partials;        // [parts][n_rows], written; what a part covers depends on the launch (tc_fold_parts)
   int unary;                  // plain epilogue without res_x: the function of common.cuh applied to every element (0: none)
+  const float* bias;          // plain epilogue: [o_out], added to the product before the unary function (null: none)
   // The product is the fused q | k | v projection of an attention layer with heads of 128, in the shared-k form, whose
   // tile of 128 features is one head: the sum over the cluster finishes what follows the projection (RMSNorm over the q
   // and k heads, rotation in the half-split pairing, q to its row, k and v to the token's place in the pages).
@@ -381,6 +382,10 @@ linear_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
             tmem_ld_wait();
 #pragma unroll
             for (int j = 0; j < 32; ++j) y[j] = __uint_as_float(v[j]) * rfac;
+            if (fold.bias) {                                     // warp-uniform; every lane holds the same 32 features
+#pragma unroll
+              for (int j = 0; j < 32; ++j) y[j] += n0 + c0 + j < o_out ? __ldg(fold.bias + n0 + c0 + j) : 0.f;
+            }
             if (fold.unary) {                                    // warp-uniform
 #pragma unroll
               for (int j = 0; j < 32; ++j) y[j] = ifb_unary(y[j], fold.unary);
@@ -457,6 +462,13 @@ linear_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
         acc.w = acc.w * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * acc.w)) * up.w;
       }
       TO* dst = out + (size_t)(m0 + r) * o_out + n0 + c;
+      if (!EPI && fold.bias) {
+        const float* bp = fold.bias + n0 + c;
+        if (c < cols) acc.x += __ldg(bp);
+        if (c + 1 < cols) acc.y += __ldg(bp + 1);
+        if (c + 2 < cols) acc.z += __ldg(bp + 2);
+        if (c + 3 < cols) acc.w += __ldg(bp + 3);
+      }
       if (!EPI && fold.unary) {
         acc.x = ifb_unary(acc.x, fold.unary); acc.y = ifb_unary(acc.y, fold.unary);
         acc.z = ifb_unary(acc.z, fold.unary); acc.w = ifb_unary(acc.w, fold.unary);
@@ -712,6 +724,10 @@ linear_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_x, con
             tmem_ld_wait();
 #pragma unroll
             for (int j = 0; j < 32; ++j) y[j] = __uint_as_float(v[j]) * rfac;
+            if (fold.bias) {                                     // warp-uniform; every lane holds the same 32 features
+#pragma unroll
+              for (int j = 0; j < 32; ++j) y[j] += n0 + c0 + j < o_out ? __ldg(fold.bias + n0 + c0 + j) : 0.f;
+            }
             if (fold.unary) {                                    // warp-uniform
 #pragma unroll
               for (int j = 0; j < 32; ++j) y[j] = ifb_unary(y[j], fold.unary);
@@ -878,16 +894,18 @@ static int tc_launch(const void* x, const void* w, void* out, int n, int o, int 
 // rsqrt(sum_p partials[p][n] / scale_width + scale_eps) before the epilogue.
 // res_x (may be null; plain epilogue, shape 0-3): the residual stream [n_rows][out_features] float32: v = x + y is
 // written back to it, out = v * res_g, and res_partials [ifb_linear_tcgen05_fold_parts(...)][n_rows] gets sums of v^2.
+// bias (may be null; plain epilogue): float32 [out_features], added to the (scaled) product.
 IFB_EXPORT int ifb_linear_tcgen05_ex(const void* x, const void* w, void* out, int out_dtype, int n_rows, int out_features,
                                      int k_dim, int epilogue, int shape, int splits, const float* scale_partials, int scale_parts,
                                      float scale_eps, int scale_width, float* res_x, const void* res_g, int res_g_dtype,
-                                     float* res_partials, int* err, cudaStream_t stream) {
+                                     float* res_partials, const float* bias, int* err, cudaStream_t stream) {
   if (n_rows <= 0 || out_features <= 0) return IFB_OK;
   if (k_dim < 8 || k_dim % 8) return IFB_ERR_SIZE;
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return IFB_ERR_ALIGN;
   const int unary = epilogue >> 4;
   epilogue &= 15;
-  if (epilogue > 1 || unary < 0 || unary > IFB_UNARY_LAST || (unary && (epilogue || res_x))) return IFB_ERR_ARG;
+  if (epilogue > 1 || unary < 0 || unary > IFB_UNARY_LAST || (unary && (epilogue || res_x)) || (bias && epilogue))
+    return IFB_ERR_ARG;
   if (shape < 0 || shape > 5 || splits < 0 || splits > 8) return IFB_ERR_ARG;
   if (scale_partials && (scale_parts < 1 || scale_width < 1)) return IFB_ERR_ARG;
   if (res_x && (!res_g || !res_partials || ((uintptr_t)res_x & 15))) return IFB_ERR_ARG;
@@ -896,6 +914,7 @@ IFB_EXPORT int ifb_linear_tcgen05_ex(const void* x, const void* w, void* out, in
   fold.rs_inv_width = scale_partials ? 1.f / (float)scale_width : 0.f;
   fold.res_x = res_x; fold.res_g = res_g; fold.res_g_dtype = res_g_dtype; fold.res_partials = res_partials;
   fold.unary = unary;
+  fold.bias = bias;
   if (out_dtype == IFB_BF16)
     return epilogue ? tc_launch<1, bf16>(x, w, out, n_rows, out_features, k_dim, err, shape, splits, fold, stream)
                     : tc_launch<0, bf16>(x, w, out, n_rows, out_features, k_dim, err, shape, splits, fold, stream);
@@ -914,8 +933,11 @@ IFB_EXPORT int ifb_linear_tcgen05_grouped(const void* x, const void* w, void* ou
   if (rows <= 0 || out_features <= 0) return IFB_OK;
   if (k_dim < 8 || k_dim % 8 || rows % G_BM || experts < 1) return IFB_ERR_SIZE;
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return IFB_ERR_ALIGN;
-  if ((epilogue != 0 && epilogue != 1) || !tile_expert) return IFB_ERR_ARG;
+  const int unary = epilogue >> 4;
+  epilogue &= 15;
+  if (epilogue > 1 || unary < 0 || unary > IFB_UNARY_LAST || (epilogue && unary) || !tile_expert) return IFB_ERR_ARG;
   TcFold fold = {};
+  fold.unary = unary;
   fold.grp_tile_expert = tile_expert;
   fold.grp_w_rows = (epilogue ? 2 : 1) * out_features;
   const long long w_rows = (long long)experts * fold.grp_w_rows;
@@ -933,7 +955,7 @@ IFB_EXPORT int ifb_linear_tcgen05_grouped(const void* x, const void* w, void* ou
 IFB_EXPORT int ifb_linear_tcgen05(const void* x, const void* w, void* out, int out_dtype, int n_rows, int out_features,
                                   int k_dim, int epilogue, int* err, int shape, cudaStream_t stream) {
   return ifb_linear_tcgen05_ex(x, w, out, out_dtype, n_rows, out_features, k_dim, epilogue, shape, 1, nullptr, 0, 0.f, 0, nullptr,
-                               nullptr, 0, nullptr, err, stream);
+                               nullptr, 0, nullptr, nullptr, err, stream);
 }
 
 // The fused q | k | v projection of an attention layer in the shared-k form with what follows it in the sum over the

@@ -11,12 +11,15 @@
 // mode 0: the scores are the logits, and gates[n][j] is the softmax over the chosen logits only.  mode 1: the scores are
 // the softmax over all experts, only experts of the `keep` groups (of `groups` equal groups of neighbours) whose best score
 // is largest can be chosen, and gates[n][j] = score * wscale, not renormalised.  mode 2: the scores are sigmoid(logit) per
-// expert (the order of the logits is the order of the scores), gates[n][j] = score * wscale.  A row of logits has `stride` entries, of
+// expert (the order of the logits is the order of the scores), gates[n][j] = score * wscale.  mode 3: the scores are
+// sigmoid(logit); what is chosen by is score + corr[e] (corr null: the score), within the `keep` best groups as in mode 1;
+// gates[n][j] = score * wscale, with `norm` divided by the sum of the chosen scores + 1e-20.  A group's value in modes 1
+// and 3 is the sum of its `gbest` (1 or 2) largest scores (with the correction).  A row of logits has `stride` entries, of
 // which the first `experts` are the router's.  A warp per row; a lane holds the logits e = lane, lane + 32, ... (up to
 // MR_PER_LANE * 32 experts); lane j keeps the j-th chosen score (up to 32 choices).
 // ------------------------------------------------------------------------------------------
 constexpr int MR_PER_LANE = 8;
-struct MrMode { int stride, mode, groups, keep; float wscale; };
+struct MrMode { int stride, mode, groups, keep; float wscale; const float* corr; int gbest, norm; };
 __device__ __forceinline__ void mr_route_row(const float* __restrict__ logits, int* __restrict__ ids, float* __restrict__ gates,
                                              int row, int experts, int top, int lane, MrMode md) {
   float val[MR_PER_LANE];
@@ -36,6 +39,14 @@ __device__ __forceinline__ void mr_route_row(const float* __restrict__ logits, i
     tot = warp_sum(tot);
 #pragma unroll
     for (int j = 0; j < MR_PER_LANE; ++j) val[j] = lane + 32 * j < experts ? val[j] / tot : -INFINITY;
+  } else if (md.mode == 3) {
+#pragma unroll
+    for (int j = 0; j < MR_PER_LANE; ++j) {
+      const int e = lane + 32 * j;
+      if (e < experts) val[j] = 1.f / (1.f + expf(-val[j])) + (md.corr ? md.corr[e] : 0.f);
+    }
+  }
+  if (md.mode == 1 || md.mode == 3) {
     if (md.groups > 1 && md.keep < md.groups) {
       const int gsz = experts / md.groups;
       float gbest[MR_PER_LANE];                         // lane holds the best score of groups lane, lane + 32, ...
@@ -46,6 +57,17 @@ __device__ __forceinline__ void mr_route_row(const float* __restrict__ logits, i
 #pragma unroll
         for (int j = 0; j < MR_PER_LANE; ++j) { const int e = lane + 32 * j; if (e < experts && e / gsz == g) b = fmaxf(b, val[j]); }
         b = warp_max(b);
+        if (md.gbest == 2 && gsz > 1) {                 // the second largest: the largest without one holder of the largest
+          int at = 0x7fffffff;
+#pragma unroll
+          for (int j = 0; j < MR_PER_LANE; ++j) { const int e = lane + 32 * j; if (e < experts && e / gsz == g && val[j] == b) at = min(at, e); }
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) at = min(at, __shfl_xor_sync(0xffffffffu, at, o));
+          float b2 = -INFINITY;
+#pragma unroll
+          for (int j = 0; j < MR_PER_LANE; ++j) { const int e = lane + 32 * j; if (e < experts && e / gsz == g && e != at) b2 = fmaxf(b2, val[j]); }
+          b += warp_max(b2);
+        }
 #pragma unroll
         for (int j = 0; j < MR_PER_LANE; ++j) if ((g & 31) == lane && (g >> 5) == j) gbest[j] = b;
       }
@@ -75,7 +97,8 @@ __device__ __forceinline__ void mr_route_row(const float* __restrict__ logits, i
     }
   }
   unsigned taken = 0;                                   // bit j: this lane's j-th logit is chosen already
-  float first = 0.f, mine = -INFINITY, sum = 0.f;       // lane j < top keeps the j-th chosen logit
+  float first = 0.f, mine = -INFINITY, sum = 0.f;       // lane j < top keeps the j-th chosen logit (and its index)
+  int mine_e = 0;
   for (int t = 0; t < top; ++t) {
     float best = -INFINITY;
     int best_e = 0x7fffffff;
@@ -92,7 +115,7 @@ __device__ __forceinline__ void mr_route_row(const float* __restrict__ logits, i
     }
     if ((best_e & 31) == lane && best_e < experts) taken |= 1u << (best_e >> 5);
     if (t == 0) first = best;
-    if (lane == t) mine = best;
+    if (lane == t) { mine = best; mine_e = best_e < experts ? best_e : 0; }
     if (lane == 0) ids[(size_t)row * top + t] = best_e < experts ? best_e : 0;
   }
   if (md.mode == 1) {
@@ -101,6 +124,14 @@ __device__ __forceinline__ void mr_route_row(const float* __restrict__ logits, i
   }
   if (md.mode == 2) {
     if (lane < top) gates[(size_t)row * top + lane] = md.wscale / (1.f + expf(-mine));
+    return;
+  }
+  if (md.mode == 3) {
+    // the weight is the score itself, without the correction: lane t forms it for the t-th chosen expert
+    const float s = lane < top ? 1.f / (1.f + expf(-logits[(size_t)row * md.stride + mine_e])) : 0.f;
+    float w = s * md.wscale;
+    if (md.norm) w /= warp_sum(s) + 1e-20f;
+    if (lane < top) gates[(size_t)row * top + lane] = w;
     return;
   }
   const float p = lane < top ? expf(mine - first) : 0.f;
@@ -146,26 +177,26 @@ moe_route_plan_small_kernel(const float* __restrict__ logits, int* __restrict__ 
 }
 
 static bool mr_mode_ok(const MrMode& md, int experts) {
-  return md.stride >= experts && md.mode >= 0 && md.mode <= 2 && md.groups >= 1 && md.keep >= 1 && md.keep <= md.groups &&
-         experts % md.groups == 0;
+  return md.stride >= experts && md.mode >= 0 && md.mode <= 3 && md.groups >= 1 && md.keep >= 1 && md.keep <= md.groups &&
+         experts % md.groups == 0 && (md.gbest == 1 || md.gbest == 2);
 }
 
 IFB_EXPORT int ifb_moe_route_plan_small(const float* logits, int* ids, float* gates, int rows, int experts, int top, int* offsets,
                                         int* perm, int* pos, int stride, int mode, int groups, int keep, float wscale,
-                                        cudaStream_t stream) {
+                                        const float* corr, int gbest, int norm, cudaStream_t stream) {
   if (rows <= 0) return IFB_OK;
   if (experts < 1 || experts > MS_THREADS || top < 1 || top > experts || top > 32 || (long long)rows * top > 4096) return IFB_ERR_SIZE;
-  const MrMode md{stride, mode, groups, keep, wscale};
+  const MrMode md{stride, mode, groups, keep, wscale, corr, gbest, norm};
   if (!mr_mode_ok(md, experts)) return IFB_ERR_ARG;
   return ifb_launch(moe_route_plan_small_kernel, dim3(1), dim3(MS_THREADS), 0, stream, logits, ids, gates, rows, experts, top,
                     offsets, perm, pos, md);
 }
 
 IFB_EXPORT int ifb_moe_route(const float* logits, int* ids, float* gates, int rows, int experts, int top, int stride, int mode,
-                             int groups, int keep, float wscale, cudaStream_t stream) {
+                             int groups, int keep, float wscale, const float* corr, int gbest, int norm, cudaStream_t stream) {
   if (rows <= 0) return IFB_OK;
   if (experts < 1 || experts > 32 * MR_PER_LANE || top < 1 || top > experts || top > 32) return IFB_ERR_SIZE;
-  const MrMode md{stride, mode, groups, keep, wscale};
+  const MrMode md{stride, mode, groups, keep, wscale, corr, gbest, norm};
   if (!mr_mode_ok(md, experts)) return IFB_ERR_ARG;
   return ifb_launch(moe_route_kernel, dim3((rows + 3) / 4), dim3(128), 0, stream, logits, ids, gates, rows, experts, top, md);
 }
@@ -365,7 +396,8 @@ IFB_EXPORT int ifb_moe_gather_scaled(const void* x, int dtype, const int* perm, 
 // ------------------------------------------------------------------------------------------
 // The grouped product.  Row i of `out` belongs to the expert e with offsets[e] <= i < offsets[e + 1] and is
 //     x[src(i)] w[e]^T,   src(i) = perm[i] / top (perm null: i),   w [experts][o_w][k]
-// GATED: w[e] holds o gate rows and then o up rows, and out[i][j] = silu(gate_j) * up_j.  A block is a tile of ML_ROWS
+// GATED: w[e] holds o gate rows and then o up rows, and out[i][j] = silu(gate_j) * up_j.  Else out[i][j] = unary(y_j), the
+// function of common.cuh (0: y itself).  A block is a tile of ML_ROWS
 // rows of one expert by ML_COLS outputs; block row y is the y-th tile in the order of the experts (each expert's rows
 // are tiled on their own; block rows beyond the last tile return).  A thread owns 2 rows x 4 outputs.
 // ------------------------------------------------------------------------------------------
@@ -373,7 +405,7 @@ constexpr int ML_ROWS = 32, ML_COLS = 64, ML_K = 32, ML_THREADS = 256;
 template <typename TA, typename TW, typename TO, bool GATED>
 __global__ void __launch_bounds__(ML_THREADS)
 moe_linear_kernel(const TA* __restrict__ x, const TW* __restrict__ w, const int* __restrict__ offsets,
-                  const int* __restrict__ perm, int top, TO* __restrict__ out, int experts, int o, int k) {
+                  const int* __restrict__ perm, int top, TO* __restrict__ out, int experts, int o, int k, int unary) {
   __shared__ float As[ML_ROWS][ML_K + 1];
   __shared__ float Ws[(GATED ? 2 : 1) * ML_COLS][ML_K + 1];
   __shared__ int src[ML_ROWS];
@@ -438,6 +470,7 @@ moe_linear_kernel(const TA* __restrict__ x, const TW* __restrict__ w, const int*
       if (feat >= o) continue;
       float y = acc[i][j];
       if (GATED) y = y / (1.f + expf(-y)) * up[i][j];
+      else if (unary) y = ifb_unary(y, unary);
       out[(size_t)row * o + feat] = from_f32<TO>(y);
     }
   }
@@ -478,7 +511,7 @@ template <bool GATED> constexpr size_t mm_smem_bytes() {
 template <typename TO, bool GATED>
 __global__ void __launch_bounds__(MM_THREADS)
 moe_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, const int* __restrict__ offsets,
-                      const int* __restrict__ perm, int top, TO* __restrict__ out, int experts, int o, int k) {
+                      const int* __restrict__ perm, int top, TO* __restrict__ out, int experts, int o, int k, int unary) {
   constexpr int WR = (GATED ? 2 : 1) * MM_COLS;              // weight rows of a tile
   extern __shared__ __align__(16) unsigned char mm_raw[];
   __nv_bfloat16* As = reinterpret_cast<__nv_bfloat16*>(mm_raw);                  // [STAGES][MM_ROWS][MM_LD]
@@ -571,6 +604,7 @@ moe_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* 
         if (row >= row1 || feat >= o) continue;
         float y = acc[blk][nt][i];
         if (GATED) y = y / (1.f + expf(-y)) * up[GATED ? blk : 0][GATED ? nt : 0][i];
+        else if (unary) y = ifb_unary(y, unary);
         out[(size_t)row * o + feat] = from_f32<TO>(y);
       }
     }
@@ -590,7 +624,7 @@ template <bool GATED> constexpr size_t sk_smem_bytes() {
 template <typename TO, bool GATED>
 __global__ void __launch_bounds__(SK_THREADS)
 moe_linear_mma_skinny_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, const int* __restrict__ offsets,
-                             const int* __restrict__ perm, int top, TO* __restrict__ out, int experts, int o, int k) {
+                             const int* __restrict__ perm, int top, TO* __restrict__ out, int experts, int o, int k, int unary) {
   constexpr int WR = (GATED ? 2 : 1) * SK_COLS;
   extern __shared__ __align__(16) unsigned char mm_raw[];
   __nv_bfloat16* As = reinterpret_cast<__nv_bfloat16*>(mm_raw);                  // [STAGES][SK_ROWS][SK_LD]
@@ -670,6 +704,7 @@ moe_linear_mma_skinny_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfl
       if (row >= row1 || feat >= o) continue;
       float y = acc[nt][i];
       if (GATED) y = y / (1.f + expf(-y)) * up[nt][i];
+      else if (unary) y = ifb_unary(y, unary);
       out[(size_t)row * o + feat] = from_f32<TO>(y);
     }
   }
@@ -677,66 +712,68 @@ moe_linear_mma_skinny_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfl
 
 template <typename TO>
 static int sk_launch(const void* x, const void* w, const int* offsets, const int* perm, int top, void* out, int rows, int experts,
-                     int o, int k, int gated, cudaStream_t s) {
+                     int o, int k, int gated, int unary, cudaStream_t s) {
   dim3 grid((o + SK_COLS - 1) / SK_COLS, (rows + SK_ROWS - 1) / SK_ROWS + experts);
   if (gated) {
     IFB_ALLOW_SMEM((moe_linear_mma_skinny_kernel<TO, true>), sk_smem_bytes<true>());
     return ifb_launch(moe_linear_mma_skinny_kernel<TO, true>, grid, dim3(SK_THREADS), sk_smem_bytes<true>(), s,
-                      (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k);
+                      (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k, unary);
   }
   IFB_ALLOW_SMEM((moe_linear_mma_skinny_kernel<TO, false>), sk_smem_bytes<false>());
   return ifb_launch(moe_linear_mma_skinny_kernel<TO, false>, grid, dim3(SK_THREADS), sk_smem_bytes<false>(), s,
-                    (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k);
+                    (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k, unary);
 }
 
 template <typename TO>
 static int mm_launch(const void* x, const void* w, const int* offsets, const int* perm, int top, void* out, int rows, int experts,
-                     int o, int k, int gated, cudaStream_t s) {
+                     int o, int k, int gated, int unary, cudaStream_t s) {
   dim3 grid((o + MM_COLS - 1) / MM_COLS, (rows + MM_ROWS - 1) / MM_ROWS + experts);
   if (grid.y > 65535) return IFB_ERR_SIZE;
   if (gated) {
     IFB_ALLOW_SMEM((moe_linear_mma_kernel<TO, true>), mm_smem_bytes<true>());
     return ifb_launch(moe_linear_mma_kernel<TO, true>, grid, dim3(MM_THREADS), mm_smem_bytes<true>(), s, (const __nv_bfloat16*)x,
-                      (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k);
+                      (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k, unary);
   }
   IFB_ALLOW_SMEM((moe_linear_mma_kernel<TO, false>), mm_smem_bytes<false>());
   return ifb_launch(moe_linear_mma_kernel<TO, false>, grid, dim3(MM_THREADS), mm_smem_bytes<false>(), s, (const __nv_bfloat16*)x,
-                    (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k);
+                    (const __nv_bfloat16*)w, offsets, perm, top, (TO*)out, experts, o, k, unary);
 }
 
 template <typename TA, typename TW, typename TO>
 static int ml_launch(const void* x, const void* w, const int* offsets, const int* perm, int top, void* out, int rows, int experts,
-                     int o, int k, int gated, cudaStream_t s) {
+                     int o, int k, int gated, int unary, cudaStream_t s) {
   dim3 grid((o + ML_COLS - 1) / ML_COLS, (rows + ML_ROWS - 1) / ML_ROWS + experts);
   if (grid.y > 65535) return IFB_ERR_SIZE;
   if (gated)
     return ifb_launch(moe_linear_kernel<TA, TW, TO, true>, grid, dim3(ML_THREADS), 0, s, (const TA*)x, (const TW*)w, offsets, perm,
-                      top, (TO*)out, experts, o, k);
+                      top, (TO*)out, experts, o, k, unary);
   return ifb_launch(moe_linear_kernel<TA, TW, TO, false>, grid, dim3(ML_THREADS), 0, s, (const TA*)x, (const TW*)w, offsets, perm,
-                    top, (TO*)out, experts, o, k);
+                    top, (TO*)out, experts, o, k, unary);
 }
 
 // x and w: float32 or bfloat16, in any mix; out: float32 or bfloat16.  rows: the number of rows of `out` (the pairs);
-// o: outputs per row (with gated, w holds 2 o rows per expert).  tensor_cores: bfloat16 x and w with k a multiple of 8
+// o: outputs per row; epilogue: 0 plain, 1 silu_gate (w holds 2 o rows per expert), 16 * u: the unary function u.  tensor_cores: bfloat16 x and w with k a multiple of 8
 // run the mma.sync kernel; everything else, and everything when it is 0, runs the plain kernel.
 IFB_EXPORT int ifb_moe_linear(const void* x, int x_dtype, const void* w, int w_dtype, const int* offsets, const int* perm, int top,
-                              void* out, int out_dtype, int rows, int experts, int o, int k, int gated, int tensor_cores,
+                              void* out, int out_dtype, int rows, int experts, int o, int k, int epilogue, int tensor_cores,
                               cudaStream_t stream) {
   if (rows <= 0 || o <= 0) return IFB_OK;
+  const int gated = epilogue & 15, unary = epilogue >> 4;
+  if (gated > 1 || unary < 0 || unary > IFB_UNARY_LAST || (gated && unary)) return IFB_ERR_ARG;
   if (experts < 1 || k < 1 || top < 1) return IFB_ERR_SIZE;
   if (tensor_cores && x_dtype == IFB_BF16 && w_dtype == IFB_BF16 && k % 8 == 0 && ((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0)) {
     const bool few = rows <= MM_SKINNY_MAX_ROWS;          // a step of few rows: tiles of 16 rows and a deep pipeline
     if (out_dtype == IFB_F32)
-      return few ? sk_launch<float>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, stream)
-                 : mm_launch<float>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, stream);
+      return few ? sk_launch<float>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, unary, stream)
+                 : mm_launch<float>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, unary, stream);
     if (out_dtype == IFB_BF16)
-      return few ? sk_launch<__nv_bfloat16>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, stream)
-                 : mm_launch<__nv_bfloat16>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, stream);
+      return few ? sk_launch<__nv_bfloat16>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, unary, stream)
+                 : mm_launch<__nv_bfloat16>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, unary, stream);
     return IFB_ERR_DTYPE;
   }
 #define ML_CASE(XD, WD, OD, TA, TW, TO)                                                                      \
   if (x_dtype == XD && w_dtype == WD && out_dtype == OD)                                                     \
-    return ml_launch<TA, TW, TO>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, stream);
+    return ml_launch<TA, TW, TO>(x, w, offsets, perm, top, out, rows, experts, o, k, gated, unary, stream);
   ML_CASE(IFB_F32, IFB_F32, IFB_F32, float, float, float)
   ML_CASE(IFB_BF16, IFB_BF16, IFB_F32, __nv_bfloat16, __nv_bfloat16, float)
   ML_CASE(IFB_BF16, IFB_BF16, IFB_BF16, __nv_bfloat16, __nv_bfloat16, __nv_bfloat16)
@@ -776,4 +813,92 @@ IFB_EXPORT int ifb_moe_combine(const float* y, const int* pos, const float* gate
   if (top < 1) return IFB_ERR_SIZE;
   return ifb_launch(moe_combine_kernel, dim3(rows), dim3(256), 0, stream, y, pos, gates, out, top, width, shared, shared_logit,
                     logit_stride);
+}
+
+// ------------------------------------------------------------------------------------------
+// The combination with what follows it in a block that adds mixer and feed-forward at once: x[n] += base[n] + (the sum of
+// moe_combine_kernel), base the mixer's result (null: none), and, with `out`, the next norm of the new row,
+// out[n] = x[n] / sqrt(mean(x[n]^2) + eps) * next_w.  A block per row, the row in shared memory; float32 throughout.
+// ------------------------------------------------------------------------------------------
+template <bool VEC>
+__global__ void __launch_bounds__(256)
+moe_combine_update_kernel(const float* __restrict__ y, const int* __restrict__ pos, const float* __restrict__ gates, int top, int width,
+                          const float* __restrict__ shared, const float* __restrict__ shared_logit, int logit_stride,
+                          const float* __restrict__ base, float* __restrict__ x, const void* __restrict__ next_w, int w_dtype, float eps,
+                          void* __restrict__ out, int out_dtype) {
+  extern __shared__ __align__(16) float mc_row[];
+  __shared__ float scratch[33];
+  __shared__ int mc_pos[32];
+  __shared__ float mc_gate[32];
+  ifb_pdl_wait();
+  ifb_pdl_trigger();
+  const int n = blockIdx.x;
+  if (threadIdx.x < top) {
+    mc_pos[threadIdx.x] = pos[(size_t)n * top + threadIdx.x];
+    mc_gate[threadIdx.x] = gates ? gates[(size_t)n * top + threadIdx.x] : 1.f;
+  }
+  float g = 1.f;
+  if (shared != nullptr && shared_logit != nullptr) g = 1.f / (1.f + expf(-shared_logit[(size_t)n * logit_stride]));
+  __syncthreads();
+  float* xr = x + (size_t)n * width;
+  float ss = 0.f;
+  constexpr int S = VEC ? 4 : 1;
+  for (int f = threadIdx.x * S; f < width; f += blockDim.x * S) {
+    float acc[S] = {}, v[S];
+    for (int j = 0; j < top; ++j) {
+      const float* yr = y + (size_t)mc_pos[j] * width + f;
+      const float w = mc_gate[j];
+      if constexpr (VEC) {
+        const float4 t = *reinterpret_cast<const float4*>(yr);
+        acc[0] = fmaf(w, t.x, acc[0]); acc[1] = fmaf(w, t.y, acc[1]); acc[2] = fmaf(w, t.z, acc[2]); acc[3] = fmaf(w, t.w, acc[3]);
+      } else {
+        acc[0] = fmaf(w, yr[0], acc[0]);
+      }
+    }
+    if constexpr (VEC) {
+      if (shared != nullptr) {
+        const float4 t = *reinterpret_cast<const float4*>(shared + (size_t)n * width + f);
+        acc[0] = fmaf(g, t.x, acc[0]); acc[1] = fmaf(g, t.y, acc[1]); acc[2] = fmaf(g, t.z, acc[2]); acc[3] = fmaf(g, t.w, acc[3]);
+      }
+      float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (base != nullptr) b = *reinterpret_cast<const float4*>(base + (size_t)n * width + f);
+      const float4 o = *reinterpret_cast<const float4*>(xr + f);
+      v[0] = o.x + (b.x + acc[0]); v[1] = o.y + (b.y + acc[1]); v[2] = o.z + (b.z + acc[2]); v[3] = o.w + (b.w + acc[3]);
+      *reinterpret_cast<float4*>(xr + f) = make_float4(v[0], v[1], v[2], v[3]);
+      *reinterpret_cast<float4*>(mc_row + f) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+      if (shared != nullptr) acc[0] = fmaf(g, shared[(size_t)n * width + f], acc[0]);
+      v[0] = xr[f] + ((base != nullptr ? base[(size_t)n * width + f] : 0.f) + acc[0]);
+      xr[f] = v[0];
+      mc_row[f] = v[0];
+    }
+#pragma unroll
+    for (int i = 0; i < S; ++i) ss += v[i] * v[i];
+  }
+  if (out == nullptr) return;
+  const float r = rsqrtf(block_sum(ss, scratch) / (float)width + eps);
+  for (int f = threadIdx.x * S; f < width; f += blockDim.x * S) {      // every thread reads back what it wrote itself
+#pragma unroll
+    for (int i = 0; i < S; ++i)
+      store_from_f32(out, out_dtype, (size_t)n * width + f + i, mc_row[f + i] * r * load_as_f32(next_w, w_dtype, f + i));
+  }
+}
+
+IFB_EXPORT int ifb_moe_combine_update(const float* y, const int* pos, const float* gates, int rows, int top, int width, const float* shared,
+                                      const float* shared_logit, int logit_stride, const float* base, float* x, const void* next_w,
+                                      int w_dtype, float eps, void* out, int out_dtype, cudaStream_t stream) {
+  if (rows <= 0 || width <= 0) return IFB_OK;
+  const size_t smem = (size_t)width * sizeof(float);
+  if (top < 1 || top > 32 || smem > 200 * 1024) return IFB_ERR_SIZE;
+  if ((out == nullptr) != (next_w == nullptr) || x == nullptr) return IFB_ERR_ARG;
+  if (out && ((w_dtype != IFB_F32 && w_dtype != IFB_BF16) || (out_dtype != IFB_F32 && out_dtype != IFB_BF16))) return IFB_ERR_DTYPE;
+  const bool vec = width % 4 == 0 && !(((uintptr_t)y | (uintptr_t)shared | (uintptr_t)base | (uintptr_t)x) & 15);
+  if (vec) {
+    IFB_ALLOW_SMEM(moe_combine_update_kernel<true>, smem);
+    return ifb_launch(moe_combine_update_kernel<true>, dim3(rows), dim3(256), smem, stream, y, pos, gates, top, width, shared, shared_logit,
+                      logit_stride, base, x, next_w, w_dtype, eps, out, out_dtype);
+  }
+  IFB_ALLOW_SMEM(moe_combine_update_kernel<false>, smem);
+  return ifb_launch(moe_combine_update_kernel<false>, dim3(rows), dim3(256), smem, stream, y, pos, gates, top, width, shared, shared_logit,
+                    logit_stride, base, x, next_w, w_dtype, eps, out, out_dtype);
 }

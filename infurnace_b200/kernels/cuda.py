@@ -71,7 +71,7 @@ class CudaKernels:
         self.scratch_generation = 0  # bumped when a scratch buffer moves: captured graphs go stale
         self.core = load_library("core", progress=progress)
         c = self.core
-        c.ifb_embed.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]
+        c.ifb_embed.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p]
         c.ifb_random_normal.argtypes = [c_void_p, c_int, c_longlong, ctypes.c_ulonglong, c_float, c_float, c_void_p]
         c.ifb_rmsnorm.argtypes = [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_float, c_void_p, c_int,
                                   c_void_p, c_int, c_int, c_void_p]
@@ -83,11 +83,11 @@ class CudaKernels:
         c.ifb_argmax_rows.argtypes = [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]
         self._argmax_scratch = None    # (values, indices, counters) of the several-blocks-per-row argmax
         c.ifb_linear_simt.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                      c_void_p]
+                                      c_void_p, c_void_p]
         c.ifb_linear_skinny.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                                         c_int, c_int, c_void_p]
         c.ifb_linear_gemv.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-                                      c_float, c_int, c_void_p]
+                                      c_float, c_int, c_void_p, c_void_p]
         c.ifb_linear_gemv_residual_norm.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                                     c_int, c_int, c_int, c_void_p]
         c.ifb_linear_gemv_qkv.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
@@ -164,7 +164,8 @@ class CudaKernels:
         return _raw_stream(torch._C._cuda_getDevice())
 
     # ------------------------------------------------------------------ embedding
-    def embed(self, table, ids, out):
+    def embed(self, table, ids, out, scale=1.0):
+        """out[n] = scale * table[ids[n]] in float32."""
         _dense(table, "table"), _dense(ids, "ids", torch.int32), _dense(out, "out", torch.float32)
         n, hidden = out.shape
         if table.shape[1] != hidden or ids.numel() != n:
@@ -172,7 +173,7 @@ class CudaKernels:
         self.launches += 1
         self._err_armed = True
         _check(self.core.ifb_embed(table.data_ptr(), _code(table), ids.data_ptr(), out.data_ptr(), n, hidden,
-                                   table.shape[0], self._dev_err.data_ptr(), self._stream()), "embed")
+                                   table.shape[0], self._dev_err.data_ptr(), float(scale), self._stream()), "embed")
 
     def random_normal(self, out, seed64, mean, std):
         """out[i] = mean + std * z_i with z_i approximately N(0, 1), a pure function of (seed64, i): the
@@ -211,10 +212,11 @@ class CudaKernels:
                                      self._stream()), "rmsnorm")
 
     # ------------------------------------------------------------------ matrix products
-    def linear(self, x, w, out, epilogue="none", row_scale=None):
+    def linear(self, x, w, out, epilogue="none", row_scale=None, bias=None):
         """out = x w^T with the epilogue (a key of ``EPILOGUES``).  ``row_scale`` (partials, parts, eps, width), from
         :meth:`linear_residual_norm`, multiplies row n by rsqrt(sum_p partials[p, n] / width + eps)
-        before the epilogue; only where :meth:`can_fold_norm` says so."""
+        before the epilogue; only where :meth:`can_fold_norm` says so.  ``bias`` float32 [out features] is added after that
+        and before a unary function (not with "silu_gate")."""
         _dense(x, "x"), _dense(w, "w"), _dense(out, "out")
         n, k = x.shape
         o = out.shape[1]
@@ -226,6 +228,8 @@ class CudaKernels:
         route = "silu_gate" if gated else "none"          # a unary function changes nothing in the choice of kernel
         if w.shape[1] != k or out.shape[0] != n or w.shape[0] != (2 * o if gated else o):
             raise KernelError(f"linear: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} do not match")
+        if bias is not None and (_dense(bias, "bias", torch.float32).numel() != o or gated):
+            raise KernelError("linear: bias is one float32 number per output feature, and 'silu_gate' takes none")
         if row_scale is not None:
             if not self.can_fold_norm(n, x.dtype, w, route) or out.dtype not in (torch.bfloat16, torch.float32):
                 raise KernelError("linear: a row scale is taken only by the bfloat16 kernels (see can_fold_norm)")
@@ -237,11 +241,11 @@ class CudaKernels:
                 and out.dtype in (torch.bfloat16, torch.float32):
             if self._on_tcgen05(n, w, route):
                 return self._linear_tcgen05(x, w, out, n, o, k, epi, splits=self.tcgen05_splits(n, o, k, gated),
-                                            row_scale=row_scale)
-            return self._linear_gemv(x, w, out, n, o, k, epi, row_scale)
+                                            row_scale=row_scale, bias=bias)
+            return self._linear_gemv(x, w, out, n, o, k, epi, row_scale, bias)
         self.launches += 1
         _check(self.core.ifb_linear_simt(x.data_ptr(), _code(x), w.data_ptr(), _code(w), out.data_ptr(), _code(out),
-                                         n, o, k, epi, self._stream()), "linear")
+                                         n, o, k, epi, _ptr(bias), self._stream()), "linear")
 
     def _on_tcgen05(self, n, w, epilogue="none", shared_k=True):
         key = (n, w.shape[0], w.shape[1], w.dtype, epilogue, shared_k)
@@ -282,7 +286,7 @@ class CudaKernels:
             return 1
         return 9 if w.numel() >= (1 << 23) else 17
 
-    def _linear_tcgen05(self, x, w, out, n, o, k, epi, shape=0, splits=1, row_scale=None, residual=None):
+    def _linear_tcgen05(self, x, w, out, n, o, k, epi, shape=0, splits=1, row_scale=None, residual=None, bias=None):
         """shape: 0 lets the library choose its tile shape; 1 narrow, 2 deep, 3 wide, 4 and 5 persistent.
         splits > 1: the k range of a tile is shared by a cluster of that many CTAs.  row_scale: as in
         :meth:`linear`.  residual (x, norm_weight, partials): as in :meth:`linear_residual_norm`."""
@@ -295,14 +299,15 @@ class CudaKernels:
         _check(self._tc_lib().ifb_linear_tcgen05_ex(
             x.data_ptr(), w.data_ptr(), out.data_ptr(), _code(out), n, o, k, epi, int(shape), int(splits),
             _ptr(partials), int(parts), float(eps), int(width), _ptr(res_x), _ptr(res_g),
-            _code(res_g) if res_g is not None else 0, _ptr(res_partials), self._dev_err.data_ptr(), self._stream()), "linear")
+            _code(res_g) if res_g is not None else 0, _ptr(res_partials), _ptr(bias), self._dev_err.data_ptr(), self._stream()),
+            "linear")
 
     def _tc_lib(self):
         if self._tc is None:
             self._tc = load_library("linear_tcgen05", progress=self._progress)
             self._tc.ifb_linear_tcgen05_ex.argtypes = [
                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float,
-                c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p]
+                c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
             self._tc.ifb_linear_tcgen05_split_clusters.argtypes = [c_int]
             self._tc.ifb_linear_tcgen05_fold_parts.argtypes = [c_int, c_int, c_int]
             self._tc.ifb_linear_tcgen05_qkv.argtypes = [
@@ -348,7 +353,7 @@ class CudaKernels:
                                       "that sampled it had no valid logits; its output is not valid")
                 raise KernelError(f"a kernel gave up waiting on a barrier (code {code}); its output is not valid")
 
-    def _linear_gemv(self, x, w, out, n, o, k, epi, row_scale=None):
+    def _linear_gemv(self, x, w, out, n, o, k, epi, row_scale=None, bias=None):
         self.launches += 1
         partials, parts, eps, width = row_scale if row_scale is not None else (None, 0, 0.0, 0)
         if partials is not None:
@@ -356,7 +361,8 @@ class CudaKernels:
             if partials.dim() != 2 or partials.shape[0] < parts or partials.shape[1] != n:
                 raise KernelError("linear: row_scale partials must be [parts, rows]")
         _check(self.core.ifb_linear_gemv(x.data_ptr(), w.data_ptr(), out.data_ptr(), _code(out), n, o, k, epi,
-                                         _ptr(partials), int(parts), float(eps), int(width), self._stream()), "linear")
+                                         _ptr(partials), int(parts), float(eps), int(width), _ptr(bias), self._stream()),
+               "linear")
 
     # A norm folded into the products around it: RMSNorm(v) = v * g * r with one r per row, so the product that
     # makes v writes v * g and partial sums of v^2, and the product that reads it multiplies by r at its end.
@@ -572,7 +578,7 @@ class CudaKernels:
                 and num_heads % num_kv_heads == 0:
             return self._paged_attention_mma(qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q,
                                              seq_lens, out, scale, window, max_q_len, max_seq_len, n, r,
-                                             min_q_len=min_q_len, weight_terms=weight_terms)
+                                             min_q_len=min_q_len, weight_terms=weight_terms)      # keys and values in one tensor
         self.launches += 1
         _check(self.core.ifb_paged_attention_simt(
             qkv.data_ptr(), _code(qkv), qkv.stride(0), kv_pages.data_ptr(), block_tables.data_ptr(),
@@ -595,17 +601,30 @@ class CudaKernels:
             num_heads, num_kv_heads, head_dim, kv_pages.shape[3], float(scale), int(window), int(max_q_len), self._stream()),
             "paged_attention")
 
-    def attention_library(self, head_dim, weight_terms=1):
+    @staticmethod
+    def attention_defines(head_dim, weight_terms=1, value_head_dim=None, softcap=False):
+        """The compile-time variant of the attention kernels: only what differs from the plain one is named."""
+        defines = {"HEAD_DIM": head_dim}
+        if weight_terms != 1:
+            defines["WEIGHT_TERMS"] = weight_terms
+        if value_head_dim not in (None, head_dim):
+            defines["VALUE_DIM"] = value_head_dim
+        if softcap:
+            defines["SOFTCAP"] = 1
+        return defines
+
+    def attention_library(self, head_dim, weight_terms=1, value_head_dim=None, softcap=False):
         if weight_terms not in (1, 2):
             raise KernelError("attention: a softmax weight has one or two bfloat16 terms")
-        key = head_dim if weight_terms == 1 else (head_dim, weight_terms)
+        defines = self.attention_defines(head_dim, weight_terms, value_head_dim, softcap)
+        key = tuple(sorted(defines.items()))
         lib = self._attn_mma.get(key)
         if lib is None:
-            defines = {"HEAD_DIM": head_dim} if weight_terms == 1 else {"HEAD_DIM": head_dim, "WEIGHT_TERMS": weight_terms}
             lib = load_library("attention_mma", defines, progress=self._progress)
-            lib.ifb_attention_mma.argtypes = [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
-                                              c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                              c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
+            lib.ifb_attention_mma.argtypes = [
+                c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int,
+                c_float, c_int, c_int, c_int, c_int, c_int, c_void_p]
             lib.ifb_attention_mma_scratch_floats.restype = c_longlong
             lib.ifb_attention_mma_scratch_floats.argtypes = [c_int, c_int, c_int]
             self._attn_mma[key] = lib
@@ -628,8 +647,31 @@ class CudaKernels:
 
     def _paged_attention_mma(self, qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q, seq_lens, out,
                              scale, window, max_q_len, max_seq_len, n, r, num_splits=None, min_q_len=1, weight_terms=1):
-        lib = self.attention_library(head_dim, weight_terms)
+        """Keys and values of one width in one tensor [pages, 2, kv_heads, page_size, head_dim]: two streams of a common stride."""
+        esize, ps = kv_pages.element_size(), kv_pages.shape[3]
+        k = (kv_pages.data_ptr(), kv_pages.stride(0), ps)
+        v = (kv_pages.data_ptr() + esize * num_kv_heads * ps * head_dim, kv_pages.stride(0), ps)
+        self._attention_mma_streams(qkv, num_heads, num_kv_heads, head_dim, head_dim, k, v, kv_pages.shape[0], block_tables, cu_q, seq_lens,
+                                    out, scale, window, max_q_len, max_seq_len, n, r, num_splits, min_q_len, weight_terms,
+                                    one_tensor=kv_pages)
+
+    ATTENTION_GROUP = 16      # query heads that share a key/value head's rows in one CTA of the small-q kernel
+
+    @classmethod
+    def attention_share(cls, group):
+        """Into how many groups the ``group`` query heads of a key/value head are split so that each has at most 16."""
+        return next(s for s in range(1, group + 1) if group % s == 0 and group // s <= cls.ATTENTION_GROUP)
+
+    def _attention_mma_streams(self, qkv, num_heads, num_kv_heads, head_dim, value_head_dim, k, v, num_pages, block_tables, cu_q,
+                               seq_lens, out, scale, window, max_q_len, max_seq_len, n, r, num_splits=None, min_q_len=1,
+                               weight_terms=1, softcap=None, sink=None, one_tensor=None):
+        """The tensor-core attention kernels over key and value streams ``k`` and ``v`` = (address, elements between pages, page
+        size).  ``one_tensor``: the tensor that holds both, where there is one (what the tcgen05 kernel for plain attention takes)."""
+        share = self.attention_share(num_heads // num_kv_heads)
+        real_kv, num_kv_heads = num_kv_heads, num_kv_heads * share           # groups of query heads from here on
+        lib = self.attention_library(head_dim, weight_terms, value_head_dim, bool(softcap))
         group = num_heads // num_kv_heads
+        page_size = k[2]
         only_small = max_q_len * group <= 16
         if num_splits is None:
             num_splits = self.attention_splits(r, num_kv_heads, max_seq_len, window)
@@ -643,26 +685,26 @@ class CudaKernels:
                 self._attn_counters = torch.zeros(max(r * num_kv_heads, 4096), dtype=torch.int32, device="cuda")
                 self.scratch_generation += 1
             counters = self._attn_counters
-        use_tc = (not only_small and self.attention_tc and weight_terms == 1 and head_dim == 128 and 128 % group == 0
-                  and kv_pages.shape[3] in (16, 32, 64) and kv_pages.data_ptr() % 128 == 0)
+        use_tc = (not only_small and self.attention_tc and one_tensor is not None and share == 1 and weight_terms == 1 and not softcap
+                  and sink is None and head_dim == 128 and 128 % group == 0 and page_size in (16, 32, 64)
+                  and one_tensor.data_ptr() % 128 == 0)
         if use_tc:
-            self._attention_tc(qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q, seq_lens, out, scale,
+            self._attention_tc(qkv, num_heads, num_kv_heads, head_dim, one_tensor, block_tables, cu_q, seq_lens, out, scale,
                                window, max_q_len, n, r)
             if min_q_len * group > 16:
                 return                 # no request of this step is left for the small-q kernel
             only_small = True          # the tile kernel's requests are done; the small-q kernel takes the rest
         self.launches += 1 + (0 if only_small else 1)
         self.small_q_calls += 1
-        if self.attention_tma and head_dim % 64 == 0 and kv_pages.shape[3] in (16, 32, 64) \
-                and kv_pages.data_ptr() % 128 == 0 and kv_pages.numel() // head_dim < 0x7fffffff:
+        if self.attention_tma and head_dim % 64 == 0 and value_head_dim % 64 == 0 and page_size in (16, 32, 64):
             self.small_q_tma_calls += 1        # the library's own condition for its TMA path
         self._err_armed = True
         _check(lib.ifb_attention_mma(
-            qkv.data_ptr(), qkv.stride(0), kv_pages.data_ptr(), kv_pages.shape[0], block_tables.data_ptr(),
-            block_tables.stride(0), cu_q.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), _ptr(scratch), _ptr(counters),
-            self._dev_err.data_ptr(), n, r, num_heads, num_kv_heads, head_dim, kv_pages.shape[3], float(scale), int(window),
-            int(max_q_len), int(num_splits), 1, 0 if only_small else 1, 1 if self.attention_tma else 0, self._stream()),
-            "paged_attention")
+            qkv.data_ptr(), qkv.stride(0), k[0], k[1], v[0], v[1], num_pages, block_tables.data_ptr(), block_tables.stride(0),
+            cu_q.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), _ptr(scratch), _ptr(counters), self._dev_err.data_ptr(), n, r, num_heads,
+            num_kv_heads, share, head_dim, value_head_dim, page_size, float(scale), int(window), float(softcap or 0.0),
+            0 if sink is None else 1, float(sink or 0.0), int(max_q_len), int(num_splits), 1, 0 if only_small else 1,
+            1 if self.attention_tma else 0, self._stream()), "paged_attention")
 
     # ------------------------------------------------------------------ post-norm sublayers, recurrence, talking attention
     def _mix_lib(self):
@@ -890,14 +932,17 @@ class CudaKernels:
             m.ifb_rotate_rows.argtypes = [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
             m.ifb_paged_attention_streams.argtypes = [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int,
                                                       c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                                      c_int, c_float, c_int, c_void_p, c_int, c_void_p]
-            m.ifb_moe_route.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p]
+                                                      c_int, c_float, c_int, c_void_p, c_int, c_float, c_float, c_void_p]
+            m.ifb_moe_route.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
+                                        c_int, c_int, c_void_p]
             m.ifb_moe_plan.argtypes = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
             m.ifb_moe_linear.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                                          c_int, c_int, c_int, c_int, c_int, c_void_p]
             m.ifb_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
             m.ifb_moe_route_plan_small.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                                                   c_int, c_int, c_int, c_int, c_float, c_void_p]
+                                                   c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p]
+            m.ifb_moe_combine_update.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
+                                                 c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p]
             m.ifb_moe_plan_padded.argtypes = [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
             m.ifb_moe_gather_rows.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p]
             m.ifb_rglru_conv.argtypes = [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -1183,10 +1228,16 @@ class CudaKernels:
                                                int(bool(interleaved)), 1 if back else 0, self._stream()), "rotate_rows")
 
     def paged_attention_streams(self, q, num_heads, num_kv_heads, head_dim, value_head_dim, k_pages, v_pages, block_tables, cu_q,
-                                seq_lens, out, scale, window, out_table, out_interleaved, max_q_len=0, max_seq_len=0):
+                                seq_lens, out, scale, window, out_table, out_interleaved, max_q_len=0, max_seq_len=0, min_q_len=1,
+                                softcap=None, sink=None, weight_terms=1, exact=True):
         """Causal softmax attention of q [n, H d] over key and value page streams (csrc/attention_streams.cu), float32
         scores, weights and sums; each head's output is rotated back by the query token's angles of ``out_table``
-        ([n, dv] (cos, sin) pairs; None: not)."""
+        ([n, dv] (cos, sin) pairs; None: not).  ``softcap`` c: a scaled score s becomes c tanh(s / c).  ``sink`` z: exp(z) joins the
+        denominator.
+
+        ``exact`` False: bfloat16 streams whose widths are multiples of 16 (at most 256), without ``out_table``, run the
+        tensor-core kernels (csrc/attention_mma.cu): float32 scores, softmax and sums, a softmax weight entering the weighted
+        sum as ``weight_terms`` bfloat16 numbers."""
         _dense(q, "q"), _dense(out, "out", q.dtype), _dense(cu_q, "cu_q", torch.int32), _dense(seq_lens, "seq_lens", torch.int32)
         if block_tables.dtype != torch.int32 or block_tables.stride(1) != 1:
             raise KernelError("paged_attention_streams: block_tables must be int32 with unit stride along pages")
@@ -1199,50 +1250,71 @@ class CudaKernels:
             raise KernelError("paged_attention_streams: the streams differ in page size")
         if out_table is not None and _dense(out_table, "out_table", torch.float32).shape != (n, dv):
             raise KernelError("paged_attention_streams: out_table is [tokens, value_head_dim]")
+        if H % G:
+            raise KernelError("paged_attention_streams: the query heads are a multiple of the key/value heads")
+        if not exact and q.dtype == torch.bfloat16 and out_table is None and d % 16 == 0 and dv % 16 == 0 and d <= 256 and dv <= 256 \
+                and max_q_len and max_seq_len:
+            return self._attention_mma_streams(q, H, G, d, dv, pk, pv, k_pages.shape[0], block_tables, cu_q, seq_lens, out, scale, window,
+                                               max_q_len, max_seq_len, n, r, None, min_q_len, weight_terms, softcap, sink)
         self.launches += 1
         self.stream_attention_calls += 1
         _check(self._hyb_lib().ifb_paged_attention_streams(
             q.data_ptr(), _code(q), pk[0], pk[1], pv[0], pv[1], block_tables.data_ptr(), block_tables.stride(0), cu_q.data_ptr(),
             seq_lens.data_ptr(), out.data_ptr(), n, r, H, G, d, dv, pk[2], float(scale), int(window), _ptr(out_table),
-            int(bool(out_interleaved)), self._stream()), "paged_attention_streams")
+            int(bool(out_interleaved)), float(softcap or 0.0), float("-inf") if sink is None else float(sink), self._stream()),
+            "paged_attention_streams")
 
     @staticmethod
-    def _route_mode(logits, experts, scoring, groups, weight_scale):
-        """(experts, stride, mode, group count, groups kept, weight scale) of a router call: ``experts`` None means every
+    def _route_mode(logits, experts, scoring, groups, weight_scale, correction=None, normalise=False, group_best=1):
+        """(experts, the router kernels' arguments from ``stride`` on) of a router call: ``experts`` None means every
         column of ``logits`` is an expert's."""
         if scoring not in ("chosen", "all", "sigmoid"):
             raise KernelError(f"moe_route: scoring {scoring!r}; known: chosen, all, sigmoid")
+        experts = int(experts) if experts is not None else logits.shape[1]
         count, keep = groups if groups else (1, 1)
-        if groups and scoring != "all":
-            raise KernelError("moe_route: groups of experts limit the choice only with scoring 'all'")
-        return (int(experts) if experts is not None else logits.shape[1], logits.shape[1], {"chosen": 0, "all": 1, "sigmoid": 2}[scoring],
-                int(count), int(keep), float(weight_scale))
+        mode = {"chosen": 0, "all": 1, "sigmoid": 2}[scoring]
+        if scoring == "sigmoid" and (correction is not None or normalise or groups):
+            mode = 3                          # the order of the scores is no longer that of the logits
+        if groups and mode not in (1, 3):
+            raise KernelError("moe_route: groups of experts limit the choice only with scoring 'all' or 'sigmoid'")
+        if (correction is not None or normalise) and mode != 3:
+            raise KernelError("moe_route: a correction and normalised weights belong to scoring 'sigmoid'")
+        if group_best not in (1, 2):
+            raise KernelError("moe_route: a group counts by its best score or by the sum of its two best")
+        if correction is not None and _dense(correction, "correction", torch.float32).numel() != experts:
+            raise KernelError("moe_route: correction is one float32 number per expert")
+        return experts, (logits.shape[1], mode, int(count), int(keep), float(weight_scale), _ptr(correction), int(group_best),
+                         1 if normalise else 0)
 
-    def moe_route(self, logits, top, ids, gates, experts=None, scoring="chosen", groups=None, weight_scale=1.0):
+    def moe_route(self, logits, top, ids, gates, experts=None, scoring="chosen", groups=None, weight_scale=1.0, correction=None,
+                  normalise=False, group_best=1):
         """ids[n] = the indices of row n's ``top`` largest scores, largest first (the lower index among equals).  scoring
         "chosen": the scores are the logits and gates[n] = the softmax over the chosen logits.  scoring "all": the scores are
         the softmax over all experts, gates[n] = score * weight_scale, and with ``groups`` = (count, keep) only experts of the
         ``keep`` groups of neighbours with the largest best score can be chosen.  scoring "sigmoid": the scores are sigmoid(logit)
-        per expert and gates[n] = score * weight_scale.  ``experts``: the first that many columns of
+        per expert and gates[n] = score * weight_scale; then ``correction`` float32 [experts] is added to the scores for the
+        choice of groups and experts only, and ``normalise`` divides the chosen scores by their sum + 1e-20.  A group's score is
+        the sum of its ``group_best`` (1 or 2) largest.  ``experts``: the first that many columns of
         ``logits`` are the router's (the rest belong to someone else).  (csrc/moe.cu)"""
         _dense(logits, "logits", torch.float32), _dense(ids, "ids", torch.int32), _dense(gates, "gates", torch.float32)
         n = logits.shape[0]
-        experts, stride, mode, count, keep, ws = self._route_mode(logits, experts, scoring, groups, weight_scale)
+        experts, mode = self._route_mode(logits, experts, scoring, groups, weight_scale, correction, normalise, group_best)
         if ids.shape != (n, top) or gates.shape != (n, top):
             raise KernelError("moe_route: ids and gates are [rows, top]")
         self.launches += 1
-        _check(self._hyb_lib().ifb_moe_route(logits.data_ptr(), ids.data_ptr(), gates.data_ptr(), n, experts, int(top), stride, mode,
-                                             count, keep, ws, self._stream()), "moe_route")
+        _check(self._hyb_lib().ifb_moe_route(logits.data_ptr(), ids.data_ptr(), gates.data_ptr(), n, experts, int(top), *mode,
+                                             self._stream()), "moe_route")
 
     MOE_SMALL_PAIRS = 512      # up to here the router and the pair list are one launch of one block
 
     def moe_route_plan(self, logits, top, ids, gates, offsets, perm, pos, experts=None, scoring="chosen", groups=None,
-                       weight_scale=1.0):
+                       weight_scale=1.0, correction=None, normalise=False, group_best=1):
         """:meth:`moe_route` and :meth:`moe_plan` of a step; one launch where the step has few pairs (decode)."""
         n = logits.shape[0]
-        experts, stride, mode, count, keep, ws = self._route_mode(logits, experts, scoring, groups, weight_scale)
+        experts, mode = self._route_mode(logits, experts, scoring, groups, weight_scale, correction, normalise, group_best)
         if n * top > self.MOE_SMALL_PAIRS or experts > 256:
-            self.moe_route(logits, top, ids, gates, experts=experts, scoring=scoring, groups=groups, weight_scale=weight_scale)
+            self.moe_route(logits, top, ids, gates, experts=experts, scoring=scoring, groups=groups, weight_scale=weight_scale,
+                           correction=correction, normalise=normalise, group_best=group_best)
             return self.moe_plan(ids, experts, offsets, perm, pos)
         _dense(logits, "logits", torch.float32), _dense(ids, "ids", torch.int32), _dense(gates, "gates", torch.float32)
         _dense(offsets, "offsets", torch.int32), _dense(perm, "perm", torch.int32), _dense(pos, "pos", torch.int32)
@@ -1251,8 +1323,7 @@ class CudaKernels:
             raise KernelError("moe_route_plan: sizes of ids, gates, offsets, perm and pos do not match")
         self.launches += 1
         _check(self._hyb_lib().ifb_moe_route_plan_small(logits.data_ptr(), ids.data_ptr(), gates.data_ptr(), n, experts, int(top),
-                                                        offsets.data_ptr(), perm.data_ptr(), pos.data_ptr(), stride, mode, count,
-                                                        keep, ws, self._stream()),
+                                                        offsets.data_ptr(), perm.data_ptr(), pos.data_ptr(), *mode, self._stream()),
                "moe_route_plan")
 
     def moe_plan(self, ids, num_experts, offsets, perm, pos):
@@ -1269,12 +1340,13 @@ class CudaKernels:
 
     def moe_linear(self, x, w, offsets, perm, top, out, epilogue="none"):
         """Row i of ``out`` belongs to the expert e with offsets[e] <= i < offsets[e + 1] and is x[perm[i] // top] @ w[e]^T
-        (perm None: x[i]); w [experts, o, k]; epilogue "silu_gate": w[e] holds gate rows, then up rows.  bfloat16 x and w
+        (perm None: x[i]); w [experts, o, k]; epilogue "silu_gate": w[e] holds gate rows, then up rows; else a unary function of
+        ``EPILOGUES``.  bfloat16 x and w
         with k a multiple of 8 run on tensor cores (mma.sync), everything else in plain float32 arithmetic."""
         _dense(x, "x"), _dense(w, "w"), _dense(offsets, "offsets", torch.int32), _dense(out, "out")
         gated = epilogue == "silu_gate"
-        if epilogue not in ("none", "silu_gate"):
-            raise KernelError(f"moe_linear: epilogue {epilogue!r}; known: none, silu_gate")
+        if epilogue not in EPILOGUES:
+            raise KernelError(f"moe_linear: unknown epilogue {epilogue!r}; known: {', '.join(EPILOGUES)}")
         rows, o = out.shape
         experts, ow, k = w.shape
         if x.shape[1] != k or ow != (2 * o if gated else o) or offsets.numel() != experts + 1:
@@ -1286,7 +1358,7 @@ class CudaKernels:
             raise KernelError("moe_linear: without perm, x has a row for each row of out")
         self.launches += 1
         _check(self._hyb_lib().ifb_moe_linear(x.data_ptr(), _code(x), w.data_ptr(), _code(w), offsets.data_ptr(), _ptr(perm),
-                                              int(top), out.data_ptr(), _code(out), rows, experts, o, k, 1 if gated else 0,
+                                              int(top), out.data_ptr(), _code(out), rows, experts, o, k, EPILOGUES[epilogue],
                                               1 if self.moe_tensor_cores else 0, self._stream()), "moe_linear")
 
     # The experts' products of a prompt on the tcgen05 kernel: every expert's rows contiguous in segments padded to the
@@ -1347,8 +1419,8 @@ class CudaKernels:
         mode); x [places, k] sorted by expert in padded segments, w [experts, o (2 o with "silu_gate"), k]."""
         _dense(x, "x", torch.bfloat16), _dense(w, "w", torch.bfloat16), _dense(tile_expert, "tile_expert", torch.int32), _dense(out, "out")
         gated = epilogue == "silu_gate"
-        if epilogue not in ("none", "silu_gate"):
-            raise KernelError(f"moe_linear_grouped: epilogue {epilogue!r}; known: none, silu_gate")
+        if epilogue not in EPILOGUES:
+            raise KernelError(f"moe_linear_grouped: unknown epilogue {epilogue!r}; known: {', '.join(EPILOGUES)}")
         rows, o = out.shape
         experts, ow, k = w.shape
         if x.shape != (rows, k) or ow != (2 * o if gated else o) or rows != tile_expert.numel() * self.MOE_TILE:
@@ -1362,7 +1434,7 @@ class CudaKernels:
         self.moe_tcgen05_calls += 1
         self._err_armed = True
         _check(lib.ifb_linear_tcgen05_grouped(x.data_ptr(), w.data_ptr(), out.data_ptr(), _code(out), rows, experts, o, k,
-                                              1 if gated else 0, tile_expert.data_ptr(), self._dev_err.data_ptr(), self._stream()),
+                                              EPILOGUES[epilogue], tile_expert.data_ptr(), self._dev_err.data_ptr(), self._stream()),
                "moe_linear_grouped")
 
     def moe_combine(self, y, pos, gates, out, shared=None, shared_logit=None):
@@ -1371,13 +1443,23 @@ class CudaKernels:
         column of a float32 matrix) is given."""
         _dense(y, "y", torch.float32), _dense(pos, "pos", torch.int32), _dense(out, "out", torch.float32)
         n = out.shape[0]
+        top, stride = self._combine_sizes(y, pos, gates, out, shared, shared_logit)
+        self.launches += 1
+        _check(self._hyb_lib().ifb_moe_combine(y.data_ptr(), pos.data_ptr(), _ptr(gates), out.data_ptr(), n, top,
+                                               out.shape[1], _ptr(shared), _ptr(shared_logit) if shared is not None else None,
+                                               stride, self._stream()), "moe_combine")
+
+    @staticmethod
+    def _combine_sizes(y, pos, gates, out, shared, shared_logit):
+        """(top, stride of the shared logit) of a combination of experts' results into rows of ``out``'s shape."""
+        n = out.shape[0]
         if gates is None:                      # every weight is 1 (the weights went into what the experts read)
             top = pos.numel() // max(n, 1)
         else:
             top = _dense(gates, "gates", torch.float32).shape[1]
             if gates.shape[0] != n:
                 raise KernelError("moe_combine: gates has a row for every row of out")
-        if pos.numel() != n * top or y.shape[0] < n * top or y.shape[1] != out.shape[1] or out.shape[0] != n:
+        if pos.numel() != n * top or y.shape[0] < n * top or y.shape[1] != out.shape[1]:
             raise KernelError("moe_combine: sizes of y, pos, gates and out do not match")
         stride = 0
         if shared is not None:
@@ -1387,10 +1469,24 @@ class CudaKernels:
                 if shared_logit.dtype != torch.float32 or shared_logit.dim() != 1 or shared_logit.shape[0] != n:
                     raise KernelError("moe_combine: shared_logit is one float32 number per row")
                 stride = shared_logit.stride(0)
+        return top, stride
+
+    def moe_combine_update(self, y, pos, gates, x, base=None, shared=None, shared_logit=None, out=None, next_weight=None, eps=0.0):
+        """x[n] += base[n] + (what :meth:`moe_combine` writes), x the float32 stream and ``base`` (float32, x's shape, or None) the
+        mixer's result; with ``out``, also out[n] = x[n] / sqrt(mean(x[n]^2) + eps) * next_weight of the new row."""
+        _dense(y, "y", torch.float32), _dense(pos, "pos", torch.int32), _dense(x, "x", torch.float32)
+        top, stride = self._combine_sizes(y, pos, gates, x, shared, shared_logit)
+        if base is not None and _dense(base, "base", torch.float32).shape != x.shape:
+            raise KernelError("moe_combine_update: base has the shape of x")
+        if (out is None) != (next_weight is None) or (out is not None and (_dense(out, "out").shape != x.shape
+                                                                            or _dense(next_weight, "next_weight").numel() != x.shape[1])):
+            raise KernelError("moe_combine_update: out and next_weight come together and have x's shape and row length")
         self.launches += 1
-        _check(self._hyb_lib().ifb_moe_combine(y.data_ptr(), pos.data_ptr(), _ptr(gates), out.data_ptr(), n, top,
-                                               out.shape[1], _ptr(shared), _ptr(shared_logit) if shared is not None else None,
-                                               stride, self._stream()), "moe_combine")
+        _check(self._hyb_lib().ifb_moe_combine_update(
+            y.data_ptr(), pos.data_ptr(), _ptr(gates), x.shape[0], top, x.shape[1], _ptr(shared),
+            _ptr(shared_logit) if shared is not None else None, stride, _ptr(base), x.data_ptr(), _ptr(next_weight),
+            _code(next_weight) if next_weight is not None else 0, float(eps), _ptr(out), _code(out) if out is not None else 0,
+            self._stream()), "moe_combine_update")
 
     # ------------------------------------------------------------------ decoders with latent attention (csrc/latent.cu)
     def _lat_lib(self):

@@ -9,3 +9,4 @@ from . import kafunex  # noqa: F401  (registers "Kafunex")
 from . import lunelorn  # noqa: F401  (registers "Lunelorn")
 from . import filorax  # noqa: F401  (registers "Filorax")
 from . import golonex  # noqa: F401  (registers "Golonex")
+from . import mubutar  # noqa: F401  (registers "Mubutar")

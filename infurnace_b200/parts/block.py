@@ -4,10 +4,15 @@ from __future__ import annotations
 import torch
 
 from ..config.specs import (
-    DepthAverageBlockSpec, LayerCall, PostNormBlockSpec, PreNormBlockSpec, SandwichBlockSpec, StreamInjectSpec, TokenSideSpec,
+    DepthAverageBlockSpec, LayerCall, ParallelBlockSpec, PostNormBlockSpec, PreNormBlockSpec, SandwichBlockSpec, StreamInjectSpec, TokenSideSpec,
 )
 from .parallel import WeightedSum
 from .registry import Folded, build_part, register_part
+
+
+def add_pending(x, pending):
+    """x += a delta that a block of another kind handed on: one tensor, or several stacked along a leading axis."""
+    x.add_(pending if pending.dim() == x.dim() else pending.sum(dim=0))
 
 
 class PreNormBlock:
@@ -147,7 +152,7 @@ class PostNormBlock:
         if pending is not None:                      # a block of another kind ran before and left its last delta
             if isinstance(pending, Folded):
                 raise TypeError("a post-norm block cannot take a folded norm from the block before it")
-            x.add_(pending)
+            add_pending(x, pending)
             ctx.shared.pop(STREAM_COPY, None)
         self._update(x, self.mixer.forward(self._input(x, ctx), ctx, call), self.mixer_norm, self.mixer_scale, ctx)
         if self.ffn is not None:
@@ -243,7 +248,7 @@ class SandwichBlock:
             if pending is not None:                  # a block of another kind ran before and left its last delta
                 if isinstance(pending, Folded):
                     raise TypeError("a sandwich block cannot take a folded norm from the block before it")
-                x.add_(pending)
+                add_pending(x, pending)
             h = ctx.buffer("h", x.shape, self.rt.act_dtype)
             self.mixer_norm.forward(x, h)
         ahead = next_layer.mixer_norm if isinstance(next_layer, SandwichBlock) else None
@@ -350,6 +355,78 @@ class DepthAverageBlock:
 register_part(DepthAverageBlockSpec, DepthAverageBlock)
 
 
+class ParallelBlock:
+    """h = norm(x); x += mixer(h) + ffn(h).
+
+    Both results belong to one addition, and it happens once, in one of three places:
+
+    * the feed-forward's last kernel, where that combines experts: it adds mixer and mixture to x and writes the next block's
+      norm in the same pass (the next block gets a :class:`ReadyInput`);
+    * the products themselves, where both parts and the next block can fold a norm (few rows, bfloat16): the mixer's output
+      product adds to x, the feed-forward's then adds to x and leaves the next norm half done (a :class:`Folded`);
+    * else the two results lie side by side in one buffer [2, tokens, hidden], which is the pending delta: the kernel of
+      the norm that follows adds both."""
+
+    folds_norms = True
+
+    def __init__(self, spec: ParallelBlockSpec, weights, runtime):
+        self.spec = spec
+        self.rt = runtime
+        self.k = runtime.kernels
+        self.mixer_norm = build_part(spec.norm, weights, runtime)
+        self.mixer = build_part(spec.mixer, weights, runtime)
+        self.ffn = build_part(spec.ffn, weights, runtime) if spec.ffn is not None else None
+
+    @property
+    def graph_safe(self):
+        return all(getattr(p, "graph_safe", False) for p in (self.mixer_norm, self.mixer, self.ffn) if p is not None)
+
+    def takes_folded(self, n):
+        """Whether the block before this one may hand over x already updated and this block's norm folded: both sublayers
+        read it."""
+        parts = [self.mixer] + ([self.ffn] if self.ffn is not None else [])
+        return bool(getattr(self.mixer_norm, "foldable", False)) and all(
+            getattr(p, "can_take_folded", None) and p.can_take_folded(n) for p in parts)
+
+    def forward(self, x, pending, ctx, call, next_layer=None):
+        n, width = x.shape
+        if isinstance(pending, ReadyInput):          # x is up to date and our norm is written
+            h = pending.values
+        elif isinstance(pending, Folded):            # x is up to date and our norm is folded
+            h = pending
+        else:
+            h = ctx.buffer("h", x.shape, self.rt.act_dtype)
+            self.mixer_norm.forward(x, h, delta=pending)
+        last = self.ffn if self.ffn is not None else self.mixer
+        if next_layer is not None and all(getattr(p, "can_fold_output", False) for p in (self.mixer, last)) and next_layer.takes_folded(n):
+            norm = next_layer.mixer_norm
+            d = self.mixer.forward(h, ctx, call, fold=(x, norm))
+            if isinstance(d, Folded):                # x holds the mixer's result; the half norm of that sum is not used
+                if self.ffn is None:
+                    return d
+                return self.ffn.forward(h, ctx, fold=(x, norm))      # a Folded, or the feed-forward's plain delta
+            if self.ffn is None:
+                return d
+            self.k.scaled_sum(d, self.ffn.forward(h, ctx), 1.0)
+            return d
+        if self.ffn is None:
+            return self.mixer.forward(h, ctx, call)
+        if getattr(self.ffn, "can_update_stream", False):
+            d = self.mixer.forward(h, ctx, call)
+            norm = next_layer.mixer_norm if next_layer is not None and hasattr(getattr(next_layer, "mixer_norm", None), "weight") \
+                and getattr(next_layer.mixer_norm, "foldable", False) else None
+            out = ctx.buffer("h", x.shape, self.rt.act_dtype) if norm is not None else None      # (h itself has been read by then)
+            self.ffn.forward(h, ctx, update=(x, d, norm, out))
+            return ReadyInput(out) if norm is not None else None
+        pair = ctx.buffer("delta_pair", (2 * n, width), torch.float32, rows=2 * ctx.max_rows).view(2, n, width)
+        self.mixer.forward(h, ctx, call, out=pair[0])
+        self.ffn.forward(h, ctx, out=pair[1])
+        return pair
+
+
+register_part(ParallelBlockSpec, ParallelBlock)
+
+
 class StreamInject:
     """x += table[row] (+ the rows the embedding kept): the step that opens a pass over a range of layers that runs
     several times.  It stands in the schedule like a layer."""
@@ -367,7 +444,7 @@ class StreamInject:
         if pending is not None:
             if isinstance(pending, Folded):
                 raise TypeError("an injection step cannot take a folded norm from the block before it")
-            x.add_(pending)
+            add_pending(x, pending)
         rows = None
         if self.spec.add_embedding:
             rows = ctx.shared.get(self._key)

@@ -30,7 +30,8 @@ class GatedMLP:
         can = getattr(self.k, "can_fold_norm", None)
         return bool(can and can(n, self.rt.act_dtype, self.w_gate_up, "silu_gate"))
 
-    def forward(self, h, ctx, fold=None):
+    def forward(self, h, ctx, fold=None, out=None):
+        """``out``: where the result goes if it is not folded into the stream (default: a buffer of the part's)."""
         h, row_scale = unfolded(h)
         n = h.shape[0]
         act = ctx.buffer("ffn_act", (n, self.spec.intermediate_size), self.rt.act_dtype)
@@ -41,7 +42,7 @@ class GatedMLP:
         folded = fold_residual_norm(self.k, ctx, "ffn", act, self.w_down, fold, self.rt.act_dtype)
         if folded is not None:
             return folded
-        delta = ctx.buffer("delta_ffn", (n, self.spec.hidden_size), torch.float32)
+        delta = out if out is not None else ctx.buffer("delta_ffn", (n, self.spec.hidden_size), torch.float32)
         self.k.linear(act, self.w_down, delta)
         return delta
 
@@ -64,11 +65,11 @@ class DenseMLP:
         self.w_up = weights[spec.up_proj]
         self.w_down = weights[spec.down_proj]
 
-    def forward(self, h, ctx, fold=None):
+    def forward(self, h, ctx, fold=None, out=None):
         n = h.shape[0]
         act = ctx.buffer("ffn_act", (n, self.spec.intermediate_size), self.rt.act_dtype)
         self.k.linear(h, self.w_up, act, epilogue=self.spec.activation)
-        delta = ctx.buffer("delta_ffn", (n, self.spec.hidden_size), torch.float32)
+        delta = out if out is not None else ctx.buffer("delta_ffn", (n, self.spec.hidden_size), torch.float32)
         self.k.linear(act, self.w_down, delta)
         return delta
 

@@ -8,8 +8,8 @@ from .registry import build_part, register_part
 
 
 class Embedding:
-    """x[t] = table[id_t], widened to float32, no scaling
-    (src/infurnace/executor/tinygrad/model.py:95)."""
+    """x[t] = scale * table[id_t], widened to float32 (the reference scales by nothing,
+    src/infurnace/executor/tinygrad/model.py:95)."""
 
     def __init__(self, spec: EmbeddingSpec, weights, runtime):
         self.spec = spec
@@ -17,21 +17,28 @@ class Embedding:
         self.k = runtime.kernels
 
     def forward(self, ids, out):
-        self.k.embed(self.table, ids, out)
+        if self.spec.scale != 1.0:
+            self.k.embed(self.table, ids, out, scale=self.spec.scale)
+        else:
+            self.k.embed(self.table, ids, out)
         return out
 
 
 class LMHead:
-    """logits = h @ W^T in float32 (model.py:151); W is the embedding table when tied
-    (src/infurnace/executor/tinygrad/weights.py:68), read in place."""
+    """logits = scale * h @ W^T in float32 (model.py:151, where there is no scale); W is the embedding table when tied
+    (src/infurnace/executor/tinygrad/weights.py:68), read in place.  The decoder puts the scale into the final norm's weight
+    where that norm offers it (``gain`` is then 1): scaling a row before its product or after is the same."""
 
     def __init__(self, spec: LMHeadSpec, weights, runtime):
         self.spec = spec
         self.weight = weights[spec.weight]
         self.k = runtime.kernels
+        self.gain = float(spec.scale)
 
     def forward(self, h, out):
         self.k.linear(h, self.weight, out)
+        if self.gain != 1.0:
+            self.k.scaled_sum(out, out, self.gain, accumulate=False)
         if self.spec.softcap:                  # c * tanh(logits / c), in place
             self.k.softcap(out, float(self.spec.softcap))
         return out
@@ -113,6 +120,9 @@ class DecoderModel:
         self.schedule = plan.resolved_schedule()
         self.final_norm = build_part(plan.final_norm, weights, runtime)
         self.lm_head = build_part(plan.lm_head, weights, runtime)
+        if getattr(self.lm_head, "gain", 1.0) != 1.0 and hasattr(self.final_norm, "scale_output"):
+            self.final_norm.scale_output(self.lm_head.gain)
+            self.lm_head.gain = 1.0
 
     @property
     def graph_safe(self) -> bool:

@@ -23,6 +23,10 @@ class RMSNorm:
         self.k.rmsnorm(x, self.weight, self.spec.eps, out, delta=delta, rows=rows)
         return out
 
+    def scale_output(self, gain):
+        """From now on the norm's result is ``gain`` times what it was: the weight, kept in float32, takes the factor."""
+        self.weight = (self.weight.float() * gain).contiguous()
+
 
 register_part(RMSNormSpec, RMSNorm)
 

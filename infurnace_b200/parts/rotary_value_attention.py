@@ -1,17 +1,19 @@
-"""Softmax attention over the paged cache whose values are normalised and rotated by their position."""
+"""Grouped-query softmax attention over page streams of keys and values: optional biases, positions on queries, keys and
+values, normalised values, a soft cap on the scores, a sink in the softmax, queries over another layer's keys and values."""
 from __future__ import annotations
 
 import torch
 
 from ..config.specs import RotaryValueAttentionSpec
-from .registry import build_part, register_part
+from .registry import build_part, fold_residual_norm, register_part, unfolded
 
 
 class RotaryValueAttention:
     """h -> o_proj(unrotate(attention(q, K, V))).
 
     q | k | v run as one product (q | k where the description has no value projection: a value head is then its key head
-    as projected, before the rotation).  One kernel rotates the q and k heads on their first rotary_dim entries, divides
+    as projected, before the rotation), the biases added in it.  A part that ``reads_cache`` has the q product alone, which
+    then writes the queries in the cache's dtype, and stores nothing.  One kernel rotates the q and k heads on their first rotary_dim entries, divides
     each value head by its root mean square and rotates it over its whole width by the token's position, writes q
     in the cache's dtype and k and v into their page streams (which may differ in width).  The attention kernel reads
     every key and value from the pages, this step's included, keeps scores, softmax weights and sums in float32,
@@ -24,11 +26,18 @@ class RotaryValueAttention:
         self.spec = spec
         self.rt = runtime
         self.k = runtime.kernels
-        self.values_are_keys = spec.v_proj is None
+        self.values_are_keys = spec.v_proj is None and not spec.reads_cache
         if self.values_are_keys and (spec.value_head_dim != spec.head_dim or spec.value_norm or spec.value_position is not None):
             raise ValueError("values that are the keys have the keys' width, no norm and no rotation of their own")
-        names = (spec.q_proj, spec.k_proj) if self.values_are_keys else (spec.q_proj, spec.k_proj, spec.v_proj)
-        self.w_qkv = torch.cat([weights[n] for n in names], dim=0).contiguous()
+        if spec.reads_cache and (spec.value_norm or spec.k_proj is not None or spec.v_proj is not None):
+            raise ValueError("a mixer that reads another's keys and values makes none")
+        pairs = [(p, b) for p, b in ((spec.q_proj, spec.q_bias), (spec.k_proj, spec.k_bias), (spec.v_proj, spec.v_bias)) if p is not None]
+        self.w_qkv = torch.cat([weights[p] for p, _ in pairs], dim=0).contiguous()
+        self.bias = None
+        if any(b is not None for _, b in pairs):          # float32, zeros where a projection has none
+            self.bias = torch.cat([weights[b].float() if b is not None else
+                                   torch.zeros(weights[p].shape[0], dtype=torch.float32, device=weights[p].device)
+                                   for p, b in pairs], dim=0).contiguous()
         self.w_o = weights[spec.o_proj]
         self.position = build_part(spec.position, weights, runtime) if spec.position is not None else None
         self.value_position = build_part(spec.value_position, weights, runtime) if spec.value_position is not None else None
@@ -36,52 +45,90 @@ class RotaryValueAttention:
             raise ValueError("the values are rotated over their whole width")
         import os
         self.exact_weights = os.environ.get("INFURNACE_EXACT_ATTENTION", "0") not in ("", "0")
-        self.width = spec.num_heads * spec.head_dim + spec.num_kv_heads * (
-            spec.head_dim + (0 if self.values_are_keys else spec.value_head_dim))
+        self.width = self.w_qkv.shape[0]
+        # what the call of the streams' attention kernel needs beyond the plain softmax
+        self.extra = {key: value for key, value in (("softcap", spec.softcap), ("sink", spec.sink_score)) if value is not None}
+        if spec.weight_terms != 1:
+            self.extra["weight_terms"] = spec.weight_terms
 
-    def _on_tensor_cores(self, kv):
+    can_fold_output = True
+
+    def can_take_folded(self, n):
+        can = getattr(self.k, "can_fold_norm", None)
+        return bool(can and can(n, self.rt.act_dtype, self.w_qkv))
+
+    def _plain_on_tensor_cores(self, kv):
         """bfloat16 with keys and values of one width in one tensor: the framework's tensor-core attention kernels run
         (scores and softmax in float32; the weights are rounded to bfloat16 as the left operand of the P V product, which
-        accumulates in float32).  Everything else, and every step when ``exact_weights`` is set, runs the plain kernel,
-        which keeps the weights in float32 through the sum."""
+        accumulates in float32).  Everything else goes to the streams' entry, which takes its tensor-core route where the
+        sizes allow (widths of their own for keys and values, a soft cap, a sink) and, when ``exact_weights`` is set, always the
+        plain kernel, which keeps the weights in float32 through the sum."""
         s = self.spec
         group = s.num_heads // s.num_kv_heads
-        return (not self.exact_weights and self.rt.act_dtype == torch.bfloat16 and kv.pages is not None
+        return (not self.exact_weights and s.softcap is None and s.sink_score is None and self.rt.act_dtype == torch.bfloat16 and kv.pages is not None
                 and s.head_dim == s.value_head_dim and s.head_dim % 16 == 0 and s.head_dim <= 256 and group <= 16
                 and hasattr(self.k, "rotate_rows"))
 
-    def forward(self, h, ctx, call):
+    def _project(self, h, row_scale, out):
+        args = {}
+        if row_scale is not None:
+            args["row_scale"] = row_scale
+        if self.bias is not None:
+            args["bias"] = self.bias
+        self.k.linear(h, self.w_qkv, out, **args)
+
+    def _queries(self, h, row_scale, ctx, call, kv, v_table):
+        """The step's queries in the cache's dtype; its keys and values, if the part makes any, in the pages."""
         s, k = self.spec, self.k
         n = h.shape[0]
-        qkv = ctx.buffer("rva_qkv", (n, self.width), torch.float32)
-        k.linear(h, self.w_qkv, qkv)
-        kv = ctx.kv(call.cache)
         pk, pv = kv.streams["k"], kv.streams["v"]
         q = ctx.buffer("rva_q", (n, s.num_heads * s.head_dim), self.rt.act_dtype)
         qk_table = self.position.table(ctx) if self.position is not None else None
-        v_table = self.value_position.table(ctx) if self.value_position is not None else None
+        if s.reads_cache:
+            self._project(h, row_scale, q)
+            if qk_table is not None:
+                k.rotate_rows(q, qk_table, s.num_heads, s.head_dim, s.position.rotary_dim, bool(s.position.interleaved))
+            return q
+        qkv = ctx.buffer("rva_qkv", (n, self.width), torch.float32)
+        self._project(h, row_scale, qkv)
         k.rotary_store(qkv, s.num_heads, s.num_kv_heads, s.head_dim, s.value_head_dim, qk_table,
                        s.position.rotary_dim if s.position is not None else 0,
                        bool(s.position.interleaved) if s.position is not None else False,
                        s.eps if s.value_norm else None, v_table,
                        bool(s.value_position.interleaved) if s.value_position is not None else False,
                        q, pk, pv, kv.slot_mapping if call.store else None, **({"values_are_keys": True} if self.values_are_keys else {}))
-        out = ctx.buffer("rva_out", (n, s.num_heads * s.value_head_dim), self.rt.act_dtype)
-        if self._on_tensor_cores(kv):
+        return q
+
+    def forward(self, h, ctx, call, fold=None, out=None):
+        """``fold``: as :meth:`GatedMLP.forward`'s.  ``out``: where the result goes if it is not folded into the stream (default: a
+        buffer of the part's)."""
+        s, k = self.spec, self.k
+        h, row_scale = unfolded(h)
+        n = h.shape[0]
+        kv = ctx.kv(call.cache)
+        pk, pv = kv.streams["k"], kv.streams["v"]
+        v_table = self.value_position.table(ctx) if self.value_position is not None else None
+        q = self._queries(h, row_scale, ctx, call, kv, v_table)
+        attn = ctx.buffer("rva_out", (n, s.num_heads * s.value_head_dim), self.rt.act_dtype)
+        if self._plain_on_tensor_cores(kv):
             # the framework's tensor-core attention over the entry's one tensor of keys and values, then the turn back
-            k.paged_attention(q, s.num_heads, s.num_kv_heads, s.head_dim, kv.pages, kv.block_tables, ctx.cu_q, ctx.seq_lens, out,
+            k.paged_attention(q, s.num_heads, s.num_kv_heads, s.head_dim, kv.pages, kv.block_tables, ctx.cu_q, ctx.seq_lens, attn,
                               s.scale, s.window or 0, ctx.max_q_len, ctx.max_seq_len, min_q_len=ctx.min_q_len,
                               **({"weight_terms": s.weight_terms} if s.weight_terms != 1 else {}))
             if v_table is not None:
-                k.rotate_rows(out, v_table, s.num_heads, s.value_head_dim, s.value_head_dim, bool(s.value_position.interleaved),
+                k.rotate_rows(attn, v_table, s.num_heads, s.value_head_dim, s.value_head_dim, bool(s.value_position.interleaved),
                               back=True)
         else:
             k.paged_attention_streams(q, s.num_heads, s.num_kv_heads, s.head_dim, s.value_head_dim, pk, pv, kv.block_tables,
-                                      ctx.cu_q, ctx.seq_lens, out, s.scale, s.window or 0, v_table,
+                                      ctx.cu_q, ctx.seq_lens, attn, s.scale, s.window or 0, v_table,
                                       bool(s.value_position.interleaved) if s.value_position is not None else False,
-                                      max_q_len=ctx.max_q_len, max_seq_len=ctx.max_seq_len)
-        delta = ctx.buffer("delta_mixer", (n, s.hidden_size), torch.float32)
-        k.linear(out, self.w_o, delta)
+                                      max_q_len=ctx.max_q_len, max_seq_len=ctx.max_seq_len, min_q_len=ctx.min_q_len,
+                                      exact=self.exact_weights, **self.extra)
+        folded = fold_residual_norm(k, ctx, "mixer", attn, self.w_o, fold, self.rt.act_dtype)
+        if folded is not None:
+            return folded
+        delta = out if out is not None else ctx.buffer("delta_mixer", (n, s.hidden_size), torch.float32)
+        k.linear(attn, self.w_o, delta)
         return delta
 
 

@@ -23,8 +23,8 @@ class ReferenceKernels:
         self.fold = fold          # offer the folded norm (for few rows, as the CUDA kernels do)
 
     # ------------------------------------------------------------------ embedding
-    def embed(self, table, ids, out):
-        out.copy_(table[ids.long()].to(out.dtype))
+    def embed(self, table, ids, out, scale=1.0):
+        out.copy_(table[ids.long()].to(out.dtype) * scale)
 
     def random_normal(self, out, seed64, mean, std):
         """out[i] = mean + std * z_i, the counter-based values of weights/random_init.py."""
@@ -56,33 +56,39 @@ class ReferenceKernels:
         out.copy_(y.to(out.dtype))
 
     # ------------------------------------------------------------------ matrix products
-    def linear(self, x, w, out, epilogue="none", row_scale=None):
+    def linear(self, x, w, out, epilogue="none", row_scale=None, bias=None):
         """out = x @ w^T (w is [out_features, in_features]); accumulation in 32-bit.
         epilogue "silu_gate": w is [2I, K] with the gate rows first; out[n, j] =
         silu(y[n, j]) * y[n, I + j].  row_scale (partials, parts, eps, width): row n of the
-        product is multiplied by rsqrt(sum_p partials[p, n] / width + eps) first."""
+        product is multiplied by rsqrt(sum_p partials[p, n] / width + eps) first; bias is added after that."""
         y = x.to(self.cd) @ w.to(self.cd).t()
         if row_scale is not None:
             partials, parts, eps, width = row_scale
             r = torch.rsqrt(partials[:parts].to(self.cd).sum(dim=0) / width + eps)
             y = y * r[:, None]
+        if bias is not None:
+            y = y + bias.to(self.cd)
+        out.copy_(self._epilogue(y, epilogue).to(out.dtype))
+
+    @staticmethod
+    def _epilogue(y, epilogue):
         if epilogue == "silu_gate":
             half = y.shape[1] // 2
             g, u = y[:, :half], y[:, half:]
-            y = g * torch.sigmoid(g) * u
-        elif epilogue == "relu2":
-            y = torch.relu(y) ** 2
-        elif epilogue == "silu":
-            y = y * torch.sigmoid(y)
-        elif epilogue == "sigmoid":
-            y = torch.sigmoid(y)
-        elif epilogue == "gelu_tanh":
-            y = 0.5 * y * (1 + torch.tanh(0.7978845608028654 * (y + 0.044715 * y ** 3)))
-        elif epilogue == "tanh":
-            y = torch.tanh(y)
-        elif epilogue != "none":
+            return g * torch.sigmoid(g) * u
+        if epilogue == "relu2":
+            return torch.relu(y) ** 2
+        if epilogue == "silu":
+            return y * torch.sigmoid(y)
+        if epilogue == "sigmoid":
+            return torch.sigmoid(y)
+        if epilogue == "gelu_tanh":
+            return 0.5 * y * (1 + torch.tanh(0.7978845608028654 * (y + 0.044715 * y ** 3)))
+        if epilogue == "tanh":
+            return torch.tanh(y)
+        if epilogue != "none":
             raise ValueError(epilogue)
-        out.copy_(y.to(out.dtype))
+        return y
 
     def can_fold_norm(self, n, dtype, w, epilogue="none"):
         return bool(self.fold) and 0 < n <= 64
@@ -517,9 +523,11 @@ class ReferenceKernels:
         rows.copy_(t.reshape(rows.shape).to(rows.dtype))
 
     def paged_attention_streams(self, q, num_heads, num_kv_heads, head_dim, value_head_dim, k_pages, v_pages, block_tables, cu_q,
-                                seq_lens, out, scale, window, out_table, out_interleaved, max_q_len=0, max_seq_len=0):
+                                seq_lens, out, scale, window, out_table, out_interleaved, max_q_len=0, max_seq_len=0, min_q_len=1,
+                                softcap=None, sink=None, weight_terms=1, exact=True):
         """Causal softmax attention of q [n, H d] over the keys and values of the request's pages (streams
-        [pages, G, page_size, width]); the output of every head is then rotated BACK by the angles of out_table (the
+        [pages, G, page_size, width]); a scaled score s becomes softcap * tanh(s / softcap), exp(sink) joins the denominator;
+        the output of every head is then rotated BACK by the angles of out_table (the
         query token's row; None: not)."""
         H, G, d, dv = num_heads, num_kv_heads, head_dim, value_head_dim
         ps = k_pages.shape[2]
@@ -536,6 +544,11 @@ class ReferenceKernels:
                 kk = k_pages[pages, :, pos % ps, :].to(self.cd).repeat_interleave(H // G, dim=1)
                 vv = v_pages[pages, :, pos % ps, :].to(self.cd).repeat_interleave(H // G, dim=1)
                 a = torch.einsum("hd,shd->hs", q[t].to(self.cd).view(H, d), kk) * scale
+                if softcap is not None:
+                    a = softcap * torch.tanh(a / softcap)
+                if sink is not None:                   # a key of score ``sink`` whose value is zero
+                    a = torch.cat((a, torch.full((H, 1), sink, dtype=self.cd)), dim=1)
+                    vv = torch.cat((vv, torch.zeros(1, H, dv, dtype=self.cd)), dim=0)
                 o = torch.einsum("hs,shd->hd", torch.softmax(a, dim=-1), vv)[None]
                 if out_table is not None:
                     c, s_ = self._table(out_table[t:t + 1])
@@ -543,12 +556,34 @@ class ReferenceKernels:
                 out[t] = o.reshape(H * dv).to(out.dtype)
 
     # ------------------------------------------------------------------ routed experts
-    def moe_route(self, logits, top, ids, gates, experts=None, scoring="chosen", groups=None, weight_scale=1.0):
+    def moe_route(self, logits, top, ids, gates, experts=None, scoring="chosen", groups=None, weight_scale=1.0, correction=None,
+                  normalise=False, group_best=1):
         """ids[n] = the ``top`` largest scores' indices, largest first (the lower index among equals).  scoring "chosen":
         scores are the logits, gates[n] = softmax over the chosen logits.  scoring "all": scores are the softmax over all
         experts, limited to the ``keep`` groups of neighbours with the largest best score when ``groups`` = (count, keep);
-        gates[n] = score * weight_scale.  Only the first ``experts`` columns of ``logits`` are the router's."""
+        gates[n] = score * weight_scale.  scoring "sigmoid": sigmoid(logit), likewise; ``correction`` is added for the choice only,
+        ``normalise`` divides the chosen scores by their sum + 1e-20; a group counts by the sum of its ``group_best`` largest.
+        Only the first ``experts`` columns of ``logits`` are the router's."""
         z = logits[:, :experts if experts is not None else logits.shape[1]].to(self.cd)
+        if scoring == "sigmoid" and (correction is not None or normalise or groups):
+            score = torch.sigmoid(z)
+            choice = score if correction is None else score + correction.to(self.cd)
+            if groups is not None and groups[1] < groups[0]:
+                count, keep = groups
+                n, E = score.shape
+                per = torch.sort(choice.view(n, count, E // count), dim=-1, descending=True).values
+                value = per[..., :group_best].sum(-1)
+                order = torch.sort(value, dim=-1, descending=True, stable=True).indices[:, :keep]
+                allowed = torch.zeros(n, count, dtype=torch.bool)
+                allowed.scatter_(1, order, True)
+                choice = choice.masked_fill(~allowed.repeat_interleave(E // count, dim=1), -float("inf"))
+            idx = torch.sort(choice, dim=-1, descending=True, stable=True).indices[:, :top]
+            w = torch.gather(score, 1, idx) * weight_scale
+            if normalise:
+                w = w / (torch.gather(score, 1, idx).sum(-1, keepdim=True) + 1e-20)
+            ids.copy_(idx.to(ids.dtype))
+            gates.copy_(w.to(gates.dtype))
+            return
         if scoring == "sigmoid":         # sigmoid(z) per expert; the order of the logits is the order of the scores
             val, idx = torch.sort(z, dim=-1, descending=True, stable=True)
             ids.copy_(idx[:, :top].to(ids.dtype))
@@ -573,10 +608,9 @@ class ReferenceKernels:
         ids.copy_(idx.to(ids.dtype))
         gates.copy_((torch.gather(score, 1, idx) * weight_scale).to(gates.dtype))
 
-    def moe_route_plan(self, logits, top, ids, gates, offsets, perm, pos, experts=None, scoring="chosen", groups=None,
-                       weight_scale=1.0):
+    def moe_route_plan(self, logits, top, ids, gates, offsets, perm, pos, experts=None, **how):
         """moe_route, then moe_plan."""
-        self.moe_route(logits, top, ids, gates, experts=experts, scoring=scoring, groups=groups, weight_scale=weight_scale)
+        self.moe_route(logits, top, ids, gates, experts=experts, **how)
         self.moe_plan(ids, experts if experts is not None else logits.shape[1], offsets, perm, pos)
 
     def moe_plan(self, ids, num_experts, offsets, perm, pos):
@@ -599,12 +633,7 @@ class ReferenceKernels:
                 continue
             rows = x[(perm[a:b].long() // top)] if perm is not None else x[a:b]
             y = rows.to(self.cd) @ w[e].to(self.cd).t()
-            if epilogue == "silu_gate":
-                half = y.shape[1] // 2
-                y = y[:, :half] * torch.sigmoid(y[:, :half]) * y[:, half:]
-            elif epilogue != "none":
-                raise ValueError(epilogue)
-            out[a:b] = y.to(out.dtype)
+            out[a:b] = self._epilogue(y, epilogue).to(out.dtype)
 
     def moe_gather_scaled(self, x, perm, top, gates, out, tile_expert=None):
         """out[place] = gates[perm[place]] * x[perm[place] // top], zeros where perm[place] < 0."""
@@ -617,8 +646,21 @@ class ReferenceKernels:
     def moe_combine(self, y, pos, gates, out, shared=None, shared_logit=None):
         """out[n] = sum_j gates[n, j] * y[pos[n * top + j]], j ascending (gates None: weights of 1); + shared[n] (times
         sigmoid(shared_logit[n]))."""
+        out.copy_(self._combined(y, pos, gates, out.shape[0], shared, shared_logit).to(out.dtype))
+
+    def moe_combine_update(self, y, pos, gates, x, base=None, shared=None, shared_logit=None, out=None, next_weight=None, eps=0.0):
+        """x += base + (what moe_combine writes); out = x / sqrt(mean(x^2) + eps) * next_weight of the new rows."""
+        acc = self._combined(y, pos, gates, x.shape[0], shared, shared_logit)
+        if base is not None:
+            acc = acc + base.to(self.cd)
+        x.copy_((x.to(self.cd) + acc).to(x.dtype))
+        if out is not None:
+            v = x.to(self.cd)
+            out.copy_((v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * next_weight.to(self.cd)).to(out.dtype))
+
+    def _combined(self, y, pos, gates, rows, shared, shared_logit):
         if gates is None:
-            gates = torch.ones(out.shape[0], pos.numel() // max(out.shape[0], 1), dtype=self.cd)
+            gates = torch.ones(rows, pos.numel() // max(rows, 1), dtype=self.cd)
         n, top = gates.shape
         acc = torch.zeros(n, y.shape[1], dtype=self.cd)
         for j in range(top):
@@ -626,7 +668,7 @@ class ReferenceKernels:
         if shared is not None:
             g = torch.sigmoid(shared_logit.to(self.cd))[:, None] if shared_logit is not None else 1.0
             acc = acc + g * shared.to(self.cd)
-        out.copy_(acc.to(out.dtype))
+        return acc
 
     # ------------------------------------------------------------------ decoders with latent attention
     def _group_norm(self, v, weight, groups, eps):
