@@ -1,4 +1,7 @@
-// Attention for prompts and long portions on the fifth-generation tensor cores, head size 128.
+// Attention for prompts and long portions on the fifth-generation tensor cores.  Compiled for one pair of widths:
+// -DHEAD_DIM=<multiple of 16, at most 192> (default 128), -DVALUE_DIM=<multiple of 16, at most 128> (default HEAD_DIM).
+// Keys and values are two page streams, as in attention_mma.cu (a stream's page p begins page_stride elements after page p - 1).
+// Rows in shared memory are whole 128-byte swizzle rows: the columns beyond a width that is no multiple of 64 are zeros.
 //
 // A CTA takes one query tile of 128 score rows of one key/value head: 128/G query tokens times the G query heads
 // of the group (row = token * G + head-in-group).  The keys are loaded in tiles of 128 (two stages each for K and V)
@@ -27,6 +30,15 @@
 // and 128 columns of output, 512 columns in all, so one CTA per SM.  The grid is the tiles of the longest request
 // times the key/value heads, the tiles with the most keys first, so that the short ones fill the SMs' last rounds.
 //
+// -DWEIGHT_TERMS=2: a softmax weight is the sum of two bfloat16 numbers, its upper 16 bits and the rounding of what they leave
+// out (16 bits of the float32 weight in all).  The two P of a half fill the 64 columns its scores had, and O += P V is the
+// products of both with the same V tile.
+// -DSOFTCAP=1: a scaled score s becomes c tanh(s / c).  Capped scores lie in [-c, c], so their exponentials need no running
+// maximum (the caller gives c of at most TC_MAX_CAP: 2^(c log2 e), summed over any context, is a float32 number): weights are
+// 2^z itself, nothing is ever rescaled.  tanh is a polynomial in two-number FMA instructions where every score of a warp's half
+// is small (|s| <= 0.7 c; absolute error 2e-7), else 1 - 2 / (1 + e^(2 s / c)).
+// A sink z (an argument; -inf: none) joins the denominator as exp(z).
+//
 // Requests are routed as in attention_mma.cu: this kernel takes those with more than 16 score rows,
 // the small-q kernel there takes the others.  Waits on barriers are bounded (TC_SPIN_LIMIT polls, then
 // a code in *err and the CTA's abort flag).
@@ -39,22 +51,35 @@
 #ifndef HEAD_DIM
 #define HEAD_DIM 128
 #endif
-#if HEAD_DIM != 128
-#error "attention_tc.cu is written for head size 128"
+#ifndef VALUE_DIM
+#define VALUE_DIM HEAD_DIM
+#endif
+#if HEAD_DIM % 16 || HEAD_DIM < 16 || HEAD_DIM > 192 || VALUE_DIM % 16 || VALUE_DIM < 16 || VALUE_DIM > 128
+#error "attention_tc.cu takes key widths up to 192 and value widths up to 128, multiples of 16"
+#endif
+#ifndef WEIGHT_TERMS
+#define WEIGHT_TERMS 1
+#endif
+#ifndef SOFTCAP
+#define SOFTCAP 0
 #endif
 
 typedef __nv_bfloat16 bf16;
-constexpr int D = 128;
+constexpr int D = HEAD_DIM, VD = VALUE_DIM;
+constexpr int KH = (D + 63) / 64, VH = (VD + 63) / 64;      // swizzle rows of 64 columns that a key, a value has
+constexpr int VN = VH * 64;                                 // columns of the output accumulator (MMA N of P V)
+constexpr float TC_MAX_CAP = 60.f;
 constexpr int ROWS = 128;                 // score rows per CTA (MMA M)
 constexpr int BK = 128;                   // keys per tile loaded
 constexpr int SUB = 64;                   // keys per score buffer (MMA N of S, K of P V per half)
 constexpr int TC_THREADS = 384;                // producer warp, two MMA warps, an idle warp, two softmax groups of four
 constexpr uint32_t TC_SPIN_LIMIT = 1u << 22;
 constexpr int HALF_BYTES = 128 * 128;     // a [128 rows][64 columns] bf16 half tile in the 128-byte swizzle: 16 KB
-constexpr int TILE_BYTES = 2 * HALF_BYTES;
-constexpr int SMEM_BYTES = 5 * TILE_BYTES /* Q, 2 K, 2 V */ + 1024 /* alignment */;   // 161 KB
+constexpr int K_BYTES = KH * HALF_BYTES, V_BYTES = VH * HALF_BYTES;
+constexpr int SMEM_BYTES = 3 * K_BYTES /* Q, 2 K */ + 2 * V_BYTES + 1024 /* alignment */;   // 161 KB at 128 and 128
+static_assert(SMEM_BYTES <= 226 * 1024, "query, key and value tiles must fit in shared memory");
 // tensor memory columns (32-bit), per stream: two score buffers [0,64) and [64,128), P (bfloat16 pairs) written
-// over the first 32 columns of a buffer once its row has been read, O [128,256).  Two streams: all 512 columns.
+// over the first 32 columns of a buffer (its second term over the last 32) once its row has been read, O [128,128+VN).  Two streams: all 512 columns.
 constexpr int COL_S = 0, COL_O = 128, COLS_PER_TILE = 256, TMEM_COLS = 512;
 constexpr int NO_ROW = -1000000000;
 
@@ -205,22 +230,59 @@ __device__ __forceinline__ uint32_t tc_pack_p(float lo, float hi) {
   return tc_pack(lo, hi);
 #endif
 }
+// A pair of weights as bfloat16 pairs: one term (rounded), or two (the upper 16 bits of each, and the rounding of the rest,
+// which is not negative).
+__device__ __forceinline__ void tc_pack_terms(float e0, float e1, uint32_t& first, uint32_t& second) {
+#if WEIGHT_TERMS == 2
+  const uint32_t u0 = __float_as_uint(e0), u1 = __float_as_uint(e1);
+  asm("prmt.b32 %0, %1, %2, 0x7632;\n" : "=r"(first) : "r"(u0), "r"(u1));
+  second = tc_pack_p(e0 - __uint_as_float(u0 & 0xffff0000u), e1 - __uint_as_float(u1 & 0xffff0000u));
+#else
+  first = tc_pack_p(e0, e1);
+  second = 0u;
+#endif
+}
+// the exponent of a weight: capped scores are exponents already
+#if SOFTCAP
+#define TC_EXPONENT(v) __uint_as_float(v)
+#else
+#define TC_EXPONENT(v) fmaf(__uint_as_float(v), scale_log2, -ref)
+#endif
 
 // K-major operand (rows of 128 bytes = 64 k, groups of 8 rows 1024 bytes apart), 128-byte swizzle: Q and K tiles.
 __device__ __forceinline__ uint64_t desc_k_major(uint32_t addr) {
   return (uint64_t)((addr >> 4) & 0x3FFF) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
 }
+#if SOFTCAP
+// Two float32 numbers per instruction.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 tc_pair(float a, float b) { f32x2 r; asm("mov.b64 %0, {%1, %2};\n" : "=l"(r) : "f"(a), "f"(b)); return r; }
+__device__ __forceinline__ void tc_unpair(f32x2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;\n" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f32x2 tc_mul2(f32x2 a, f32x2 b) { f32x2 r; asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ f32x2 tc_fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+// tanh(y) = y (1 + y^2 (T0 + y^2 (T1 + y^2 (T2 + y^2 T3)))) for |y| <= 0.7, a least-maximum fit of that form: absolute error
+// 1.4e-7, 2e-7 in float32 arithmetic.
+constexpr float TC_T0 = -0.33330065f, TC_T1 = 0.13276916f, TC_T2 = -0.05067464f, TC_T3 = 0.01359966f;
+#endif
+// What becomes of a product q . k before its weight 2^z.  SOFTCAP: y = s * to_y (the scaled score over the cap),
+// z = cap_log2 * tanh(y); `limit`: |s| up to which y is in the polynomial's range.  Else z = s * scale_log2.
+struct TcScore { float scale_log2, to_y, cap_log2, limit; };
+constexpr float TC_TANH_RANGE = 0.7f;
 // MN-major operand, 128-byte swizzle: the V tile [key][dim] as B = [dim (N)][key (K)].  64 dims (128 bytes) are one
 // swizzle row; the next 64 dims lie HALF_BYTES further (leading byte offset); 8 keys are 1024 bytes (stride byte offset).
 __device__ __forceinline__ uint64_t desc_mn_major(uint32_t addr) {
   return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(HALF_BYTES >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) |
          (2ull << 61);
 }
-// float32 accumulator, bfloat16 A and B, M = 128; S = Q K^T: N = 64 keys, B K-major; O += P V: N = 128 (the head
-// size), B MN-major.
+// float32 accumulator, bfloat16 A and B, M = 128; S = Q K^T: N = 64 keys, B K-major; O += P V: N = VN (the values'
+// columns), B MN-major.
 constexpr uint32_t IDESC_BASE = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 4) << 24);
 constexpr uint32_t IDESC_S = IDESC_BASE | ((uint32_t)(SUB >> 3) << 17);
-constexpr uint32_t IDESC_PV = IDESC_BASE | ((uint32_t)(128 >> 3) << 17) | (1u << 16);
+constexpr uint32_t IDESC_PV = IDESC_BASE | ((uint32_t)(VN >> 3) << 17) | (1u << 16);
 
 struct TcBars {
   // [stream][stage or buffer]; q_empty: both issuers have read the query tile; o_free: the softmax warps have read the
@@ -251,11 +313,15 @@ __device__ __forceinline__ bool tc_item(int k, int cta, int ctas, int nt, int nk
   return true;
 }
 
+// The two streams as matrices of rows: how many rows a page spans and how many rows there are.
+struct TcRows { int k_page, v_page, k_total, v_total; };
+
 __global__ void __launch_bounds__(TC_THREADS, 1)
-attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map, int total_rows,
-                    int* __restrict__ err, const int* __restrict__ block_tables, int bt_stride,
-                    const int* __restrict__ cu_q, const int* __restrict__ seq_lens, bf16* __restrict__ out, int nq, int nkv,
-                    int page_size, float scale_log2, int window) {
+attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
+                    const __grid_constant__ CUtensorMap v_map, TcRows mrows, int* __restrict__ err,
+                    const int* __restrict__ block_tables, int bt_stride, const int* __restrict__ cu_q,
+                    const int* __restrict__ seq_lens, bf16* __restrict__ out, int nq, int nkv, int share, int page_size,
+                    TcScore score, float sink, int window) {
   extern __shared__ unsigned char tc_smem_raw[];
   __shared__ TcBars bars;
   __shared__ uint32_t tmem_slot;
@@ -264,9 +330,9 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
   volatile int* abort_flag = &abort_word;
   const uint32_t raw = tc_smem_u32(tc_smem_raw);
   unsigned char* smem = tc_smem_raw + (((raw + 1023u) & ~1023u) - raw);
-  unsigned char* Qs = smem;                                  // the query tile, [2 halves][128 rows][128 bytes]
-  unsigned char* Ks = smem + TILE_BYTES;                     // two stages of K tiles, same layout
-  unsigned char* Vs = smem + 3 * TILE_BYTES;                 // two stages of V tiles
+  unsigned char* Qs = smem;                                  // the query tile, [KH][128 rows][128 bytes]
+  unsigned char* Ks = smem + K_BYTES;                        // two stages of K tiles, same layout
+  unsigned char* Vs = smem + 3 * K_BYTES;                    // two stages of V tiles, [VH][128 rows][128 bytes]
   const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;     // warp-uniform
   const int r = blockIdx.z, cta = blockIdx.x, ctas = gridDim.x;
   const int G = nq / nkv;
@@ -283,6 +349,10 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
   const int* bt = block_tables + (size_t)r * bt_stride;
   const int ps_shift = __ffs(page_size) - 1;
 
+  if (tpt * G < ROWS) {                                      // rows of the tile that no query fills: zeros, once
+    for (int i = threadIdx.x; i < K_BYTES / 16; i += TC_THREADS) reinterpret_cast<uint4*>(Qs)[i] = make_uint4(0u, 0u, 0u, 0u);
+    asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+  }
   if (threadIdx.x == 0) {
     tc_mbar_init(&bars.q_full, 1);
     tc_mbar_init(&bars.q_empty, 2);
@@ -319,7 +389,8 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
     ifb_pdl_wait();
     if (!kv) ifb_pdl_trigger();
     const int ppt = BK >> ps_shift;                          // pages per tile: 8, 4 or 2
-    const int n_ops = ppt * 2;                               // x 2 halves: at most 16 per tile
+    const int halves = kv ? VH : KH;                         // swizzle rows per key or value
+    const int n_ops = ppt * halves;                          // at most 8 x 3 per tile
     bool ok = true;
     int jt = 0, ic = 0;                                      // tiles and items so far
     for (int k = 0; k < n_rounds && ok; ++k) {
@@ -329,9 +400,9 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
         if (ic > 0) ok = tc_mbar_wait(&bars.q_empty, (ic - 1) & 1, abort_flag, err, 10);
         if (!ok) break;
         if (lane == 0) {
-          tc_mbar_expect_tx(&bars.q_full, TILE_BYTES);
-          tc_tma_3d(Qs, &q_map, &bars.q_full, 0, it.kvh * G, q0 + it.t0);
-          tc_tma_3d(Qs + HALF_BYTES, &q_map, &bars.q_full, 64, it.kvh * G, q0 + it.t0);
+          tc_mbar_expect_tx(&bars.q_full, (uint32_t)(KH * tpt * G * 128));
+#pragma unroll
+          for (int hf = 0; hf < KH; ++hf) tc_tma_3d(Qs + hf * HALF_BYTES, &q_map, &bars.q_full, hf * 64, it.kvh * G, q0 + it.t0);
         }
         __syncwarp();
       }
@@ -344,14 +415,16 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
             if (ok) ok = tc_mbar_wait(kv ? &bars.v_empty[x][st] : &bars.k_empty[x][st], ((jt >> 1) - 1) & 1, abort_flag, err, 11);
         }
         if (!ok) break;
-        if (lane == 0) tc_mbar_expect_tx(full, TILE_BYTES);
+        if (lane == 0) tc_mbar_expect_tx(full, kv ? V_BYTES : K_BYTES);
         __syncwarp();
         if (lane < n_ops) {
-          const int pg = lane >> 1, half = lane & 1;
+          const int pg = lane / halves, half = lane % halves;
           const int key0 = it.T0 + j * BK + pg * page_size;
-          int y = total_rows;                                // beyond the tensor: zeros
-          if (key0 <= it.hi && key0 + page_size - 1 >= it.lo) y = ((bt[key0 >> ps_shift] * 2 + kv) * nkv + it.kvh) * page_size;
-          tc_tma_2d((kv ? Vs : Ks) + st * TILE_BYTES + half * HALF_BYTES + pg * page_size * 128, &kv_map, full, half * 64, y);
+          int y = kv ? mrows.v_total : mrows.k_total;        // beyond the tensor: zeros
+          if (key0 <= it.hi && key0 + page_size - 1 >= it.lo)
+            y = bt[key0 >> ps_shift] * (kv ? mrows.v_page : mrows.k_page) + it.kvh / share * page_size;
+          tc_tma_2d((kv ? Vs + st * V_BYTES : Ks + st * K_BYTES) + half * HALF_BYTES + pg * page_size * 128, kv ? &v_map : &k_map, full,
+                    half * 64, y);
         }
       }
       ++ic;
@@ -374,16 +447,16 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
       const int n_mine = (it.n_half + 1 - x) / 2;
       ok = tc_mbar_wait(&bars.q_full, ic & 1, abort_flag, err, 12);
       auto issue_qk = [&](int i) {
-        // S = Q K^T for the stream's 64 keys of the item's tile i: 8 steps of 16 along the head size, 4 per 64-column
-        // half of Q and K; then the stream is done with the tile of keys (and, after its last half, with the queries)
+        // S = Q K^T for the stream's 64 keys of the item's tile i: D / 16 steps of 16 along the head size, 4 per 64-column
+        // part of Q and K; then the stream is done with the tile of keys (and, after its last half, with the queries)
         const int st = (kc + i) & 1, buf = (hc + i) & 1;
         ok = ok && tc_mbar_wait(&bars.k_full[st], ((kc + i) >> 1) & 1, abort_flag, err, 13);
         if (!ok) return;
         tc_fence_after();
         if (tc_elect_one()) {
-          const uint64_t qd = desc_k_major(q_addr), kd = desc_k_major(k_addr + st * TILE_BYTES);
+          const uint64_t qd = desc_k_major(q_addr), kd = desc_k_major(k_addr + st * K_BYTES);
 #pragma unroll
-          for (int ks = 0; ks < 8; ++ks) {
+          for (int ks = 0; ks < D / 16; ++ks) {
             const uint32_t off = ((ks >> 2) * HALF_BYTES + (ks & 3) * 32) >> 4;       // descriptor addresses count 16 bytes
             tc_mma_ss(tb + COL_S + buf * SUB, qd + off, kd + off, IDESC_S, ks != 0);
           }
@@ -405,10 +478,15 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
         tc_fence_after();
         // O += P V: 4 steps of 16 keys; P at 8 columns (16 bfloat16) per step, V 2048 bytes (16 key rows) per step
         if (tc_elect_one()) {
-          const uint64_t vd = desc_mn_major(v_addr + st * TILE_BYTES);
+          const uint64_t vd = desc_mn_major(v_addr + st * V_BYTES);
 #pragma unroll
           for (int ks = 0; ks < 4; ++ks)
             tc_mma_ts(tb + COL_O, tb + COL_S + buf * SUB + ks * 8, vd + ks * (2048 >> 4), IDESC_PV, (i | ks) != 0);
+          if (WEIGHT_TERMS == 2) {                           // the weights' second terms, 32 columns on
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks)
+              tc_mma_ts(tb + COL_O, tb + COL_S + buf * SUB + 32 + ks * 8, vd + ks * (2048 >> 4), IDESC_PV, 1u);
+          }
           tc_commit(&bars.o_done[x]);
           tc_commit(&bars.v_empty[x][st]);
         }
@@ -451,7 +529,7 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
       const int p = tok < t1x ? p_first + tok : NO_ROW;
       const int row_lo = window > 0 ? p - window + 1 : 0;
       const int lox = it.lo, hix = it.hi;
-      float m_used = -INFINITY, l = 0.f;
+      float m_used = SOFTCAP ? 0.f : -INFINITY, l = 0.f;      // capped scores: the reference is 0 throughout
       for (int u = 0; u < n_mine && ok; ++u) {
         const int c = hc + u, h = c & 1;
         ok = __all_sync(0xffffffffu, tc_mbar_wait(&bars.s_full[x][h], (c >> 1) & 1, abort_flag, err, 15)) != 0;    // warp-uniform
@@ -470,6 +548,49 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
 #pragma unroll
         for (int cc = 0; cc < 2; ++cc) tc_ld32(s_addr + cc * 32, v[cc]);
         tc_wait_ld();
+        bool o_waited = false;                 // whether this step has waited for the previous half's P V
+#if SOFTCAP
+        // the capped scores in the base-2 domain, in place
+        {
+          float am[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+          for (int cc = 0; cc < 2; ++cc)
+#pragma unroll
+            for (int i = 0; i < 32; i += 2)
+              am[(cc << 1) | ((i >> 1) & 1)] = tc_max3(am[(cc << 1) | ((i >> 1) & 1)], fabsf(__uint_as_float(v[cc][i])), fabsf(__uint_as_float(v[cc][i + 1])));
+          const float top = fmaxf(fmaxf(am[0], am[1]), fmaxf(am[2], am[3]));
+          if (__all_sync(0xffffffffu, top <= score.limit)) {
+            const f32x2 ty = tc_pair(score.to_y, score.to_y), c0 = tc_pair(score.cap_log2, score.cap_log2);
+            const float a1 = score.cap_log2 * TC_T0, a2 = score.cap_log2 * TC_T1, a3 = score.cap_log2 * TC_T2, a4 = score.cap_log2 * TC_T3;
+            const f32x2 c1 = tc_pair(a1, a1), c2 = tc_pair(a2, a2), c3 = tc_pair(a3, a3), c4 = tc_pair(a4, a4);
+#pragma unroll
+            for (int cc = 0; cc < 2; ++cc)
+#pragma unroll
+              for (int i = 0; i < 32; i += 2) {
+                const f32x2 y = tc_mul2(tc_pair(__uint_as_float(v[cc][i]), __uint_as_float(v[cc][i + 1])), ty);
+                const f32x2 w = tc_mul2(y, y);
+                f32x2 t = tc_fma2(w, c4, c3);
+                t = tc_fma2(w, t, c2);
+                t = tc_fma2(w, t, c1);
+                t = tc_fma2(w, t, c0);
+                float z0, z1;
+                tc_unpair(tc_mul2(y, t), z0, z1);
+                v[cc][i] = __float_as_uint(z0); v[cc][i + 1] = __float_as_uint(z1);
+              }
+          } else {
+            const float e2 = score.to_y * 2.8853900817779268f, two = -2.f * score.cap_log2;      // 2 log2(e)
+#pragma unroll
+            for (int cc = 0; cc < 2; ++cc)
+#pragma unroll
+              for (int i = 0; i < 32; ++i) {
+                float rc;
+                asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(rc) : "f"(1.f + tc_exp2(__uint_as_float(v[cc][i]) * e2)));
+                v[cc][i] = __float_as_uint(fmaf(two, rc, score.cap_log2));
+              }
+          }
+        }
+#else
+        const float scale_log2 = score.scale_log2;
         // the row's maximum over the visible keys, four chains
         float mxc[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
         if (interior) {
@@ -499,7 +620,6 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
           m_used = m_new;
         }
         const float ref = m_used == -INFINITY ? 0.f : m_used;
-        bool o_waited = false;                 // whether this step has waited for the previous half's P V
         if (u > 0 && any_grow) {
           // O is rescaled between the previous half's P V, which must have landed, and this half's, which waits for P
           ok = __all_sync(0xffffffffu, tc_mbar_wait(o_done, (c - 1) & 1, abort_flag, err, 16)) != 0;
@@ -508,7 +628,7 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
           tc_fence_after();
           l *= factor;
 #pragma unroll 1
-          for (int cc = 0; cc < 8; ++cc) {
+          for (int cc = 0; cc < VN / 16; ++cc) {
             uint32_t o[16];
             tc_ld16(lane_addr + COL_O + cc * 16, o);
             tc_wait_ld();
@@ -517,33 +637,35 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
             tc_st16(lane_addr + COL_O + cc * 16, o);
           }
         }
+#endif
         // p = 2^(s - ref), the row sum, and P as bfloat16 pairs over the first 32 columns of this score buffer (its
         // scores are all in registers by now)
         float lc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int cc = 0; cc < 2; ++cc) {
           uint32_t pk[16];
+          uint32_t pr[16];                                     // the second terms, where there are two
           if (interior) {
-#pragma unroll
             tc_static_for<16>([&](auto idx) {
               constexpr int i = decltype(idx)::value * 2;
-              const float e0 = tc_exp2_mixed<i>(fmaf(__uint_as_float(v[cc][i]), scale_log2, -ref));
-              const float e1 = tc_exp2_mixed<i + 1>(fmaf(__uint_as_float(v[cc][i + 1]), scale_log2, -ref));
+              const float e0 = tc_exp2_mixed<i>(TC_EXPONENT(v[cc][i]));
+              const float e1 = tc_exp2_mixed<i + 1>(TC_EXPONENT(v[cc][i + 1]));
               lc[i & 2] += e0; lc[(i & 2) + 1] += e1;
-              pk[i >> 1] = tc_pack_p(e0, e1);
+              tc_pack_terms(e0, e1, pk[i >> 1], pr[i >> 1]);
             });
           } else {
 #pragma unroll
             for (int i = 0; i < 32; i += 2) {
               const bool v0 = cc * 32 + i < vis_hi && cc * 32 + i >= vis_lo;
               const bool v1 = cc * 32 + i + 1 < vis_hi && cc * 32 + i + 1 >= vis_lo;
-              const float e0 = v0 ? tc_exp2(fmaf(__uint_as_float(v[cc][i]), scale_log2, -ref)) : 0.f;
-              const float e1 = v1 ? tc_exp2(fmaf(__uint_as_float(v[cc][i + 1]), scale_log2, -ref)) : 0.f;
+              const float e0 = v0 ? tc_exp2(TC_EXPONENT(v[cc][i])) : 0.f;
+              const float e1 = v1 ? tc_exp2(TC_EXPONENT(v[cc][i + 1])) : 0.f;
               lc[i & 2] += e0; lc[(i & 2) + 1] += e1;
-              pk[i >> 1] = tc_pack_p(e0, e1);
+              tc_pack_terms(e0, e1, pk[i >> 1], pr[i >> 1]);
             }
           }
           tc_st16(s_addr + cc * 16, pk);
+          if (WEIGHT_TERMS == 2) tc_st16(s_addr + 32 + cc * 16, pr);
         }
         l += (lc[0] + lc[1]) + (lc[2] + lc[3]);
         tc_wait_st();
@@ -562,7 +684,8 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
       }
       if (ok && n_mine > 0) ok = __all_sync(0xffffffffu, tc_mbar_wait(o_done, (hc + n_mine - 1) & 1, abort_flag, err, 17)) != 0;
       // The streams hand each other their maxima and sums; each then divides and stores half of the head's columns,
-      // out = (2^(m0 - m) O0 + 2^(m1 - m) O1) / (2^(m0 - m) l0 + 2^(m1 - m) l1) with m the larger of the two maxima.
+      // out = (2^(m0 - m) O0 + 2^(m1 - m) O1) / (2^(m0 - m) l0 + 2^(m1 - m) l1 + 2^(sink - m)) with m the largest of the two
+      // maxima and the sink.
       const int par = ic & 1;
       merge_m[par][x][row] = m_used;
       merge_l[par][x][row] = l;
@@ -572,19 +695,20 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
       const bool go = __all_sync(0xffffffffu, !*abort_flag) != 0;      // warp-uniform: the loads below are the whole warp's
       if (go) {
         const float m0 = merge_m[par][0][row], m1 = merge_m[par][1][row], l0 = merge_l[par][0][row], l1 = merge_l[par][1][row];
-        const float m = fmaxf(m0, m1);
+        const float m = fmaxf(fmaxf(m0, m1), sink);
         const float a0 = m0 == -INFINITY ? 0.f : tc_exp2(m0 - m), a1 = m1 == -INFINITY ? 0.f : tc_exp2(m1 - m);
-        const float denom = a0 * l0 + a1 * l1;
+        const float denom = a0 * l0 + a1 * l1 + (sink == -INFINITY ? 0.f : tc_exp2(sink - m));
         const float inv = denom > 0.f ? 1.f / denom : 0.f;
         const float w0 = a0 * inv, w1 = a1 * inv;
         const bool two = it.n_half > 1;                          // stream 1's accumulator holds something of this item
         const uint32_t o_addr = tmem + ((uint32_t)(qd * 32) << 16) + COL_O;
-        bf16* dst = p != NO_ROW ? out + ((size_t)(q0 + tok) * nq + kvh * G + row % G) * D + x * 64 : nullptr;
+        bf16* dst = p != NO_ROW ? out + ((size_t)(q0 + tok) * nq + kvh * G + row % G) * VD : nullptr;
 #pragma unroll 1
-        for (int cc = 0; cc < 2; ++cc) {
+        for (int cc = 0; cc < VN / 64; ++cc) {
+          const int col0 = x * (VN / 2) + cc * 32;
           uint32_t oa[32], ob[32];
-          tc_ld32(o_addr + x * 64 + cc * 32, oa);
-          if (two) tc_ld32(o_addr + COLS_PER_TILE + x * 64 + cc * 32, ob);
+          tc_ld32(o_addr + col0, oa);
+          if (two) tc_ld32(o_addr + COLS_PER_TILE + col0, ob);
           tc_wait_ld();
           float y[32];
 #pragma unroll
@@ -601,7 +725,7 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
               pk.y = tc_pack(y[i + 2], y[i + 3]);
               pk.z = tc_pack(y[i + 4], y[i + 5]);
               pk.w = tc_pack(y[i + 6], y[i + 7]);
-              *reinterpret_cast<uint4*>(dst + cc * 32 + i) = pk;
+              if (VN == VD || col0 + i < VD) *reinterpret_cast<uint4*>(dst + col0 + i) = pk;
             }
           }
         }
@@ -626,37 +750,51 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
 
 
 // ---------------------------------------------------------------------------------------------------
-// qkv [n_tokens, row_stride] bfloat16 (the q heads are the first nq * 128 columns), pages [num_pages, 2, nkv, page_size, 128],
-// out [n_tokens, nq * 128].  Takes the requests with q_len * (nq / nkv) > 16.  The group size nq / nkv must divide 128 and
-// page_size must be 16, 32 or 64.  err: a device int that stays 0 unless a bounded wait gave up.
-IFB_EXPORT int ifb_attention_tc(const void* qkv, int row_stride, const void* pages, long long num_pages, const int* block_tables,
-                                int bt_stride, const int* cu_q, const int* seq_lens, void* out, int* err, int n_tokens, int n_req,
-                                int nq, int nkv, int d, int page_size, float scale, int window, int max_q_len,
+// qkv [n_tokens, row_stride] bfloat16 (the q heads are the first nq * d columns), k_pages / v_pages: the two streams, pages
+// k_page_stride / v_page_stride elements apart, num_pages of them, each [kv heads][page_size][d or dv]; out [n_tokens, nq * dv].
+// nkv: groups of query heads (at most 128 each), `share` of which read one key/value head.  Takes the requests with
+// q_len * (nq / nkv) > 16.  page_size must be 16, 32 or 64.  softcap: 0 none (a library compiled with SOFTCAP takes a positive
+// one of at most 60 and no other takes one).  has_sink: exp(sink) joins the denominators (with SOFTCAP, sink at most 60).
+// err: a device int that stays 0 unless a bounded wait gave up.
+IFB_EXPORT int ifb_attention_tc(const void* qkv, int row_stride, const void* k_pages, long long k_page_stride, const void* v_pages,
+                                long long v_page_stride, long long num_pages, const int* block_tables, int bt_stride, const int* cu_q,
+                                const int* seq_lens, void* out, int* err, int n_tokens, int n_req, int nq, int nkv, int share, int d,
+                                int dv, int page_size, float scale, int window, float softcap, int has_sink, float sink, int max_q_len,
                                 cudaStream_t stream) {
   if (n_tokens <= 0 || n_req <= 0) return IFB_OK;
-  if (d != D) return IFB_ERR_SIZE;
-  if (nkv < 1 || nq % nkv || window < 0 || !err) return IFB_ERR_ARG;
-  const int G = nq / nkv;
-  if (G > ROWS || ROWS % G) return IFB_ERR_SIZE;
+  if (d != D || dv != VD) return IFB_ERR_SIZE;
+  if (nkv < 1 || nq % nkv || share < 1 || nkv % share || window < 0 || !err || num_pages < 1) return IFB_ERR_ARG;
+  if (SOFTCAP ? !(softcap > 0.f && softcap <= TC_MAX_CAP) || (has_sink && sink > TC_MAX_CAP) : softcap != 0.f) return IFB_ERR_ARG;
+  const int G = nq / nkv, heads = nkv / share;
+  if (G > ROWS) return IFB_ERR_SIZE;
   if (page_size != 16 && page_size != 32 && page_size != 64) return IFB_ERR_SIZE;
-  if (row_stride % 8 || ((uintptr_t)qkv & 15) || ((uintptr_t)pages & 127) || ((uintptr_t)out & 15)) return IFB_ERR_ALIGN;
-  const long long rows = num_pages * 2 * nkv * page_size;
-  if (rows >= 0x7fffffffLL || n_req > 65535) return IFB_ERR_SIZE;
-  CUtensorMap q_map, kv_map;
+  if (row_stride % 8 || (((uintptr_t)qkv | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)out) & 15)) return IFB_ERR_ALIGN;
+  if (k_page_stride % D || v_page_stride % VD || k_page_stride < (long long)heads * page_size * D ||
+      v_page_stride < (long long)heads * page_size * VD)
+    return IFB_ERR_ARG;
+  const long long k_page = k_page_stride / D, v_page = v_page_stride / VD;
+  const long long k_rows = (num_pages - 1) * k_page + (long long)heads * page_size, v_rows = (num_pages - 1) * v_page + (long long)heads * page_size;
+  if (k_rows >= 0x7fffffffLL || v_rows >= 0x7fffffffLL || n_req > 65535) return IFB_ERR_SIZE;
+  const int tpt = ROWS / G;                                  // tokens per query tile
+  CUtensorMap q_map, k_map, v_map;
   {
     const unsigned long long dims[3] = {(unsigned long long)D, (unsigned long long)nq, (unsigned long long)n_tokens};
     const unsigned long long strides[2] = {(unsigned long long)D * 2, (unsigned long long)row_stride * 2};
-    const unsigned box[3] = {64, (unsigned)G, (unsigned)(ROWS / G)};
+    const unsigned box[3] = {64, (unsigned)G, (unsigned)tpt};
     if (ifb_tensor_map_bf16(&q_map, qkv, 3, dims, strides, box)) return IFB_ERR_ARG;
   }
+  const unsigned box[2] = {64, (unsigned)page_size};
   {
-    const unsigned long long dims[2] = {(unsigned long long)D, (unsigned long long)rows};
+    const unsigned long long dims[2] = {(unsigned long long)D, (unsigned long long)k_rows};
     const unsigned long long strides[1] = {(unsigned long long)D * 2};
-    const unsigned box[2] = {64, (unsigned)page_size};
-    if (ifb_tensor_map_bf16(&kv_map, pages, 2, dims, strides, box)) return IFB_ERR_ARG;
+    if (ifb_tensor_map_bf16(&k_map, k_pages, 2, dims, strides, box)) return IFB_ERR_ARG;
+  }
+  {
+    const unsigned long long dims[2] = {(unsigned long long)VD, (unsigned long long)v_rows};
+    const unsigned long long strides[1] = {(unsigned long long)VD * 2};
+    if (ifb_tensor_map_bf16(&v_map, v_pages, 2, dims, strides, box)) return IFB_ERR_ARG;
   }
   IFB_ALLOW_SMEM(attn_tile_tc_kernel, SMEM_BYTES);
-  const int tpt = ROWS / G;                                  // tokens per query tile
   const long long items = (long long)((max_q_len + tpt - 1) / tpt) * nkv;      // of the longest request
   static int sm_count = 0;
   if (!sm_count) {
@@ -664,7 +802,15 @@ IFB_EXPORT int ifb_attention_tc(const void* qkv, int row_stride, const void* pag
     if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess)
       sm_count = 1;
   }
+  constexpr float LOG2E = 1.4426950408889634f;
+  TcScore score = {scale * LOG2E, 0.f, 0.f, 0.f};
+  if (SOFTCAP) {
+    score.to_y = scale / softcap;
+    score.cap_log2 = softcap * LOG2E;
+    score.limit = scale != 0.f ? TC_TANH_RANGE / fabsf(score.to_y) : INFINITY;
+  }
+  const TcRows rows = {(int)k_page, (int)v_page, (int)k_rows, (int)v_rows};
   dim3 grid((unsigned)(items < sm_count ? items : sm_count), 1, n_req);       // a CTA per SM walks the request's items
-  return ifb_launch(attn_tile_tc_kernel, grid, dim3(TC_THREADS), (size_t)SMEM_BYTES, stream, q_map, kv_map, (int)rows, err, block_tables,
-                    bt_stride, cu_q, seq_lens, (bf16*)out, nq, nkv, page_size, scale * 1.4426950408889634f, window);
+  return ifb_launch(attn_tile_tc_kernel, grid, dim3(TC_THREADS), (size_t)SMEM_BYTES, stream, q_map, k_map, v_map, rows, err, block_tables,
+                    bt_stride, cu_q, seq_lens, (bf16*)out, nq, nkv, share, page_size, score, has_sink ? sink * LOG2E : -INFINITY, window);
 }

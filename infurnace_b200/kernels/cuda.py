@@ -130,7 +130,7 @@ class CudaKernels:
         self._dev_err = torch.zeros(1, dtype=torch.int32, device="cuda")
         self.attention_tma = True      # keys and values by TMA where the sizes allow (else 16-byte async copies)
         self.attention_tc = True       # prompts on tcgen05 where the sizes allow (head size 128, pages of 16/32/64)
-        self._attn_tc = None
+        self._attn_tc = {}             # compile-time variant -> library
         self.tc_attention_calls = 0    # launches of the tcgen05 attention kernel, of the small-q kernel, and of the latter
         self.small_q_calls = 0         # with keys and values by TMA (what ran is what tests of the product path ask)
         self.small_q_tma_calls = 0
@@ -585,21 +585,43 @@ class CudaKernels:
             block_tables.stride(0), cu_q.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), n, r, num_heads,
             num_kv_heads, head_dim, kv_pages.shape[3], float(scale), int(window), self._stream()), "paged_attention")
 
-    def _attention_tc(self, qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q, seq_lens, out, scale,
-                      window, max_q_len, n, r):
-        if self._attn_tc is None:
-            self._attn_tc = load_library("attention_tc", progress=self._progress)
-            self._attn_tc.ifb_attention_tc.argtypes = [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
-                                                       c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                                       c_int, c_int, c_void_p]
+    def _attention_tc_library(self, head_dim, weight_terms, value_head_dim, softcap):
+        defines = self.attention_defines(head_dim, weight_terms, value_head_dim, softcap)
+        if defines == {"HEAD_DIM": 128}:
+            defines = {}                                   # the library's own defaults
+        key = tuple(sorted(defines.items()))
+        lib = self._attn_tc.get(key)
+        if lib is None:
+            lib = self._attn_tc[key] = load_library("attention_tc", defines or None, progress=self._progress)
+            lib.ifb_attention_tc.argtypes = [
+                c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int, c_float, c_int, c_void_p]
+        return lib
+
+    TC_CAP_LIMIT = 60.0       # soft caps (and sinks beside them) up to here: 2^(cap log2 e) summed over any context is a float32 number
+
+    def _attention_tc_fits(self, head_dim, value_head_dim, page_size, group, weight_terms, softcap, sink, one_tensor):
+        """Whether prompts of these sizes run on the tcgen05 attention kernel: plain attention with heads of 128 in one tensor
+        and one-term weights, or capped scores over streams of any widths that its tiles hold."""
+        if not self.attention_tc or page_size not in (16, 32, 64):
+            return False
+        if softcap:
+            return (head_dim % 16 == 0 and head_dim <= 192 and value_head_dim % 16 == 0 and value_head_dim <= 128 and group <= 128
+                    and softcap <= self.TC_CAP_LIMIT and (sink is None or sink <= self.TC_CAP_LIMIT))
+        return (one_tensor is not None and weight_terms == 1 and sink is None and head_dim == 128 and 128 % group == 0
+                and one_tensor.data_ptr() % 128 == 0)
+
+    def _attention_tc_streams(self, qkv, num_heads, num_kv_heads, share, head_dim, value_head_dim, k, v, num_pages, block_tables, cu_q,
+                              seq_lens, out, scale, window, max_q_len, n, r, weight_terms, softcap, sink):
         self._err_armed = True
         self.launches += 1
         self.tc_attention_calls += 1
-        _check(self._attn_tc.ifb_attention_tc(
-            qkv.data_ptr(), qkv.stride(0), kv_pages.data_ptr(), kv_pages.shape[0], block_tables.data_ptr(),
-            block_tables.stride(0), cu_q.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), self._dev_err.data_ptr(), n, r,
-            num_heads, num_kv_heads, head_dim, kv_pages.shape[3], float(scale), int(window), int(max_q_len), self._stream()),
-            "paged_attention")
+        lib = self._attention_tc_library(head_dim, weight_terms, value_head_dim, bool(softcap))
+        _check(lib.ifb_attention_tc(
+            qkv.data_ptr(), qkv.stride(0), k[0], k[1], v[0], v[1], num_pages, block_tables.data_ptr(), block_tables.stride(0),
+            cu_q.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), self._dev_err.data_ptr(), n, r, num_heads, num_kv_heads, share,
+            head_dim, value_head_dim, k[2], float(scale), int(window), float(softcap or 0.0), 0 if sink is None else 1,
+            float(sink or 0.0), int(max_q_len), self._stream()), "paged_attention")
 
     @staticmethod
     def attention_defines(head_dim, weight_terms=1, value_head_dim=None, softcap=False):
@@ -668,7 +690,7 @@ class CudaKernels:
         """The tensor-core attention kernels over key and value streams ``k`` and ``v`` = (address, elements between pages, page
         size).  ``one_tensor``: the tensor that holds both, where there is one (what the tcgen05 kernel for plain attention takes)."""
         share = self.attention_share(num_heads // num_kv_heads)
-        real_kv, num_kv_heads = num_kv_heads, num_kv_heads * share           # groups of query heads from here on
+        num_kv_heads = num_kv_heads * share           # groups of query heads from here on
         lib = self.attention_library(head_dim, weight_terms, value_head_dim, bool(softcap))
         group = num_heads // num_kv_heads
         page_size = k[2]
@@ -685,12 +707,9 @@ class CudaKernels:
                 self._attn_counters = torch.zeros(max(r * num_kv_heads, 4096), dtype=torch.int32, device="cuda")
                 self.scratch_generation += 1
             counters = self._attn_counters
-        use_tc = (not only_small and self.attention_tc and one_tensor is not None and share == 1 and weight_terms == 1 and not softcap
-                  and sink is None and head_dim == 128 and 128 % group == 0 and page_size in (16, 32, 64)
-                  and one_tensor.data_ptr() % 128 == 0)
-        if use_tc:
-            self._attention_tc(qkv, num_heads, num_kv_heads, head_dim, one_tensor, block_tables, cu_q, seq_lens, out, scale,
-                               window, max_q_len, n, r)
+        if not only_small and self._attention_tc_fits(head_dim, value_head_dim, page_size, group, weight_terms, softcap, sink, one_tensor):
+            self._attention_tc_streams(qkv, num_heads, num_kv_heads, share, head_dim, value_head_dim, k, v, num_pages, block_tables, cu_q,
+                                       seq_lens, out, scale, window, max_q_len, n, r, weight_terms, softcap, sink)
             if min_q_len * group > 16:
                 return                 # no request of this step is left for the small-q kernel
             only_small = True          # the tile kernel's requests are done; the small-q kernel takes the rest
