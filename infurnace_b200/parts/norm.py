@@ -69,6 +69,10 @@ class GroupRMSNorm:
         self.k = runtime.kernels
 
     def forward(self, x, out, delta=None, rows=None, mult=1.0, keep=None):
+        if delta is not None and delta.dim() == 3:       # several results side by side (a block whose sublayers run in parallel)
+            for other in delta[1:]:
+                self.k.scaled_sum(delta[0], other, 1.0)
+            delta = delta[0]
         self.k.group_rmsnorm(x, self.weight, self.spec.groups, self.spec.eps, out, delta=delta, mult=mult, rows=rows, keep=keep)
         return out
 

@@ -47,11 +47,11 @@ def sink_attention(q, k, v, scale, cap):
     """q [T, H, d], k [T, G, d], v [T, G, dv]: query head h reads key/value head h // (H / G), position i every j <= i."""
     T, H, G = q.shape[0], q.shape[1], k.shape[1]
     out = torch.zeros(T, H, v.shape[2], dtype=F64)
+    later = torch.ones(T, T).triu(1).bool()
     for h in range(H):
         g = h // (H // G)
-        for i in range(T):
-            s = capped((k[:i + 1, g] @ q[i, h]) * scale, cap)
-            out[i, h] = attention_weights(s) @ v[:i + 1, g]
+        s = capped((q[:, h] @ k[:, g].T) * scale, cap).masked_fill(later, -float("inf"))
+        out[:, h] = attention_weights(s) @ v[:, g]
     return out
 
 
@@ -120,7 +120,7 @@ def forward(cfg, weights, tokens, return_layers=False):
     """Logits [T, vocab] of one sequence from its first token (and the stream after every layer)."""
     eps = float(cfg["norm"]["eps"])
     ids = torch.as_tensor(tokens, dtype=torch.long)
-    x = w64(weights, "embed")[ids] * float(cfg["embedding"]["scale"])
+    x = w64(weights, "embed")[ids] * float((cfg.get("embedding") or {}).get("scale", 1.0))
     after, held = [], {}
     for i, layer in enumerate(cfg["layers"]):
         p, m = f"l{i}.", layer["mixer"]
@@ -135,7 +135,7 @@ def forward(cfg, weights, tokens, return_layers=False):
             y = y + feed_forward(h, weights, p + "mlp.", layer["mlp"])
         x = x + y
         after.append(x)
-    logits = rms_norm(x, w64(weights, "final.norm"), eps) @ w64(weights, "head").T * float(cfg["logit_scale"])
+    logits = rms_norm(x, w64(weights, "final.norm"), eps) @ w64(weights, "head").T * float(cfg.get("logit_scale", 1.0))
     return (logits, torch.stack(after)) if return_layers else logits
 
 
