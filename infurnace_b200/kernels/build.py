@@ -50,6 +50,8 @@ LIBRARIES: Dict[str, tuple] = {
 # what the build check compiles beside "core": the head size of the Qwen3 checkpoints and those of
 # the tiny test models; any other multiple of 16 up to 256 is compiled when a model first needs it
 DEFAULT_VARIANTS = [("attention_mma", {"HEAD_DIM": d}) for d in (128, 16, 32, 48)]
+# capped scores with two-term weights, heads of 128: decoding and prompts
+DEFAULT_VARIANTS += [(name, {"HEAD_DIM": 128, "WEIGHT_TERMS": 2, "SOFTCAP": 1}) for name in ("attention_mma", "attention_tc")]
 
 def register_library(name: str, sources: Sequence[str], flags: Sequence[str] = (), *, replace: bool = False) -> None:
     """Make a library of CUDA sources from outside the package known to :func:`load_library`, so that a
