@@ -687,6 +687,29 @@ def recurrent_config(size):
             "token_side": {"dim": 32}, "logit_softcap": 30.0}
 
 
+def parallel_config(size):
+    """A Mubutar config.json mapping at the width, depth, head sizes and ACTIVE parameter count of design_configs(size):
+    layers with keys and values of their own and a gated dense feed-forward (two thirds of that width: gate, up and down
+    against up and down) alternate with layers that read the layer before and have 8 ungated experts in 4 groups of which 2
+    are kept and 2 experts run, each a quarter of that width, beside a shared expert of half of it; cap 50."""
+    W, layers, H, G, d, _, _, _, ff, _ = {
+        "s": (1024, 8, 16, 4, 64, 8, 64, 128, 3072, 512),
+        "m": (2048, 8, 16, 4, 128, 16, 64, 128, 6144, 1024),
+        "l": (4096, 8, 32, 8, 128, 32, 64, 128, 12288, 1024),
+    }[size]
+    entries = []
+    for i in range(layers):
+        mixer = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 50.0}
+        mlp = {"kind": "dense", "ff": ff * 2 // 3}
+        if i % 2:
+            mixer["kv_from"] = i - 1
+            mlp = {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 2},
+                   "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}}
+        entries.append({"type": "attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Mubutar", "embedding": {"scale": W ** 0.5}, "layers": entries, "logit_scale": 0.5,
+            "norm": {"eps": 1e-6}, "vocab": 32768, "width": W}
+
+
 def window_pairs(window, positions):
     """Sum over query positions of the keys each sees under a sliding window."""
     return sum(min(p + 1, window) for p in positions)
@@ -721,7 +744,7 @@ class DesignTimer(KernelClassTimer):
                                           "rotate_rows", "paged_attention_streams", "moe_route", "moe_plan", "moe_linear",
                                           "moe_combine", "moe_plan_padded", "moe_gather", "moe_linear_grouped", "moe_route_plan",
                                           "group_rmsnorm", "depth_average", "causal_conv", "latent_prepare", "latent_attention",
-                                          "gate_heads", "rglru_conv", "rglru_scan", "moe_gather_scaled")
+                                          "gate_heads", "rglru_conv", "rglru_scan", "moe_gather_scaled", "moe_combine_update")
 
     def __init__(self, kernels, vocab, pairs, key_bytes, positions=(), head_weights=()):
         super().__init__(kernels, vocab)
@@ -839,6 +862,8 @@ def run_designs(args):
             pair = (("filorax", latent_config(size)), ("lunelorn", hybrid_config(size)))
         if args.recurrent:
             pair = (("golonex", recurrent_config(size)), ("lunelorn", hybrid_config(size)))
+        if args.parallel:            # the closest in attention and dense products, and the closest in experts
+            pair = (("mubutar", parallel_config(size)), ("qwen3", qwen), ("lunelorn", hybrid_config(size)))
         for design, conf in pair:
             pool = batch * (context + 64) + PREFILL_TOKENS + 64
             opts = EngineOptions(dtype="bfloat16", page_size=16, num_pages=pool // 16, max_num_seqs=batch,
@@ -1062,6 +1087,87 @@ def time_hybrid_kernels(args):
     return 0
 
 
+def time_parallel_kernels(args):
+    """Mubutar's own kernels alone beside their likes, on tensors made on the device at the sizes of parallel_config: attention
+    with capped scores, a sink and two-term weights beside the plain attention of the same heads (a 2,048-token and an
+    8,192-token prompt, a decode step of 8 requests 2,040 tokens in), the corrected router within groups beside the softmax router, and the
+    combination that updates the stream and forms the next norm beside combination and norm apart.  Microseconds by CUDA
+    events, the median of 20 calls with L2 flushed between them; one JSON line.  (--design-sizes m: a profiler's small case.)"""
+    import torch
+    from infurnace_b200.kernels import load_cuda_kernels
+    K = load_cuda_kernels()
+    hbm_peak, tc_peak, peak_src = read_peaks()
+    g = torch.Generator(device="cuda").manual_seed(1)
+    flush = torch.empty(64 << 20, dtype=torch.float32, device="cuda")
+
+    def timed(f, reps=20):
+        times = []
+        for i in range(reps + 3):
+            flush.zero_()
+            s, e = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            s.record()
+            f()
+            e.record()
+            torch.cuda.synchronize()
+            times.append(s.elapsed_time(e) * 1e3)
+        return round(statistics.median(times[3:]), 1)
+
+    def randn(*shape, dtype=torch.float32):
+        return torch.randn(*shape, device="cuda", generator=g).to(dtype)
+
+    def attention(H, G, d, tokens, requests, past, capped, ps=16):
+        n, L = tokens * requests, past + tokens
+        maxp = -(-L // ps)
+        pages = randn(requests * maxp + 1, 2, G, ps, d, dtype=torch.bfloat16)
+        bt = torch.arange(requests * maxp, dtype=torch.int32, device="cuda").view(requests, maxp).contiguous()
+        cu = torch.arange(requests + 1, dtype=torch.int32, device="cuda") * tokens
+        seq = torch.full((requests,), L, dtype=torch.int32, device="cuda")
+        q, out = randn(n, H * d, dtype=torch.bfloat16), torch.empty(n, H * d, dtype=torch.bfloat16, device="cuda")
+        if capped:
+            us = timed(lambda: K.paged_attention_streams(q, H, G, d, d, pages[:, 0], pages[:, 1], bt, cu, seq, out, d ** -0.5, 0, None, False,
+                                                         max_q_len=tokens, max_seq_len=L, min_q_len=tokens, softcap=50.0, sink=0.0,
+                                                         weight_terms=2, exact=False))
+        else:
+            us = timed(lambda: K.paged_attention(q, H, G, d, pages, bt, cu, seq, out, d ** -0.5, 0, tokens, L, min_q_len=tokens))
+        pairs = requests * sum(past + t + 1 for t in range(tokens))
+        bound = max(4 * H * d * pairs / (tc_peak * 1e6), 4 * requests * L * G * d / (hbm_peak * 1e3))
+        return {"us": us, "of_bound": round(bound / us, 3)}
+
+    def routers(n, E=8, top=2):
+        z, c = 2 * randn(n, E), 0.3 * randn(E)
+        ids, gates = torch.zeros(n, top, dtype=torch.int32, device="cuda"), torch.zeros(n, top, device="cuda")
+        return {"corrected_us": timed(lambda: K.moe_route(z, top, ids, gates, scoring="sigmoid", groups=(4, 2), correction=c, normalise=True, group_best=2)),
+                "softmax_us": timed(lambda: K.moe_route(z, top, ids, gates, scoring="all", groups=(4, 2)))}
+
+    def combinations(n, W, top=2):
+        y, pos = randn(n * top, W), torch.randperm(n * top, device="cuda", generator=g).to(torch.int32)
+        gates, x, base, shared, w = randn(n, top), randn(n, W), randn(n, W), randn(n, W), randn(W)
+        out, delta = torch.empty(n, W, dtype=torch.bfloat16, device="cuda"), torch.empty(n, W, device="cuda")
+
+        def apart():
+            K.moe_combine(y, pos, gates, delta, shared)
+            K.rmsnorm(x, w, 1e-6, out, delta=delta)
+        one = timed(lambda: K.moe_combine_update(y, pos, gates, x, base=base, shared=shared, out=out, next_weight=w, eps=1e-6))
+        least = n * W * (4 * top + 4 * 4 + 2)
+        return {"one_us": one, "one_of_bound": round(least / hbm_peak / 1e3 / one, 3), "apart_us": timed(apart)}
+
+    sizes = {}
+    for size in args.design_sizes.split(","):
+        conf = parallel_config(size)
+        m, W = conf["layers"][0]["mixer"], conf["width"]
+        att = (m["heads"], m["kv_heads"], m["dim"])
+        sizes[size] = {"attention": {kind: {"prompt_2048": attention(*att, PREFILL_TOKENS, 1, 0, capped),
+                                            "prompt_8192": attention(*att, 4 * PREFILL_TOKENS, 1, 0, capped),
+                                            "decode_b8": attention(*att, 1, 8, 2040, capped)}
+                                     for kind, capped in (("capped", True), ("plain", False))},
+                       "router": {"prompt": routers(PREFILL_TOKENS), "decode_b8": routers(8)},
+                       "combination": {"prompt": combinations(PREFILL_TOKENS, W), "decode_b8": combinations(8, W)}}
+    K.check_device_errors()
+    print(json.dumps({"metric": "parallel_kernels_alone", "dtype": "bfloat16 operands", "unit": "us", "sizes": sizes,
+                      "peaks": {"hbm_gbs": hbm_peak, "tensor_tflops": tc_peak, "source": peak_src}}))
+    return 0
+
+
 def time_recurrent_kernels(args):
     """The real-gated recurrence's kernels each alone (its convolution, the block-diagonal gate product, the walk), beside
     the element-wise recurrence of the closest design (minGRU) and the framework's other short convolution (the one in
@@ -1166,6 +1272,8 @@ def main():
                     help="with --designs: the Filorax design beside Lunelorn (equal width, depth and active parameters)")
     ap.add_argument("--recurrent", action="store_true",
                     help="with --designs: the Golonex design beside Lunelorn (equal width, depth and active parameters)")
+    ap.add_argument("--parallel", action="store_true",
+                    help="with --designs: the Mubutar design beside Qwen3 and Lunelorn (equal width, depth and active parameters)")
     ap.add_argument("--design-sizes", default="s,m", help="with --designs: which of the sizes s, m, l (commas between)")
     ap.add_argument("--kernels-alone", action="store_true",
                     help="with --designs: only the talking attention and the gated recurrence, each alone (a small case)")
@@ -1181,6 +1289,8 @@ def main():
     args.warmup = max(3, args.warmup)
     if args.designs:
         if args.kernels_alone:
+            if args.parallel:
+                return time_parallel_kernels(args)
             if args.recurrent:
                 return time_recurrent_kernels(args)
             return time_hybrid_kernels(args) if args.hybrid else time_design_kernels(args)
