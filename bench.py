@@ -691,7 +691,7 @@ def parallel_config(size):
     """A Mubutar config.json mapping at the width, depth, head sizes and ACTIVE parameter count of design_configs(size):
     layers with keys and values of their own and a gated dense feed-forward (two thirds of that width: gate, up and down
     against up and down) alternate with layers that read the layer before and have 8 ungated experts in 4 groups of which 2
-    are kept and 2 experts run, each a quarter of that width, beside a shared expert of half of it; cap 50."""
+    are kept and 2 experts run, each a quarter of that width, beside a shared expert of half of it; cap 40."""
     W, layers, H, G, d, _, _, _, ff, _ = {
         "s": (1024, 8, 16, 4, 64, 8, 64, 128, 3072, 512),
         "m": (2048, 8, 16, 4, 128, 16, 64, 128, 6144, 1024),
@@ -699,7 +699,7 @@ def parallel_config(size):
     }[size]
     entries = []
     for i in range(layers):
-        mixer = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 50.0}
+        mixer = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 40.0}
         mlp = {"kind": "dense", "ff": ff * 2 // 3}
         if i % 2:
             mixer["kv_from"] = i - 1
@@ -1125,7 +1125,7 @@ def time_parallel_kernels(args):
         q, out = randn(n, H * d, dtype=torch.bfloat16), torch.empty(n, H * d, dtype=torch.bfloat16, device="cuda")
         if capped:
             us = timed(lambda: K.paged_attention_streams(q, H, G, d, d, pages[:, 0], pages[:, 1], bt, cu, seq, out, d ** -0.5, 0, None, False,
-                                                         max_q_len=tokens, max_seq_len=L, min_q_len=tokens, softcap=50.0, sink=0.0,
+                                                         max_q_len=tokens, max_seq_len=L, min_q_len=tokens, softcap=40.0, sink=0.0,
                                                          weight_terms=2, exact=False))
         else:
             us = timed(lambda: K.paged_attention(q, H, G, d, pages, bt, cu, seq, out, d ** -0.5, 0, tokens, L, min_q_len=tokens))

@@ -95,14 +95,17 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 // What stands between a product q . k and the exponent of its weight: SOFTCAP 0: `a` = scale * log2(e), s * a.  SOFTCAP 1:
-// the capped score c tanh(scale s / c) in the base-2 domain, `a` = c log2(e), `b` = 2 scale log2(e) / c:
-// a (1 - 2 / (1 + 2^(b s))), whose absolute error is a few 2^-23 of a (exact at both ends: 2^(b s) may be 0 or infinite).
-struct AttScale { float a, b; };
+// the capped score c tanh(y), y = `y` s = scale s / c, in the base-2 domain: `a` = c log2(e) times the polynomial of
+// attention_tc.cu where |y| <= 0.7 (so that scores far below a large cap keep their accuracy), else 1 - 2 / (1 + 2^(b s)),
+// `b` = 2 y log2(e) (right at both ends: 2^(b s) may be 0 or infinite).
+struct AttScale { float a, b, y; };
 __device__ __forceinline__ float att_score(float s, const AttScale& sc) {
 #if SOFTCAP
+  const float y = s * sc.y, u = y * y;
+  const float small = y * fmaf(u, fmaf(u, fmaf(u, fmaf(u, 0.01359966f, -0.05067464f), 0.13276916f), -0.33330065f), 1.f);
   float r;
   asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.f + fast_exp2(s * sc.b)));
-  return fmaf(-2.f * sc.a, r, sc.a);
+  return sc.a * (u <= 0.49f ? small : fmaf(-2.f, r, 1.f));
 #else
   return s * sc.a;
 #endif
@@ -911,7 +914,7 @@ IFB_EXPORT int ifb_attention_mma(const void* qkv, int row_stride, const void* k_
   a.seq_lens = seq_lens; a.out = out; a.scratch = scratch; a.counters = counters; a.n_tokens = n_tokens; a.n_req = n_req; a.nq = nq;
   a.nkv = nkv; a.share = share; a.page_size = page_size; a.window = window; a.max_q_len = max_q_len; a.num_splits = num_splits;
   a.run_small = run_small; a.run_tiles = run_tiles;
-  a.sc = SOFTCAP ? AttScale{softcap * LOG2E, 2.f * scale * LOG2E / softcap} : AttScale{scale * LOG2E, 0.f};
+  a.sc = SOFTCAP ? AttScale{softcap * LOG2E, 2.f * scale * LOG2E / softcap, scale / softcap} : AttScale{scale * LOG2E, 0.f, 0.f};
   a.sink = has_sink ? sink * LOG2E : -INFINITY;
   const long long k_page = k_page_stride / D, v_page = v_page_stride / VD;
   const long long k_rows = (num_pages - 1) * k_page + (long long)heads * page_size, v_rows = (num_pages - 1) * v_page + (long long)heads * page_size;

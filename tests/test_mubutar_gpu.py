@@ -171,7 +171,7 @@ def test_capped_attention_with_a_sink(K, dtype, H, G, D, VD):
     g = gen(H * 1000 + D + VD)
     lens_new, lens_old = [37, 1, 150, 3, 2], [0, 100, 60, 17, 64]
     for ps, cap, sink, spread, uniform in ((16, 4.0, 0.0, 4.0, False), (32, 30.0, 0.0, 1.0, True), (64, 20.0, 2.5, 12.0, False), (16, 55.0, None, 30.0, False),
-                                           (8, 5.0, -3.0, 3.0, False), (16, None, 0.0, 2.0, False), (16, 500.0, 0.0, 3.0, False)):
+                                           (8, 5.0, -3.0, 3.0, False), (16, None, 0.0, 2.0, False), (16, 1e6, 0.0, 3.0, False)):
         uniform = uniform and D == VD
         if cap is None and (D, VD) not in PLAIN and D % 16 == 0:
             continue
