@@ -34,7 +34,7 @@ LIBRARIES: Dict[str, tuple] = {
     "linear_tcgen05": (["linear_tcgen05.cu"], []),
     # the few-rows product with its scratch inside the library, for callers that must not allocate
     "linear_skinny_static": (["linear_skinny_static.cu"], []),
-    "attention_tc": (["attention_tc.cu"], []),            # head size 128
+    "attention_tc": (["attention_tc.cu"], []),            # heads of 128, or defines={"HEAD_DIM": d, "VALUE_DIM": v, ...}
     # post-norm sublayers (embedding with a position vector, residual update), the gated recurrence, talking attention
     "mixers": (["sublayer.cu", "gated_scan.cu", "attention_talk.cu", "attention_talk_mma.cu"], []),
     # sandwich-norm blocks, recurrences over a matrix state or an element-wise one, attention with rotated values over

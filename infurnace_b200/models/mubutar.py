@@ -3,7 +3,7 @@
 A decoder over a float32 residual stream whose layers have one norm each: h = norm1(x), x += mixer(h) + ff(h), both
 sublayers reading the same h.  The embedding's rows and the logits are multiplied by one number each.  The mixer is
 grouped-query attention without positions: q, k and v with biases, keys and values of different widths, scores capped
-(c * tanh(s / c)), one added to the softmax's denominator; a layer may have queries only and read the keys and values of an
+(c * tanh(s / c)), exp(0) beside the keys in the softmax's denominator; a layer may have queries only and read the keys and values of an
 earlier layer (its layer call then names that layer's cache entry and stores nothing).  The feed-forward is a gated silu
 one, or a mixture of ungated relu² experts: sigmoid scores, chosen by score plus a correction within the best groups of
 neighbouring experts (a group counts by its two best), weighted by the chosen scores over their sum, beside a shared expert
@@ -23,7 +23,7 @@ from .registry import register_architecture
 MAX_POSITIONS = 1 << 20        # positions have no end in this design; block tables need one
 DENSE_ACTIVATION = "silu"
 EXPERT_ACTIVATION = "relu2"
-SINK_SCORE = 0.0               # the softmax's denominator is 1 + the sum: a sink whose score is 0
+SINK_SCORE = 0.0               # exp(0) joins the softmax's denominator
 GROUP_BEST = 2                 # a group of experts counts by the sum of its two best choice scores
 WEIGHT_TERMS = 2               # softmax weights are 32-bit in this design: on tensor cores they enter the sum as two terms
 

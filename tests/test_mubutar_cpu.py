@@ -42,7 +42,7 @@ def tolerance(ref):
 # ------------------------------------------------------------------------------ each mechanism of the oracle alone
 def test_the_oracles_mechanisms_alone():
     f64 = torch.float64
-    # one is added to the denominator: n equal scores of 0 get 1 / (n + 1) each; far below 0 nothing is left for the keys
+    # the sink stands beside the keys: n equal scores of 0 get 1 / (n + 1) each; far below 0 nothing is left for the keys
     assert torch.allclose(P.attention_weights(torch.zeros(3, dtype=f64)), torch.full((3,), 0.25, dtype=f64))
     assert float(P.attention_weights(torch.full((3,), -40.0, dtype=f64)).sum()) < 1e-15
     assert torch.allclose(P.attention_weights(torch.tensor([500.0, 0.0], dtype=f64)), torch.tensor([1.0, 0.0], dtype=f64))
@@ -66,7 +66,7 @@ def test_the_oracles_mechanisms_alone():
     # a group counts by the sum of its two best: the group of the single best expert loses
     z = torch.tensor([[4.0, -4.0, -4.0, 1.0, 1.0, -4.0]], dtype=f64)
     assert P.route(z, torch.zeros(6, dtype=f64), 2, (2, 1))[0].tolist() == [[3, 4]]
-    # experts of the other groups count as minus infinity, not as 0: every choice score is negative here
+    # nothing of the other groups is ever chosen, also where every score left is below zero
     assert set(P.route(z, torch.full((6,), -3.0, dtype=f64), 3, (2, 1))[0][0].tolist()) == {3, 4, 5}
     # a group of one expert counts by it; the lower index wins among equals
     assert P.route(torch.zeros(1, 4, dtype=f64), torch.zeros(4, dtype=f64), 2, (4, 2))[0].tolist() == [[0, 1]]
