@@ -34,7 +34,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
 
-from ..config.specs import KVCacheNeed, ModelPlan, PagedCacheNeed, StateNeed
+from ..config.specs import EMBEDDING_CACHE, KVCacheNeed, ModelPlan, PagedCacheNeed, StateNeed
 from ..errors import CacheError, OutOfPages
 from .block_pool import BlockPool
 
@@ -82,6 +82,9 @@ class CacheLayout:
         self.kv: Dict[tuple, Tuple[KVCacheNeed, List[int]]] = {}
         self.state: Dict[tuple, Tuple[StateNeed, List[int]]] = {}
         self.group_of: Dict[int, tuple] = {}
+        embedding_need = getattr(plan.embedding, "cache_need", None)
+        if embedding_need is not None:
+            self._enter(EMBEDDING_CACHE, embedding_need())
         for call in plan.resolved_schedule():
             self._enter(call.cache, plan.layers[call.layer].cache_need())
 

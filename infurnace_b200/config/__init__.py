@@ -6,7 +6,7 @@ from .specs import (  # noqa: F401
     NormedEmbeddingSpec, StreamInjectSpec, RetentionSpec, TimeMixSpec, GatedUnitSpec, RotaryValueAttentionSpec,
     ParallelMixerSpec, RoutedExpertsSpec, TokenSideSpec, SandwichBlockSpec,
     PagedStream, PagedCacheNeed, GroupRMSNormSpec, CausalConvSpec, LatentAttentionSpec, DepthAverageBlockSpec,
-    RealGatedRecurrenceSpec, ParallelBlockSpec,
+    RealGatedRecurrenceSpec, ParallelBlockSpec, BigramEmbeddingSpec, DeltaRuleSpec, EMBEDDING_CACHE,
 )
 from .qwen3 import Qwen3Config  # noqa: F401
 from .kafunex import KafunexConfig  # noqa: F401
@@ -14,3 +14,4 @@ from .lunelorn import LunelornConfig  # noqa: F401
 from .filorax import FiloraxConfig  # noqa: F401
 from .golonex import GolonexConfig  # noqa: F401
 from .mubutar import MubutarConfig  # noqa: F401
+from .tigelorn import TigelornConfig  # noqa: F401

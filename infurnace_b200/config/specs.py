@@ -104,14 +104,16 @@ class StateNeed:
 # --------------------------------------------------------------------------- parts
 @dataclass(frozen=True)
 class RMSNormSpec:
-    """y = x * rsqrt(mean(x^2) + eps) * weight, statistics in 32-bit
-    (src/infurnace/executor/tinygrad/model.py:11-13)."""
+    """y = x * rsqrt(mean(x^2) + eps) * (offset + weight), statistics in 32-bit
+    (src/infurnace/executor/tinygrad/model.py:11-13, where there is no offset).  ``offset`` 1: the weight is stored around
+    zero."""
     size: int
     eps: float
     weight: str  # tensor name
+    offset: float = 0.0
 
     def tensors(self) -> Mapping[str, TensorSpec]:
-        return {self.weight: TensorSpec((self.size,))}
+        return {self.weight: TensorSpec((self.size,), init=(1.0 - self.offset, 0.1) if self.offset else None)}
 
 
 @dataclass(frozen=True)
@@ -181,7 +183,7 @@ class AttentionSpec:
 @dataclass(frozen=True)
 class GatedMLPSpec:
     """x -> down(act(gate(x)) * up(x)), no bias (model.py:146-148).  ``activation``
-    names the gate's function; "silu" is z * sigmoid(z)."""
+    names the gate's function: "silu" is z * sigmoid(z), "gelu_tanh" the tanh form of gelu."""
     hidden_size: int
     intermediate_size: int
     activation: str
@@ -235,6 +237,30 @@ class EmbeddingSpec:
 
     def tensors(self) -> Mapping[str, TensorSpec]:
         return {self.weight: TensorSpec((self.vocab_size, self.hidden_size))}
+
+
+EMBEDDING_CACHE = "embedding"       # id of the cache entry of an embedding that keeps state
+
+
+@dataclass(frozen=True)
+class BigramEmbeddingSpec:
+    """x[t] = table[id_t] + pairs[row_t] in float32.  row_t = (id_(t-1) * mul_prev + id_t * mul_cur) mod buckets; the first
+    token of a sequence takes row number ``buckets``, the last of the pair table [buckets + 1, hidden].  The previous token
+    is state: one number per sequence, in the cache entry ``EMBEDDING_CACHE``."""
+    vocab_size: int
+    hidden_size: int
+    weight: str
+    pairs: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+    def tensors(self) -> Mapping[str, TensorSpec]:
+        return {self.weight: TensorSpec((self.vocab_size, self.hidden_size)),
+                self.pairs: TensorSpec((self.buckets + 1, self.hidden_size))}
+
+    def cache_need(self):
+        return StateNeed((1,))
 
 
 @dataclass(frozen=True)
@@ -457,7 +483,11 @@ class RetentionSpec:
     """Linear attention with one fixed decay per head, no softmax and no denominator.  Per head a float32 state
     S [dim, vdim], zero at the start of a sequence: S <- decay_h S + (k * key_scale) v^T, o = S^T q.  Each head's o
     is divided by its root mean square (no weight), the heads side by side are multiplied by silu(G h) and go
-    through ``o_proj``."""
+    through ``o_proj``.
+
+    ``input_activation`` "silu": q, k and v are silu of their projections.  ``joint_norm`` names a weight [heads * vdim]:
+    all heads side by side are divided by ONE root mean square and multiplied by it, in the place of the norm per head.
+    ``gate_activation``: the function on G h, "silu" or "sigmoid"."""
     hidden_size: int
     num_heads: int
     head_dim: int
@@ -470,12 +500,18 @@ class RetentionSpec:
     v_proj: str
     g_proj: str
     o_proj: str
+    input_activation: Optional[str] = None
+    joint_norm: Optional[str] = None
+    gate_activation: str = "silu"
 
     def tensors(self) -> Mapping[str, TensorSpec]:
         hd, hv = self.num_heads * self.head_dim, self.num_heads * self.value_head_dim
-        return {self.q_proj: TensorSpec((hd, self.hidden_size)), self.k_proj: TensorSpec((hd, self.hidden_size)),
-                self.v_proj: TensorSpec((hv, self.hidden_size)), self.g_proj: TensorSpec((hv, self.hidden_size)),
-                self.o_proj: TensorSpec((self.hidden_size, hv))}
+        t = {self.q_proj: TensorSpec((hd, self.hidden_size)), self.k_proj: TensorSpec((hd, self.hidden_size)),
+             self.v_proj: TensorSpec((hv, self.hidden_size)), self.g_proj: TensorSpec((hv, self.hidden_size)),
+             self.o_proj: TensorSpec((self.hidden_size, hv))}
+        if self.joint_norm is not None:
+            t[self.joint_norm] = TensorSpec((hv,))
+        return t
 
     def cache_need(self):
         return StateNeed((self.num_heads, self.head_dim, self.value_head_dim))
@@ -593,6 +629,67 @@ class RealGatedRecurrenceSpec:
 
 
 @dataclass(frozen=True)
+class DeltaRuleSpec:
+    """The gated delta rule with a decay per key channel.  q = conv(Q h), k = conv(K h) (``num_kv_heads`` heads of
+    ``head_dim``), v = conv(V h) (``num_heads`` of ``value_head_dim``), each through a causal convolution per channel over time
+    (tensor [channels, taps], the last column is the current token's, zeros before the start) and then silu; head h
+    uses q/k head floor(h / (num_heads / num_kv_heads)).  q and k are divided by sqrt(sum(x^2) + ``unit_eps``) per head, q
+    is multiplied by head_dim^(-1/2).  beta = sigmoid(B h), one number per head.
+    g = exp(-exp(``a_log``_head) * softplus(``decay_up`` ``decay_down`` h + ``decay_bias``)) per head and key channel.
+    Per head a float32 state S [head_dim, value_head_dim] from zero: S <- diag(g) S; u = beta * (v - S^T k);
+    S <- S + k u^T; o = S^T q.  Each head's o is divided by its root mean square, times ``out_norm`` [value_head_dim]
+    (shared by the heads), times sigmoid(``gate_up`` ``gate_down`` h); then ``o_proj``.  The convolutions' last taps - 1
+    inputs are state too.  ``rank`` (the width of the two bottlenecks) None: the stored tensors give it."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_head_dim: int
+    taps: int
+    eps: float
+    q_proj: str
+    k_proj: str
+    v_proj: str
+    q_conv: str
+    k_conv: str
+    v_conv: str
+    beta_proj: str
+    a_log: str
+    decay_down: str
+    decay_up: str
+    decay_bias: str
+    gate_down: str
+    gate_up: str
+    out_norm: str
+    o_proj: str
+    unit_eps: float = 1e-6
+    rank: Optional[int] = None
+
+    @property
+    def channels(self) -> int:
+        return 2 * self.num_kv_heads * self.head_dim + self.num_heads * self.value_head_dim
+
+    def tensors(self) -> Mapping[str, TensorSpec]:
+        W, H = self.hidden_size, self.num_heads
+        kd, hd, hv = self.num_kv_heads * self.head_dim, H * self.head_dim, H * self.value_head_dim
+        taps = {"init": (0.0, 0.4)}
+        return {
+            self.q_proj: TensorSpec((kd, W)), self.q_conv: TensorSpec((kd, self.taps), **taps),
+            self.k_proj: TensorSpec((kd, W)), self.k_conv: TensorSpec((kd, self.taps), **taps),
+            self.v_proj: TensorSpec((hv, W)), self.v_conv: TensorSpec((hv, self.taps), **taps),
+            self.beta_proj: TensorSpec((H, W)), self.a_log: TensorSpec((H,), init=(0.0, 1.0)),
+            self.decay_down: TensorSpec((self.rank, W)), self.decay_up: TensorSpec((hd, self.rank)),
+            self.decay_bias: TensorSpec((hd,), init=(-3.0, 1.5)),
+            self.gate_down: TensorSpec((self.rank, W)), self.gate_up: TensorSpec((hv, self.rank)),
+            self.out_norm: TensorSpec((self.value_head_dim,)), self.o_proj: TensorSpec((W, hv)),
+        }
+
+    def cache_need(self):
+        """Entry 0: the matrix states; entry 1: the convolutions' last inputs (q, k and v side by side)."""
+        return (StateNeed((self.num_heads, self.head_dim, self.value_head_dim)), StateNeed((max(self.taps - 1, 1), self.channels)))
+
+
+@dataclass(frozen=True)
 class RotaryValueAttentionSpec:
     """Grouped-query softmax attention whose values carry positions too.  q and k are rotated on their first
     ``position.rotary_dim`` entries (:class:`RotarySpec`).  ``value_norm``: each value head is divided by its root
@@ -607,7 +704,10 @@ class RotaryValueAttentionSpec:
     c * tanh(s / c) before the mask and the softmax.  ``sink_score`` z: exp(z) joins the softmax's denominator, with no key
     and no value (0: one is added to it).  ``reads_cache``: the mixer has queries only (no k and v tensors) and attends over
     the keys and values that another layer's mixer stores; its layer call names that layer's cache entry with ``store``
-    False.  ``position`` then turns the queries only."""
+    False.  ``position`` then turns the queries only.
+
+    ``unit_qk``: after the rotation each q and k head is divided by its root mean square (no weight, ``eps``).  ``gate``:
+    the heads side by side are multiplied element by element by sigmoid(G h) before ``o_proj``."""
     hidden_size: int
     num_heads: int
     num_kv_heads: int
@@ -630,6 +730,8 @@ class RotaryValueAttentionSpec:
     softcap: Optional[float] = None
     sink_score: Optional[float] = None
     reads_cache: bool = False
+    unit_qk: bool = False
+    gate: Optional[str] = None
 
     def tensors(self) -> Mapping[str, TensorSpec]:
         W = self.hidden_size
@@ -642,6 +744,8 @@ class RotaryValueAttentionSpec:
                 t[proj] = TensorSpec((width, W))
             if bias is not None:
                 t[bias] = TensorSpec((width,), init=(0.0, 0.3))
+        if self.gate is not None:
+            t[self.gate] = TensorSpec((self.num_heads * self.value_head_dim, W))
         return t
 
     def cache_need(self):
@@ -942,7 +1046,7 @@ class ModelPlan:
     vocab_size: int
     hidden_size: int
     max_positions: int
-    embedding: EmbeddingSpec
+    embedding: object                    # may keep state of its own (``cache_need``): cache entry EMBEDDING_CACHE
     layers: Tuple[object, ...]
     schedule: Tuple[LayerCall, ...]
     final_norm: object

@@ -176,7 +176,7 @@ __device__ __forceinline__ void store_from_f32(void* p, int dtype, size_t i, flo
 }
 
 // A function of one number applied to each element of a product before it is stored (the `epilogue` argument of the
-// products carries it in the bits above the lowest four): 0 none, 1 relu(y)^2, 2 silu, 3 sigmoid, 4 gelu (tanh form), 5 tanh.
+// products carries it in the bits above the lowest four; in a gated product it is the gate's, and 0 means silu there): 0 none, 1 relu(y)^2, 2 silu, 3 sigmoid, 4 gelu (tanh form), 5 tanh.
 #define IFB_UNARY_NONE 0
 #define IFB_UNARY_RELU2 1
 #define IFB_UNARY_SILU 2
@@ -194,6 +194,9 @@ __device__ __forceinline__ float ifb_unary(float y, int kind) {
     default: return y;
   }
 }
+
+// The function on the gate of a gated product (epilogue 1): silu, or the unary function in the epilogue's upper bits.
+__device__ __forceinline__ float ifb_gate_act(float g, int kind) { return kind ? ifb_unary(g, kind) : g / (1.f + expf(-g)); }
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

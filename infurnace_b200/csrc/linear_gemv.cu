@@ -42,7 +42,7 @@ struct GvRowScale {        // consumer side: null `partials` = none
   const float* partials;   // [parts][n_rows] partial sums of squares
   int parts;
   float eps, inv_width;    // r = rsqrt(sum * inv_width + eps)
-  int unary;               // plain epilogue only: the function of common.cuh applied to every element (0: none)
+  int unary;               // the function of common.cuh applied to every element (0: none), or to the gates (0: silu)
   const float* bias;       // plain epilogue only: [o_out], added before the unary function (null: none)
 };
 struct GvResidual {        // producer side, epilogue 2
@@ -84,7 +84,7 @@ __device__ __forceinline__ void gv_cluster_barrier() {
 }
 
 // NB: blocks of 8 tokens per CTA.  EPI 0: out = y.  EPI 1: w holds gate rows [0, O) and up rows [O, 2O);
-// out = silu(gate) * up.  EPI 2: v = x + y is written back to x, out = v * g.  EPI 4: as EPI 1 with 8 features per
+// out = act(gate) * up, act = silu or rs.unary.  EPI 2: v = x + y is written back to x, out = v * g.  EPI 4: as EPI 1 with 8 features per
 // CTA, whose 8 gate rows and 8 up rows are the two halves of one 16-row tile (half the registers of EPI 1, so two CTAs
 // per SM where EPI 1 with two stages has one).  WARPS: warps of a CTA (they split k).
 // STAGES: steps of 128 of k whose weights (and, for one block of tokens, activations) a warp has requested at any
@@ -301,14 +301,14 @@ linear_gemv_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, TO* _
       y[e] = rs.partials ? s * row_factor[n] : s;
     }
     float r = y[0];
-    if (EPI == 1) r = r / (1.f + expf(-r)) * y[NE - 1];
+    if (EPI == 1) r = ifb_gate_act(r, rs.unary) * y[NE - 1];
     if (EPI == 4) {                                    // this item is the gate of feature o0 + m; its up sits 8 rows on
       if (m >= 8) continue;
       float up = 0.f;
 #pragma unroll
       for (int wv = 0; wv < WARPS; ++wv) up += gv_red[((size_t)wv * NB * 8 + n) * GV_ROWS + m + 8];
       if (rs.partials) up *= row_factor[n];
-      if (valid) out[(size_t)tok * o_out + o] = from_f32<TO>(r / (1.f + expf(-r)) * up);
+      if (valid) out[(size_t)tok * o_out + o] = from_f32<TO>(ifb_gate_act(r, rs.unary) * up);
       continue;
     }
     if (EPI == 3) { qk_y0 = y[0]; qk_y1 = y[NE - 1]; continue; }      // finished below, after the loop (one item per thread)
@@ -505,7 +505,7 @@ IFB_EXPORT int ifb_linear_gemv(const void* x, const void* w, void* out, int out_
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return IFB_ERR_ALIGN;
   const int unary = epilogue >> 4;
   epilogue &= 15;
-  if (epilogue > 1 || unary < 0 || unary > IFB_UNARY_LAST || (epilogue && (unary || bias))) return IFB_ERR_ARG;
+  if (epilogue > 1 || unary < 0 || unary > IFB_UNARY_LAST || (epilogue && bias)) return IFB_ERR_ARG;
   if (scale_partials && (scale_parts < 1 || scale_width < 1)) return IFB_ERR_ARG;
   const int nb = gv_blocks_of_8(n_rows);
   if ((n_rows + nb * 8 - 1) / (nb * 8) > 65535) return IFB_ERR_SIZE;

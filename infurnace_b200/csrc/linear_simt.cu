@@ -11,7 +11,7 @@
 #define TILE_K 16
 
 // EPI 0: out = unary(y + bias) (common.cuh: ifb_unary; 0 = y itself; bias null: none).  EPI 1 (silu_gate): w has 2*o_out rows, gate rows first;
-// out[n, o] = silu(y[n, o]) * y[n, o_out + o].
+// out[n, o] = act(y[n, o]) * y[n, o_out + o] with act = silu or the unary function.
 template <typename TX, typename TW, typename TO, int EPI>
 __global__ void __launch_bounds__(256)
 linear_simt_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restrict__ out, int n_rows, int o_out,
@@ -76,7 +76,7 @@ linear_simt_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __res
       const int o = o0 + to * 4 + j;
       if (o >= o_out) continue;
       float y = acc[0][i][j];
-      if (EPI) { const float g = y; y = g / (1.f + expf(-g)) * acc[EPI ? 1 : 0][i][j]; }
+      if (EPI) y = ifb_gate_act(y, unary) * acc[EPI ? 1 : 0][i][j];
       else {
         if (bias) y += bias[o];
         if (unary) y = ifb_unary(y, unary);
@@ -92,17 +92,17 @@ static int launch(const void* x, const void* w, void* out, int n, int o, int k, 
   const int unary = epi >> 4;
   if ((epi & 15) == 0)
     return ifb_launch(linear_simt_kernel<TX, TW, TO, 0>, grid, dim3(256), 0, s, (const TX*)x, (const TW*)w, (TO*)out, n, o, k, unary, bias);
-  return ifb_launch(linear_simt_kernel<TX, TW, TO, 1>, grid, dim3(256), 0, s, (const TX*)x, (const TW*)w, (TO*)out, n, o, k, 0, (const float*)nullptr);
+  return ifb_launch(linear_simt_kernel<TX, TW, TO, 1>, grid, dim3(256), 0, s, (const TX*)x, (const TW*)w, (TO*)out, n, o, k, unary, (const float*)nullptr);
 }
 
 // out_features is the width of `out` (for the silu_gate epilogue, half of w's rows).  epilogue: 0 plain, 1 silu_gate,
-// 16 * u: plain with the unary function u of common.cuh applied to every element.  bias (plain epilogue; may be null):
+// 16 * u: plain with the unary function u of common.cuh applied to every element, 1 + 16 * u: gated with u in silu's place.  bias (plain epilogue; may be null):
 // float32 [out_features], added before the unary function.
 IFB_EXPORT int ifb_linear_simt(const void* x, int x_dtype, const void* w, int w_dtype, void* out, int out_dtype,
                                int n_rows, int out_features, int k_dim, int epilogue, const float* bias, cudaStream_t stream) {
   if (n_rows <= 0 || out_features <= 0) return IFB_OK;
   if (k_dim < 1) return IFB_ERR_SIZE;
-  if ((epilogue & 15) > 1 || (epilogue >> 4) > IFB_UNARY_LAST || ((epilogue & 15) && (epilogue >> 4)) || epilogue < 0 ||
+  if ((epilogue & 15) > 1 || (epilogue >> 4) > IFB_UNARY_LAST || epilogue < 0 ||
       (bias && (epilogue & 15)))
     return IFB_ERR_ARG;
   if ((n_rows + TILE_N - 1) / TILE_N > 65535) return IFB_ERR_SIZE;

@@ -144,6 +144,14 @@ __device__ __forceinline__ uint64_t make_smem_desc(uint32_t smem_addr) {
   return (uint64_t)((smem_addr >> 4) & 0x3FFF) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
 }
 
+// The gate's function with the hardware's exp2 and reciprocal (relative error about 1e-6; the result is rounded to the
+// output type): silu, or gelu in the tanh form, which is g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3)); others exactly.
+__device__ __forceinline__ float tc_gate(float g, int kind) {
+  if (kind != IFB_UNARY_NONE && kind != IFB_UNARY_GELU_TANH) return ifb_unary(g, kind);
+  const float z = kind ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
+  return g * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * z));
+}
+
 // A normalisation folded into the products around it (RMSNorm(v) = v * g * r with one r per row): the product that
 // makes v (plain epilogue) adds the residual stream, writes v back to it, writes v * g as its output and leaves sums of
 // v^2 over slices of the features; the product that reads v * g multiplies its rows by r, from those sums added in a
@@ -156,7 +164,7 @@ struct TcFold {
   const void* res_g;          // [o_out] norm weight
   int res_g_dtype;
   float* res_partials;        // [parts][n_rows], written; what a part covers depends on the launch (tc_fold_parts)
-  int unary;                  // plain epilogue without res_x: the function of common.cuh applied to every element (0: none)
+  int unary;                  // without res_x: the function of common.cuh applied to every element (0: none), or to the gates (0: silu)
   const float* bias;          // plain epilogue: [o_out], added to the product before the unary function (null: none)
   // The product is the fused q | k | v projection of an attention layer with heads of 128, in the shared-k form, whose
   // tile of 128 features is one head: the sum over the cluster finishes what follows the projection (RMSNorm over the q
@@ -371,12 +379,12 @@ linear_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
             uint32_t u[32];
             tmem_ld32(lane_base + FO + c0, u);
             tmem_ld_wait();
+            if (fold.unary) {                                    // warp-uniform: another function than silu on the gate
 #pragma unroll
-            for (int j = 0; j < 32; ++j) {
-              // silu(g) * u with the hardware's exp2 and reciprocal (relative error about 1e-6; the result is
-              // rounded to the output type)
-              const float g = __uint_as_float(v[j]) * rfac;
-              y[j] = g * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * g)) * (__uint_as_float(u[j]) * rfac);
+              for (int j = 0; j < 32; ++j) y[j] = tc_gate(__uint_as_float(v[j]) * rfac, fold.unary) * (__uint_as_float(u[j]) * rfac);
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) y[j] = tc_gate(__uint_as_float(v[j]) * rfac, 0) * (__uint_as_float(u[j]) * rfac);
             }
           } else {
             tmem_ld_wait();
@@ -456,10 +464,8 @@ linear_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
           const float4 v = ld_cluster_f4(at + FO * 4, z);
           up.x += v.x; up.y += v.y; up.z += v.z; up.w += v.w;
         }
-        acc.x = acc.x * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * acc.x)) * up.x;
-        acc.y = acc.y * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * acc.y)) * up.y;
-        acc.z = acc.z * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * acc.z)) * up.z;
-        acc.w = acc.w * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * acc.w)) * up.w;
+        acc.x = tc_gate(acc.x, fold.unary) * up.x; acc.y = tc_gate(acc.y, fold.unary) * up.y;
+        acc.z = tc_gate(acc.z, fold.unary) * up.z; acc.w = tc_gate(acc.w, fold.unary) * up.w;
       }
       TO* dst = out + (size_t)(m0 + r) * o_out + n0 + c;
       if (!EPI && fold.bias) {
@@ -715,10 +721,12 @@ linear_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap tmap_x, con
             uint32_t u[32];
             tmem_ld32(lane_base + FO + c0, u);
             tmem_ld_wait();
+            if (fold.unary) {                                    // warp-uniform: another function than silu on the gate
 #pragma unroll
-            for (int j = 0; j < 32; ++j) {
-              const float gte = __uint_as_float(v[j]) * rfac;
-              y[j] = gte * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * gte)) * (__uint_as_float(u[j]) * rfac);
+              for (int j = 0; j < 32; ++j) y[j] = tc_gate(__uint_as_float(v[j]) * rfac, fold.unary) * (__uint_as_float(u[j]) * rfac);
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) y[j] = tc_gate(__uint_as_float(v[j]) * rfac, 0) * (__uint_as_float(u[j]) * rfac);
             }
           } else {
             tmem_ld_wait();
@@ -884,7 +892,8 @@ static int tc_launch(const void* x, const void* w, void* out, int n, int o, int 
   return tc_launch_cfg<Narrow, TO>(x, w, out, n, o, k, err, s, fold);
 }
 
-// epilogue: 0 plain, 1 silu_gate, 16 * u: plain with the unary function u of common.cuh applied to every element.
+// epilogue: 0 plain, 1 silu_gate, 16 * u: plain with the unary function u of common.cuh applied to every element,
+// 1 + 16 * u: gated with u in silu's place.
 // x [n_rows, k] and w [out_features (x2 for the silu_gate epilogue), k] bfloat16, 16-byte aligned, k a multiple of 8;
 // out bfloat16 or float32.  `err` points to a device int that stays 0 unless a bounded wait gave up.  shape: 0 lets the
 // library choose, 1-3 force the one-tile-per-CTA kernel narrow, deep or wide, 4 and 5 the persistent kernel with tiles
@@ -904,7 +913,7 @@ IFB_EXPORT int ifb_linear_tcgen05_ex(const void* x, const void* w, void* out, in
   if (((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return IFB_ERR_ALIGN;
   const int unary = epilogue >> 4;
   epilogue &= 15;
-  if (epilogue > 1 || unary < 0 || unary > IFB_UNARY_LAST || (unary && (epilogue || res_x)) || (bias && epilogue))
+  if (epilogue > 1 || unary < 0 || unary > IFB_UNARY_LAST || (unary && res_x) || (bias && epilogue))
     return IFB_ERR_ARG;
   if (shape < 0 || shape > 5 || splits < 0 || splits > 8) return IFB_ERR_ARG;
   if (scale_partials && (scale_parts < 1 || scale_width < 1)) return IFB_ERR_ARG;

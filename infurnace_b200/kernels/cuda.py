@@ -18,8 +18,9 @@ from .build import load_library
 
 F32, BF16 = 0, 1
 # the `epilogue` argument of the products: 0 plain, 1 silu_gate (w holds gate rows, then up rows), 16 * u: plain with the
-# unary function u applied to every element (csrc/common.cuh: ifb_unary)
-EPILOGUES = {"none": 0, "silu_gate": 1, "relu2": 16, "silu": 32, "sigmoid": 48, "gelu_tanh": 64, "tanh": 80}
+# unary function u applied to every element, 1 + 16 * u: gated with u on the gate (csrc/common.cuh: ifb_unary)
+EPILOGUES = {"none": 0, "silu_gate": 1, "relu2": 16, "silu": 32, "sigmoid": 48, "gelu_tanh": 64, "tanh": 80,
+             "gelu_gate": 65}
 _CODES = {torch.float32: F32, torch.bfloat16: BF16}
 _ERRORS = {1: "a dtype (or combination of dtypes) has no kernel", 2: "a size is outside what the kernel takes",
            3: "an address or row length breaks the kernel's alignment rule", 4: "arguments contradict each other"}
@@ -224,12 +225,12 @@ class CudaKernels:
             epi = EPILOGUES[epilogue]
         except KeyError:
             raise KernelError(f"linear: unknown epilogue {epilogue!r}; known: {', '.join(EPILOGUES)}") from None
-        gated = epi == 1
+        gated = bool(epi & 1)
         route = "silu_gate" if gated else "none"          # a unary function changes nothing in the choice of kernel
         if w.shape[1] != k or out.shape[0] != n or w.shape[0] != (2 * o if gated else o):
             raise KernelError(f"linear: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)} do not match")
         if bias is not None and (_dense(bias, "bias", torch.float32).numel() != o or gated):
-            raise KernelError("linear: bias is one float32 number per output feature, and 'silu_gate' takes none")
+            raise KernelError("linear: bias is one float32 number per output feature, and the gated epilogues take none")
         if row_scale is not None:
             if not self.can_fold_norm(n, x.dtype, w, route) or out.dtype not in (torch.bfloat16, torch.float32):
                 raise KernelError("linear: a row scale is taken only by the bfloat16 kernels (see can_fold_norm)")

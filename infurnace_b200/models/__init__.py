@@ -10,3 +10,4 @@ from . import lunelorn  # noqa: F401  (registers "Lunelorn")
 from . import filorax  # noqa: F401  (registers "Filorax")
 from . import golonex  # noqa: F401  (registers "Golonex")
 from . import mubutar  # noqa: F401  (registers "Mubutar")
+from . import tigelorn  # noqa: F401  (registers "Tigelorn")

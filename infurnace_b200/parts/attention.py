@@ -4,6 +4,7 @@ from __future__ import annotations
 import torch
 
 from ..config.specs import AttentionSpec
+from .norm import norm_gain
 from .registry import build_part, fold_residual_norm, register_part, unfolded
 
 
@@ -27,8 +28,8 @@ class PagedAttention:
         wq, wk, wv = weights[spec.q_proj], weights[spec.k_proj], weights[spec.v_proj]
         self.w_qkv = torch.cat((wq, wk, wv), dim=0).contiguous()
         self.w_o = weights[spec.o_proj]
-        self.q_norm_w = weights[spec.q_norm.weight] if spec.q_norm is not None else None
-        self.k_norm_w = weights[spec.k_norm.weight] if spec.k_norm is not None else None
+        self.q_norm_w = norm_gain(spec.q_norm, weights) if spec.q_norm is not None else None
+        self.k_norm_w = norm_gain(spec.k_norm, weights) if spec.k_norm is not None else None
         eps = [n.eps for n in (spec.q_norm, spec.k_norm) if n is not None]
         if len(set(eps)) > 1:
             raise ValueError("q_norm and k_norm must share eps: one kernel normalises both")

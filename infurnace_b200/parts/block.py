@@ -60,6 +60,8 @@ class PreNormBlock:
             h = ctx.buffer("h", x.shape, self.rt.act_dtype)
             self.mixer_norm.forward(x, h, delta=pending)
         if self.ffn is None:
+            if self.side is None and next_layer is not None and getattr(self.mixer, "can_fold_output", False) and next_layer.takes_folded(n):
+                return self.mixer.forward(h, ctx, call, fold=(x, next_layer.mixer_norm))     # a Folded, or the mixer's plain delta
             d = self.mixer.forward(h, ctx, call)
             return self._finish(x, d, ctx, next_layer)
         take = getattr(self.ffn, "can_take_folded", None)

@@ -4,7 +4,7 @@ from __future__ import annotations
 import torch
 
 from ..config.specs import LatentAttentionSpec
-from .registry import build_part, register_part
+from .registry import build_part, fold_residual_norm, register_part, unfolded
 
 
 class LatentAttention:
@@ -21,25 +21,30 @@ class LatentAttention:
     (the framework's grouped product, a head being what an expert is there); the attention kernel over the pages, this
     step's tokens included, with window and sink; a grouped product with UV_h; one kernel that applies the output gate
     and puts the heads side by side; the output product.  Where the queries have a latent of their own, they are two more
-    products with an RMS norm between them, and the first product holds latent, rotated key | gate only."""
+    products with an RMS norm between them, the first of which is part of the step's first product: query latent | latent,
+    rotated key | gate."""
 
     graph_safe = True
+    can_fold_output = True
+
+    def can_take_folded(self, n):
+        can = getattr(self.k, "can_fold_norm", None)
+        return bool(can and can(n, self.rt.act_dtype, self.w_in))
 
     def __init__(self, spec: LatentAttentionSpec, weights, runtime):
         self.spec = s = spec
         self.rt = runtime
         self.k = runtime.kernels
         H, D, V, R = s.num_heads, s.head_dim, s.value_head_dim, s.kv_rank
-        # with a latent of their own the queries are two products with a norm between them, and the step's first product
-        # holds latent, rotated key | gate only
+        # with a latent of their own the queries are two products with a norm between them
         self.q_latent = bool(s.q_rank)
-        parts = [weights[s.down_proj]] if self.q_latent else [weights[s.q_proj], weights[s.down_proj]]
+        parts = [weights[s.q_down if self.q_latent else s.q_proj], weights[s.down_proj]]
         if s.gate is not None:
             parts.append(weights[s.gate])
         self.w_in = torch.cat(parts, dim=0).contiguous()
         if self.q_latent:
-            self.w_q_down, self.w_q_up, self.q_norm_w = weights[s.q_down], weights[s.q_proj], weights[s.q_norm]
-        self.down_col = 0 if self.q_latent else H * (D + s.rot_dim)
+            self.w_q_up, self.q_norm_w = weights[s.q_proj], weights[s.q_norm].float().contiguous()
+        self.down_col = s.q_rank if self.q_latent else H * (D + s.rot_dim)
         self.gate_col = self.down_col + R + s.rot_dim
         self.gate_width = H if s.gate_per_head else H * V
         self.norm_w = weights[s.latent_norm]
@@ -62,19 +67,18 @@ class LatentAttention:
             return -(-n // t) * t, t
         return n, 0
 
-    def forward(self, h, ctx, call):
+    def forward(self, h, ctx, call, fold=None):
         s, k = self.spec, self.k
+        h, row_scale = unfolded(h)
         n = h.shape[0]
         H, D, V, R, r = s.num_heads, s.head_dim, s.value_head_dim, s.kv_rank, s.rot_dim
         act = self.rt.act_dtype
         proj = ctx.buffer("la_proj", (n, self.w_in.shape[0]), torch.float32)
-        k.linear(h, self.w_in, proj)
+        k.linear(h, self.w_in, proj, **({"row_scale": row_scale} if row_scale is not None else {}))
         q = None
         if self.q_latent:
-            cq_raw = ctx.buffer("la_cq_raw", (n, s.q_rank), torch.float32)
-            k.linear(h, self.w_q_down, cq_raw)
             cq = ctx.buffer("la_cq", (n, s.q_rank), act)
-            k.rmsnorm(cq_raw, self.q_norm_w, s.eps, cq)
+            k.norm_gate_rows(proj[:, :s.q_rank], cq, groups=1, weight=self.q_norm_w, eps=s.eps)
             q = ctx.buffer("la_q", (n, H * (D + r)), torch.float32)
             k.linear(cq, self.w_q_up, q)
         extra = {}
@@ -114,6 +118,9 @@ class LatentAttention:
             k.gate_heads(y.view(H, seg, V), gate, out, n, per_head=True)
         else:
             k.gate_heads(y.view(H, seg, V), gate, out, n)
+        folded = fold_residual_norm(k, ctx, "mixer", out, self.w_o, fold, act)
+        if folded is not None:
+            return folded
         delta = ctx.buffer("delta_mixer", (n, s.hidden_size), torch.float32)
         k.linear(out, self.w_o, delta)
         return delta

@@ -9,15 +9,17 @@ from .registry import fold_residual_norm, register_part, unfolded
 
 
 class GatedMLP:
-    """down(silu(gate(h)) * up(h)) (src/infurnace/executor/tinygrad/model.py:146-148).
+    """down(act(gate(h)) * up(h)), act silu or the tanh form of gelu (src/infurnace/executor/tinygrad/model.py:146-148).
     gate and up run as one product against their row-wise concatenation (exact), with the
     activation and the product of the two halves in that kernel's epilogue."""
 
     graph_safe = True     # launches depend on the step's sizes only, never on values read on the host
+    EPILOGUES = {"silu": "silu_gate", "gelu_tanh": "gelu_gate"}
 
     def __init__(self, spec: GatedMLPSpec, weights, runtime):
-        if spec.activation != "silu":
-            raise ModelConfigError(f"activation {spec.activation!r}: only 'silu' has a kernel")
+        if spec.activation not in self.EPILOGUES:
+            raise ModelConfigError(f"activation {spec.activation!r}: the gated feed-forward has {', '.join(self.EPILOGUES)}")
+        self.epilogue = self.EPILOGUES[spec.activation]
         self.spec = spec
         self.rt = runtime
         self.k = runtime.kernels
@@ -36,9 +38,9 @@ class GatedMLP:
         n = h.shape[0]
         act = ctx.buffer("ffn_act", (n, self.spec.intermediate_size), self.rt.act_dtype)
         if row_scale is not None:
-            self.k.linear(h, self.w_gate_up, act, epilogue="silu_gate", row_scale=row_scale)
+            self.k.linear(h, self.w_gate_up, act, epilogue=self.epilogue, row_scale=row_scale)
         else:
-            self.k.linear(h, self.w_gate_up, act, epilogue="silu_gate")
+            self.k.linear(h, self.w_gate_up, act, epilogue=self.epilogue)
         folded = fold_residual_norm(self.k, ctx, "ffn", act, self.w_down, fold, self.rt.act_dtype)
         if folded is not None:
             return folded

@@ -3,7 +3,7 @@ from __future__ import annotations
 
 import torch
 
-from ..config.specs import EmbeddingSpec, LMHeadSpec, ModelPlan, NormedEmbeddingSpec, SinusoidEmbeddingSpec
+from ..config.specs import EMBEDDING_CACHE, BigramEmbeddingSpec, EmbeddingSpec, LMHeadSpec, ModelPlan, NormedEmbeddingSpec, SinusoidEmbeddingSpec
 from .registry import build_part, register_part
 
 
@@ -94,6 +94,25 @@ class NormedEmbedding:
         return out
 
 
+class BigramEmbedding:
+    """x[t] = table[id_t] + pairs[row_t] in float32, row_t from the token and the one before it in its sequence (a row of its
+    own for the first).  The token before a portion's first comes from the request's row of the cache entry
+    ``EMBEDDING_CACHE``, which then takes the portion's last token; all of it is one kernel."""
+
+    uses_context = True
+
+    def __init__(self, spec: BigramEmbeddingSpec, weights, runtime):
+        self.spec = spec
+        self.table, self.pairs = weights[spec.weight], weights[spec.pairs]
+        self.k = runtime.kernels
+
+    def forward(self, ids, out, ctx=None):
+        s = self.spec
+        self.k.embed_bigram(self.table, self.pairs, ids, ctx.positions, ctx.req_index, ctx.cu_q, ctx.seq_lens, ctx.state_slots,
+                            ctx.state(EMBEDDING_CACHE), s.buckets, s.mul_prev, s.mul_cur, out)
+        return out
+
+
 # key of ``ctx.shared`` under which the embedding's rows are kept for the step
 EMBEDDING_ROWS = ("embedding_rows",)
 
@@ -102,6 +121,7 @@ EMBEDDING_ROWS = ("embedding_rows",)
 STREAM_COPY = ("stream_copy",)
 
 register_part(EmbeddingSpec, Embedding)
+register_part(BigramEmbeddingSpec, BigramEmbedding)
 register_part(SinusoidEmbeddingSpec, SinusoidEmbedding)
 register_part(LMHeadSpec, LMHead)
 register_part(NormedEmbeddingSpec, NormedEmbedding)

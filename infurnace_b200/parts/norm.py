@@ -5,6 +5,13 @@ from ..config.specs import GroupRMSNormSpec, RMSNormSpec, ScalarRMSNormSpec
 from .registry import register_part
 
 
+def norm_gain(spec: RMSNormSpec, weights):
+    """What the normalised row is multiplied by: the stored weight, or, where it is stored around ``spec.offset``, the sum
+    (formed and kept in float32)."""
+    w = weights[spec.weight]
+    return w if not spec.offset else (w.float() + spec.offset).contiguous()
+
+
 class RMSNorm:
     """out = (x + delta) * rsqrt(mean((x + delta)^2) + eps) * weight, statistics in 32-bit
     (src/infurnace/executor/tinygrad/model.py:11-13).  x is the float32 residual stream;
@@ -16,7 +23,7 @@ class RMSNorm:
 
     def __init__(self, spec: RMSNormSpec, weights, runtime):
         self.spec = spec
-        self.weight = weights[spec.weight]
+        self.weight = norm_gain(spec, weights)
         self.k = runtime.kernels
 
     def forward(self, x, out, delta=None, rows=None):

@@ -1,12 +1,13 @@
 """Recurrent mixers whose state lives in the request's state slot: the HGRN2 gated recurrence, retention with a fixed
-decay per head, RWKV-style time mixing (all three a matrix state per head), the element-wise minGRU and the real-gated
+decay per head, RWKV-style time mixing, the gated delta rule (all four a matrix state per head), the element-wise minGRU and the real-gated
 linear recurrent unit behind a short convolution."""
 from __future__ import annotations
 
 import torch
 
-from ..config.specs import GatedRecurrenceSpec, GatedUnitSpec, RealGatedRecurrenceSpec, RetentionSpec, TimeMixSpec
-from .registry import register_part
+from ..config.specs import DeltaRuleSpec, GatedRecurrenceSpec, GatedUnitSpec, RealGatedRecurrenceSpec, RetentionSpec, TimeMixSpec
+from ..errors import WeightError
+from .registry import fold_residual_norm, register_part, unfolded
 
 
 class GatedRecurrence:
@@ -51,37 +52,69 @@ register_part(GatedRecurrenceSpec, GatedRecurrence)
 
 
 class Retention:
-    """h -> o_proj(unit_norm(S^T q) * silu(G h)) with S <- decay_h S + (k * key_scale) v^T per head.
+    """h -> o_proj(norm(S^T q) * act(G h)) with S <- decay_h S + (k * key_scale) v^T per head.
 
     q | k | v | g run as one product into float32 (what enters the recurrence is 32-bit).  The recurrence kernel is
     the framework's walk of a matrix state per head (``linear_scan``) with a constant decay per head; it divides each
     head's output by its root mean square and multiplies by silu of the gate columns before it writes the rows that
-    ``o_proj`` reads.  A prompt, a portion and a decoded token are the same call: the slot's state carries the past."""
+    ``o_proj`` reads.  Where the heads are normed together, or the gate is a sigmoid, the recurrence leaves its float32
+    outputs and a second kernel does both.  q, k and v may pass silu as the recurrence reads them.  A prompt, a portion and a
+    decoded token are the same call: the slot's state carries the past.  The part can share its first and last products with
+    mixers beside it (``w_in``, ``mix``, ``w_o``)."""
 
     graph_safe = True
+    can_fold_output = True
+    joint = True
+    b_in = None
+
+    def can_take_folded(self, n):
+        can = getattr(self.k, "can_fold_norm", None)
+        return bool(can and can(n, self.rt.act_dtype, self.w_in))
 
     def __init__(self, spec: RetentionSpec, weights, runtime):
         self.spec = spec
         self.rt = runtime
         self.k = runtime.kernels
-        self.w_all = torch.cat([weights[n] for n in (spec.q_proj, spec.k_proj, spec.v_proj, spec.g_proj)], dim=0).contiguous()
+        if spec.input_activation not in (None, "silu") or spec.gate_activation not in ("silu", "sigmoid"):
+            raise ValueError("retention: the inputs' activation is silu or none, the gate's silu or sigmoid")
+        self.w_in = torch.cat([weights[n] for n in (spec.q_proj, spec.k_proj, spec.v_proj, spec.g_proj)], dim=0).contiguous()
         self.w_o = weights[spec.o_proj]
+        self.joint_w = weights[spec.joint_norm].float().contiguous() if spec.joint_norm is not None else None
         self.decay = torch.tensor(spec.decay, dtype=torch.float32, device=runtime.device)
         self.hd = spec.num_heads * spec.head_dim
-        self.hv = spec.num_heads * spec.value_head_dim
+        self.hv = self.out_width = spec.num_heads * spec.value_head_dim
 
-    def forward(self, h, ctx, call):
-        s, k, hd, hv = self.spec, self.k, self.hd, self.hv
+    def forward(self, h, ctx, call, fold=None):
+        s, k = self.spec, self.k
+        h, row_scale = unfolded(h)
         n = h.shape[0]
-        proj = ctx.buffer("ret_proj", (n, 2 * hd + 2 * hv), torch.float32)
-        k.linear(h, self.w_all, proj)
-        out = ctx.buffer("ret_out", (n, hv), self.rt.act_dtype)
-        k.linear_scan(proj[:, :hd], proj[:, hd:2 * hd], proj[:, 2 * hd:2 * hd + hv], None, s.num_heads, s.head_dim,
-                      s.value_head_dim, ctx.state(call.cache), ctx.state_slots, ctx.cu_q, ctx.seq_lens, out, s.eps,
-                      decay=self.decay, key_scale=s.key_scale, gate=proj[:, 2 * hd + hv:], max_q_len=ctx.max_q_len)
+        proj = ctx.buffer("ret_proj", (n, self.w_in.shape[0]), torch.float32)
+        k.linear(h, self.w_in, proj, **({"row_scale": row_scale} if row_scale is not None else {}))
+        out = ctx.buffer("ret_out", (n, self.hv), self.rt.act_dtype)
+        self.mix(proj, ctx, call, out)
+        folded = fold_residual_norm(k, ctx, "mixer", out, self.w_o, fold, self.rt.act_dtype)
+        if folded is not None:
+            return folded
         delta = ctx.buffer("delta_mixer", (n, s.hidden_size), torch.float32)
         k.linear(out, self.w_o, delta)
         return delta
+
+    def mix(self, proj, ctx, call, out, gain=1.0):
+        """From the input product's rows (``proj``, maybe a slice of a wider product) to ``gain`` times the gated heads in
+        ``out``, whose rows may be a slice too."""
+        s, k, hd, hv = self.spec, self.k, self.hd, self.hv
+        n = proj.shape[0]
+        one_pass = self.joint_w is None and s.gate_activation == "silu" and gain == 1.0 and out.is_contiguous()
+        gate = proj[:, 2 * hd + hv:]
+        extra = {"activation": s.input_activation} if s.input_activation is not None else {}
+        o = out if one_pass else ctx.buffer("ret_raw", (n, hv), torch.float32)
+        k.linear_scan(proj[:, :hd], proj[:, hd:2 * hd], proj[:, 2 * hd:2 * hd + hv], None, s.num_heads, s.head_dim,
+                      s.value_head_dim, ctx.state(call.cache), ctx.state_slots, ctx.cu_q, ctx.seq_lens, o, s.eps,
+                      decay=self.decay, key_scale=s.key_scale, max_q_len=ctx.max_q_len,
+                      **({"gate": gate} if one_pass else {"finish": False}), **extra)
+        if not one_pass:
+            k.norm_gate_rows(o, out, groups=1 if self.joint_w is not None else s.num_heads, weight=self.joint_w, eps=s.eps,
+                             gate=gate, activation=s.gate_activation, scale=gain)
 
 
 register_part(RetentionSpec, Retention)
@@ -134,11 +167,82 @@ class TimeMix:
 register_part(TimeMixSpec, TimeMix)
 
 
+class DeltaRule:
+    """h -> o_proj(norm(S^T q) * sigmoid(g2 g1 h)); S <- diag(g) S, S <- S + k (beta (v - S^T k))^T per head.
+
+    q | k | v | beta | the two bottlenecks run as one product into float32.  One kernel runs the short convolutions over each
+    request's tokens from the inputs its slot kept (cache entry 1), applies silu and makes q and k unit vectors, forms beta,
+    and hands the bottlenecks on in the products' dtype.  Their two second matrices are one product against a
+    block-diagonal matrix (exact: the other block is zeros) into float32.  The recurrence kernel forms the decays in float32
+    from those rows and walks each request's tokens from the slot's state (cache entry 0), or, for long portions, runs chunks
+    of 16 tokens side by side as far as they do not depend on the state; each head's norm and gate follow."""
+
+    graph_safe = True
+    can_fold_output = True
+
+    def __init__(self, spec: DeltaRuleSpec, weights, runtime):
+        self.spec = s = spec
+        self.rt = runtime
+        self.k = runtime.kernels
+        H, D, V = s.num_heads, s.head_dim, s.value_head_dim
+        if H % s.num_kv_heads:
+            raise ValueError("delta rule: the heads are a multiple of the query/key heads")
+        down = [weights[n] for n in (s.decay_down, s.gate_down)]
+        up = [weights[n] for n in (s.decay_up, s.gate_up)]
+        if any(d.shape[0] != u.shape[1] for d, u in zip(down, up)):
+            raise WeightError(f"weights do not match the model: {s.decay_up} / {s.gate_up} do not take what {s.decay_down} / "
+                              f"{s.gate_down} give")
+        self.w_in = torch.cat([weights[n] for n in (s.q_proj, s.k_proj, s.v_proj, s.beta_proj)] + down, dim=0).contiguous()
+        self.low_width = sum(d.shape[0] for d in down)
+        self.low_cols = -(-self.low_width // 8) * 8       # the second product's k: a multiple of 8, zeros beyond
+        w_up = torch.zeros((H * (D + V), self.low_cols), dtype=up[0].dtype, device=up[0].device)
+        w_up[:H * D, :down[0].shape[0]] = up[0]
+        w_up[H * D:, down[0].shape[0]:self.low_width] = up[1]
+        self.w_up = w_up
+        f32 = lambda t: t.to(torch.float32).contiguous()      # small parameters: the kernels read float32
+        self.taps = f32(torch.cat([weights[n] for n in (s.q_conv, s.k_conv, s.v_conv)], dim=0))
+        self.rate = torch.exp(f32(weights[s.a_log]))
+        self.decay_bias, self.norm_w = f32(weights[s.decay_bias]), f32(weights[s.out_norm])
+        self.w_o = weights[s.o_proj]
+
+    def can_take_folded(self, n):
+        can = getattr(self.k, "can_fold_norm", None)
+        return bool(can and can(n, self.rt.act_dtype, self.w_in))
+
+    def forward(self, h, ctx, call, fold=None):
+        s, k = self.spec, self.k
+        h, row_scale = unfolded(h)
+        n = h.shape[0]
+        H, G, D, V = s.num_heads, s.num_kv_heads, s.head_dim, s.value_head_dim
+        proj = ctx.buffer("dr_proj", (n, self.w_in.shape[0]), torch.float32)
+        k.linear(h, self.w_in, proj, **({"row_scale": row_scale} if row_scale is not None else {}))
+        qkv = ctx.buffer("dr_qkv", (n, s.channels), torch.float32)
+        beta = ctx.buffer("dr_beta", (n, H), torch.float32)
+        low = ctx.buffer("dr_low", (n, self.low_cols), self.rt.act_dtype)
+        k.delta_prepare(proj, G, H, D, V, self.taps, s.unit_eps, ctx.state((call.cache, 1)), ctx.state_slots, ctx.cu_q, ctx.seq_lens,
+                        ctx.req_index, qkv, beta, low, self.low_width)
+        up = ctx.buffer("dr_up", (n, H * (D + V)), torch.float32)
+        k.linear(low, self.w_up, up)
+        out = ctx.buffer("dr_out", (n, H * V), self.rt.act_dtype)
+        k.delta_rule(qkv, up, beta, G, H, D, V, self.rate, self.decay_bias, self.norm_w, s.eps, ctx.state((call.cache, 0)),
+                     ctx.state_slots, ctx.cu_q, ctx.seq_lens, out, max_q_len=ctx.max_q_len)
+        folded = fold_residual_norm(k, ctx, "mixer", out, self.w_o, fold, self.rt.act_dtype)
+        if folded is not None:
+            return folded
+        delta = ctx.buffer("delta_mixer", (n, s.hidden_size), torch.float32)
+        k.linear(out, self.w_o, delta)
+        return delta
+
+
+register_part(DeltaRuleSpec, DeltaRule)
+
+
 class GatedUnit:
     """minGRU: z | x | g run as one product into float32; one kernel adds the biases, forms gate and candidate,
     walks each request's tokens element by element from the slot's state and writes S * silu(g)."""
 
     graph_safe = True
+    delta_buffer = "delta_unit"
 
     def __init__(self, spec: GatedUnitSpec, weights, runtime):
         self.spec = spec

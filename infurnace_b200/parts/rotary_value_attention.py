@@ -1,5 +1,5 @@
 """Grouped-query softmax attention over page streams of keys and values: optional biases, positions on queries, keys and
-values, normalised values, a soft cap on the scores, a sink in the softmax, queries over another layer's keys and values."""
+values, normalised values, queries and keys of unit size, an output gate, a soft cap on the scores, a sink in the softmax, queries over another layer's keys and values."""
 from __future__ import annotations
 
 import torch
@@ -18,7 +18,12 @@ class RotaryValueAttention:
     in the cache's dtype and k and v into their page streams (which may differ in width).  The attention kernel reads
     every key and value from the pages, this step's included, keeps scores, softmax weights and sums in float32,
     and rotates each head's summed output back by the query's position before it stores it.  The angles come from
-    the rotary parts' per-step tables (cosine and sine of every token's angles, float32)."""
+    the rotary parts' per-step tables (cosine and sine of every token's angles, float32).
+
+    With ``unit_qk`` the storing kernel also divides the rotated q and k heads by their root mean square.  With a ``gate``
+    its matrix is a further block of rows of the one input product, and one kernel multiplies the heads by the gates'
+    sigmoids.  The part can stand inside a :class:`ParallelMixer` whose mixers share their first and last products
+    (``w_in``, ``b_in``, ``mix``, ``w_o``)."""
 
     graph_safe = True
 
@@ -31,11 +36,16 @@ class RotaryValueAttention:
             raise ValueError("values that are the keys have the keys' width, no norm and no rotation of their own")
         if spec.reads_cache and (spec.value_norm or spec.k_proj is not None or spec.v_proj is not None):
             raise ValueError("a mixer that reads another's keys and values makes none")
+        if spec.reads_cache and (spec.unit_qk or spec.gate is not None):
+            raise ValueError("queries over another's keys have no norm and no gate")
         pairs = [(p, b) for p, b in ((spec.q_proj, spec.q_bias), (spec.k_proj, spec.k_bias), (spec.v_proj, spec.v_bias)) if p is not None]
-        self.w_qkv = torch.cat([weights[p] for p, _ in pairs], dim=0).contiguous()
-        self.bias = None
+        self.qkv_width = sum(weights[p].shape[0] for p, _ in pairs)
+        if spec.gate is not None:
+            pairs.append((spec.gate, None))
+        self.w_in = torch.cat([weights[p] for p, _ in pairs], dim=0).contiguous()
+        self.b_in = None
         if any(b is not None for _, b in pairs):          # float32, zeros where a projection has none
-            self.bias = torch.cat([weights[b].float() if b is not None else
+            self.b_in = torch.cat([weights[b].float() if b is not None else
                                    torch.zeros(weights[p].shape[0], dtype=torch.float32, device=weights[p].device)
                                    for p, b in pairs], dim=0).contiguous()
         self.w_o = weights[spec.o_proj]
@@ -45,7 +55,8 @@ class RotaryValueAttention:
             raise ValueError("the values are rotated over their whole width")
         import os
         self.exact_weights = os.environ.get("INFURNACE_EXACT_ATTENTION", "0") not in ("", "0")
-        self.width = self.w_qkv.shape[0]
+        self.out_width = spec.num_heads * spec.value_head_dim
+        self.joint = not spec.reads_cache                 # may share its products with the mixers beside it
         # what the call of the streams' attention kernel needs beyond the plain softmax
         self.extra = {key: value for key, value in (("softcap", spec.softcap), ("sink", spec.sink_score)) if value is not None}
         if spec.weight_terms != 1:
@@ -55,7 +66,7 @@ class RotaryValueAttention:
 
     def can_take_folded(self, n):
         can = getattr(self.k, "can_fold_norm", None)
-        return bool(can and can(n, self.rt.act_dtype, self.w_qkv))
+        return bool(can and can(n, self.rt.act_dtype, self.w_in))
 
     def _plain_on_tensor_cores(self, kv):
         """bfloat16 with keys and values of one width in one tensor: the framework's tensor-core attention kernels run
@@ -73,30 +84,35 @@ class RotaryValueAttention:
         args = {}
         if row_scale is not None:
             args["row_scale"] = row_scale
-        if self.bias is not None:
-            args["bias"] = self.bias
-        self.k.linear(h, self.w_qkv, out, **args)
+        if self.b_in is not None:
+            args["bias"] = self.b_in
+        self.k.linear(h, self.w_in, out, **args)
 
-    def _queries(self, h, row_scale, ctx, call, kv, v_table):
-        """The step's queries in the cache's dtype; its keys and values, if the part makes any, in the pages."""
+    def _queries(self, proj, ctx, call, kv, v_table):
+        """The step's queries in the cache's dtype; its keys and values in the pages."""
         s, k = self.spec, self.k
-        n = h.shape[0]
+        n = proj.shape[0]
         pk, pv = kv.streams["k"], kv.streams["v"]
         q = ctx.buffer("rva_q", (n, s.num_heads * s.head_dim), self.rt.act_dtype)
         qk_table = self.position.table(ctx) if self.position is not None else None
-        if s.reads_cache:
-            self._project(h, row_scale, q)
-            if qk_table is not None:
-                k.rotate_rows(q, qk_table, s.num_heads, s.head_dim, s.position.rotary_dim, bool(s.position.interleaved))
-            return q
-        qkv = ctx.buffer("rva_qkv", (n, self.width), torch.float32)
-        self._project(h, row_scale, qkv)
-        k.rotary_store(qkv, s.num_heads, s.num_kv_heads, s.head_dim, s.value_head_dim, qk_table,
+        extra = {"values_are_keys": True} if self.values_are_keys else {}
+        if s.unit_qk:
+            extra["qk_eps"] = s.eps
+        k.rotary_store(proj[:, :self.qkv_width], s.num_heads, s.num_kv_heads, s.head_dim, s.value_head_dim, qk_table,
                        s.position.rotary_dim if s.position is not None else 0,
                        bool(s.position.interleaved) if s.position is not None else False,
                        s.eps if s.value_norm else None, v_table,
                        bool(s.value_position.interleaved) if s.value_position is not None else False,
-                       q, pk, pv, kv.slot_mapping if call.store else None, **({"values_are_keys": True} if self.values_are_keys else {}))
+                       q, pk, pv, kv.slot_mapping if call.store else None, **extra)
+        return q
+
+    def _queries_alone(self, h, row_scale, ctx):
+        """The queries of a part that makes no keys: their product writes the cache's dtype."""
+        s, k = self.spec, self.k
+        q = ctx.buffer("rva_q", (h.shape[0], s.num_heads * s.head_dim), self.rt.act_dtype)
+        self._project(h, row_scale, q)
+        if self.position is not None:
+            k.rotate_rows(q, self.position.table(ctx), s.num_heads, s.head_dim, s.position.rotary_dim, bool(s.position.interleaved))
         return q
 
     def forward(self, h, ctx, call, fold=None, out=None):
@@ -105,11 +121,37 @@ class RotaryValueAttention:
         s, k = self.spec, self.k
         h, row_scale = unfolded(h)
         n = h.shape[0]
+        attn = ctx.buffer("rva_out", (n, self.out_width), self.rt.act_dtype)
+        if s.reads_cache:
+            self._attend(self._queries_alone(h, row_scale, ctx), attn, ctx, ctx.kv(call.cache),
+                         self.value_position.table(ctx) if self.value_position is not None else None)
+        else:
+            proj = ctx.buffer("rva_proj", (n, self.w_in.shape[0]), torch.float32)
+            self._project(h, row_scale, proj)
+            self.mix(proj, ctx, call, attn)
+        folded = fold_residual_norm(k, ctx, "mixer", attn, self.w_o, fold, self.rt.act_dtype)
+        if folded is not None:
+            return folded
+        delta = out if out is not None else ctx.buffer("delta_mixer", (n, s.hidden_size), torch.float32)
+        k.linear(attn, self.w_o, delta)
+        return delta
+
+    def mix(self, proj, ctx, call, out, gain=1.0):
+        """From the input product's rows (``proj`` [n, rows of w_in], maybe a slice of a wider product) to the rows that the
+        output product reads: ``gain`` times the (gated) heads into ``out``, whose rows may be a slice too."""
+        s, k = self.spec, self.k
         kv = ctx.kv(call.cache)
-        pk, pv = kv.streams["k"], kv.streams["v"]
         v_table = self.value_position.table(ctx) if self.value_position is not None else None
-        q = self._queries(h, row_scale, ctx, call, kv, v_table)
-        attn = ctx.buffer("rva_out", (n, s.num_heads * s.value_head_dim), self.rt.act_dtype)
+        q = self._queries(proj, ctx, call, kv, v_table)
+        direct = s.gate is None and gain == 1.0 and out.is_contiguous()
+        heads = out if direct else ctx.buffer("rva_heads", (proj.shape[0], self.out_width), self.rt.act_dtype)
+        self._attend(q, heads, ctx, kv, v_table)
+        if not direct:
+            k.norm_gate_rows(heads, out, gate=proj[:, self.qkv_width:] if s.gate is not None else None, activation="sigmoid", scale=gain)
+
+    def _attend(self, q, attn, ctx, kv, v_table):
+        s, k = self.spec, self.k
+        pk, pv = kv.streams["k"], kv.streams["v"]
         if self._plain_on_tensor_cores(kv):
             # the framework's tensor-core attention over the entry's one tensor of keys and values, then the turn back
             k.paged_attention(q, s.num_heads, s.num_kv_heads, s.head_dim, kv.pages, kv.block_tables, ctx.cu_q, ctx.seq_lens, attn,
@@ -124,12 +166,6 @@ class RotaryValueAttention:
                                       bool(s.value_position.interleaved) if s.value_position is not None else False,
                                       max_q_len=ctx.max_q_len, max_seq_len=ctx.max_seq_len, min_q_len=ctx.min_q_len,
                                       exact=self.exact_weights, **self.extra)
-        folded = fold_residual_norm(k, ctx, "mixer", attn, self.w_o, fold, self.rt.act_dtype)
-        if folded is not None:
-            return folded
-        delta = out if out is not None else ctx.buffer("delta_mixer", (n, s.hidden_size), torch.float32)
-        k.linear(attn, self.w_o, delta)
-        return delta
 
 
 register_part(RotaryValueAttentionSpec, RotaryValueAttention)

@@ -26,6 +26,22 @@ class ReferenceKernels:
     def embed(self, table, ids, out, scale=1.0):
         out.copy_(table[ids.long()].to(out.dtype) * scale)
 
+    def embed_bigram(self, table, pairs, ids, positions, req_index, cu_q, seq_lens, state_slots, state, buckets, mul_prev, mul_cur, out):
+        """out[t] = table[ids[t]] + pairs[(prev * mul_prev + ids[t] * mul_cur) mod buckets] (row ``buckets`` at position 0);
+        prev is the request's token before t, state[slot] for the first of this step; state[slot] takes the step's last."""
+        out.copy_(table[ids.long()].to(out.dtype))
+        for r in range(seq_lens.numel()):
+            if int(seq_lens[r]) <= 0:
+                continue
+            slot = int(state_slots[r])
+            prev = int(state[slot])
+            for t in range(int(cu_q[r]), int(cu_q[r + 1])):
+                cur = int(ids[t])
+                row = buckets if int(positions[t]) == 0 else (prev * mul_prev + cur * mul_cur) % buckets
+                out[t] += pairs[row].to(out.dtype)
+                prev = cur
+            state[slot] = float(prev)
+
     def random_normal(self, out, seed64, mean, std):
         """out[i] = mean + std * z_i, the counter-based values of weights/random_init.py."""
         from infurnace_b200.weights.random_init import normal_values
@@ -76,6 +92,10 @@ class ReferenceKernels:
             half = y.shape[1] // 2
             g, u = y[:, :half], y[:, half:]
             return g * torch.sigmoid(g) * u
+        if epilogue == "gelu_gate":
+            half = y.shape[1] // 2
+            g, u = y[:, :half], y[:, half:]
+            return 0.5 * g * (1 + torch.tanh(0.7978845608028654 * (g + 0.044715 * g ** 3))) * u
         if epilogue == "relu2":
             return torch.relu(y) ** 2
         if epilogue == "silu":
@@ -358,11 +378,13 @@ class ReferenceKernels:
             last[slot] = cur[-1].to(last.dtype)
 
     def linear_scan(self, q, k, v, w, heads, dim, vdim, state, state_slots, cu_q, seq_lens, out, eps, decay=None, w_bias=None,
-                    key_scale=1.0, bonus=None, norm_weight=None, gate=None, max_q_len=1):
-        """Per request and head, token by token on state[slot] [heads, dim, vdim] (float32): with the decay
+                    key_scale=1.0, bonus=None, norm_weight=None, gate=None, max_q_len=1, activation=None, finish=True):
+        """``activation`` "silu": q, k and v pass it first.  ``finish`` False: out is o itself.  Per request and head, token by token on state[slot] [heads, dim, vdim] (float32): with the decay
         d = decay[head] (constant) or exp(-exp(w + w_bias)) per key channel, kk = k * key_scale:
         without bonus  S = d S + kk v^T, o = S^T q;  with bonus u  o = (S + u kk v^T)^T q, then S = d S + kk v^T.
         out = o / rms(o) per head (* norm_weight [heads * vdim]) (* silu(gate))."""
+        if activation == "silu":
+            q, k, v = (x.to(self.cd) * torch.sigmoid(x.to(self.cd)) for x in (q, k, v))
         for r in range(seq_lens.numel()):
             if int(seq_lens[r]) <= 0:
                 continue
@@ -383,13 +405,85 @@ class ReferenceKernels:
                 else:
                     S = d[:, :, None] * S + kv
                     o = torch.einsum("hde,hd->he", S, qt)
-                o = (o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps)).reshape(heads * vdim)
+                if finish:
+                    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+                o = o.reshape(heads * vdim)
                 if norm_weight is not None:
                     o = o * norm_weight.to(self.cd)
                 if gate is not None:
                     g = gate[t].to(self.cd)
                     o = o * g * torch.sigmoid(g)
                 out[t] = o.to(out.dtype)
+            state[slot] = S.to(state.dtype)
+
+    def norm_gate_rows(self, x, out, groups=1, weight=None, eps=None, gate=None, activation="sigmoid", scale=1.0):
+        """out = scale * norm(x) * act(gate): the norm (eps None: none) divides each of ``groups`` equal parts of a row by its
+        own root mean square and multiplies by ``weight`` (of the row's length, or of a part's, shared by the parts)."""
+        n, width = x.shape
+        y = x.to(self.cd).view(n, groups, width // groups)
+        if eps is not None:
+            y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+        if weight is not None:
+            y = y * weight.to(self.cd).view(-1, width // groups)
+        y = y.reshape(n, width) * scale
+        if gate is not None:
+            g = gate.to(self.cd)
+            y = y * torch.sigmoid(g) * (g if activation == "silu" else 1.0)
+        out.copy_(y.to(out.dtype))
+
+    def delta_prepare(self, proj, kv_heads, heads, dim, vdim, taps_weight, unit_eps, state, state_slots, cu_q, seq_lens, req_index, qkv,
+                      beta, low, low_width):
+        """proj rows hold q | k | v | beta | bottlenecks.  Per request: y_t = silu(sum_j w[:, j] x_(t - taps + 1 + j)) over its
+        tokens, the inputs before the step's first from state[slot] [taps - 1, channels], which takes the last ones; q and k
+        heads divided by sqrt(sum + unit_eps), q times dim^(-1/2); beta = sigmoid; low = the bottlenecks, zeros beyond."""
+        C, taps = taps_weight.shape
+        kd = kv_heads * dim
+        x = proj[:, :C].to(self.cd)
+        w = taps_weight.to(self.cd)
+        for r in range(seq_lens.numel()):
+            if int(seq_lens[r]) <= 0:
+                continue
+            slot = int(state_slots[r])
+            a, b = int(cu_q[r]), int(cu_q[r + 1])
+            past = state[slot].to(self.cd)[:taps - 1]
+            ext = torch.cat((past, x[a:b]))
+            for t in range(b - a):
+                y = (ext[t:t + taps] * w.t()).sum(0)
+                y = y * torch.sigmoid(y)
+                q, k = y[:kd].view(kv_heads, dim), y[kd:2 * kd].view(kv_heads, dim)
+                q = q / torch.sqrt(q.pow(2).sum(-1, keepdim=True) + unit_eps) * dim ** -0.5
+                k = k / torch.sqrt(k.pow(2).sum(-1, keepdim=True) + unit_eps)
+                qkv[a + t] = torch.cat((q.reshape(-1), k.reshape(-1), y[2 * kd:])).to(qkv.dtype)
+            if taps > 1:
+                state[slot] = ext[ext.shape[0] - (taps - 1):].to(state.dtype)
+        beta.copy_(torch.sigmoid(proj[:, C:C + heads].to(self.cd)).to(beta.dtype))
+        low.zero_()
+        low[:, :low_width] = proj[:, C + heads:C + heads + low_width].to(low.dtype)
+
+    def delta_rule(self, qkv, up, beta, kv_heads, heads, dim, vdim, rate, decay_bias, norm_weight, eps, state, state_slots, cu_q, seq_lens,
+                   out, max_q_len=1):
+        """up rows hold the raw decays [heads * dim] | gates [heads * vdim].  g = exp(-rate_h softplus(raw + decay_bias)); per head on
+        state[slot]: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; out = o / rms(o) * norm_weight * sigmoid(gate)."""
+        kd, rep = kv_heads * dim, heads // kv_heads
+        cd = self.cd
+        for r in range(seq_lens.numel()):
+            if int(seq_lens[r]) <= 0:
+                continue
+            slot = int(state_slots[r])
+            S = state[slot].to(cd)
+            for t in range(int(cu_q[r]), int(cu_q[r + 1])):
+                row = qkv[t].to(cd)
+                q = row[:kd].view(kv_heads, dim).repeat_interleave(rep, dim=0)
+                k = row[kd:2 * kd].view(kv_heads, dim).repeat_interleave(rep, dim=0)
+                v = row[2 * kd:].view(heads, vdim)
+                raw = up[t, :heads * dim].to(cd) + decay_bias.to(cd)
+                g = torch.exp(-rate.to(cd)[:, None] * torch.logaddexp(raw, torch.zeros_like(raw)).view(heads, dim))
+                S = S * g[:, :, None]
+                u = beta[t].to(cd)[:, None] * (v - torch.einsum("hde,hd->he", S, k))
+                S = S + k[:, :, None] * u[:, None, :]
+                o = torch.einsum("hde,hd->he", S, q)
+                o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_weight.to(cd)
+                out[t] = (o.reshape(-1) * torch.sigmoid(up[t, heads * dim:].to(cd))).to(out.dtype)
             state[slot] = S.to(state.dtype)
 
     def gated_unit_scan(self, proj, z_bias, x_bias, state, state_slots, cu_q, seq_lens, out, max_q_len=1):
@@ -490,8 +584,8 @@ class ReferenceKernels:
         return pairs[..., 0][:, None, :], pairs[..., 1][:, None, :]
 
     def rotary_store(self, qkv, num_heads, num_kv_heads, head_dim, value_head_dim, qk_table, rotary_dim, interleaved, value_eps,
-                     v_table, v_interleaved, q_out, k_pages, v_pages, slot_mapping, values_are_keys=False):
-        """qkv [n, H d + G d + G dv] ([n, H d + G d] with ``values_are_keys``: a value head is its key head before rotation).  q and k are rotated by the angles of qk_table ([n, rotary_dim] (cos, sin)
+                     v_table, v_interleaved, q_out, k_pages, v_pages, slot_mapping, values_are_keys=False, qk_eps=None):
+        """``qk_eps``: the q and k heads are divided by their root mean square after the rotation.  qkv [n, H d + G d + G dv] ([n, H d + G d] with ``values_are_keys``: a value head is its key head before rotation).  q and k are rotated by the angles of qk_table ([n, rotary_dim] (cos, sin)
         pairs; None: not rotated); each value head is divided by its root mean square (value_eps None: not) and
         rotated over its whole width by v_table (None: not).  q_out gets q; k and v go to their pages
         [pages, G, page_size, width] at slot_mapping (None: nothing is stored)."""
@@ -502,6 +596,8 @@ class ReferenceKernels:
         if qk_table is not None:
             c, s_ = self._table(qk_table)
             q, k = self._turn(q, c, s_, rotary_dim, interleaved), self._turn(k, c, s_, rotary_dim, interleaved)
+        if qk_eps is not None:
+            q, k = (x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + qk_eps) for x in (q, k))
         if value_eps is not None:
             v = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + value_eps)
         if v_table is not None:
