@@ -1,6 +1,7 @@
 // Softmax attention whose values carry positions, over page streams that may differ in width.
 //
-// (1) rotary_store: per token, the q and k heads are rotated on their first rot_dims entries by the token's angles,
+// (1) rotary_store: per token, the q and k heads are rotated on their first rot_dims entries by the token's angles and
+// (optional) divided by their root mean square after that,
 // each value head is divided by its root mean square (optional) and rotated over its whole width by the token's
 // angles (optional); q goes to a row buffer, k and v into their page streams at the token's slot.  Where a model has no
 // value projection the values are the key heads as projected, before their rotation.  The angles come
@@ -39,7 +40,7 @@ __global__ void __launch_bounds__(128)
 rotary_store_kernel(const float* __restrict__ qkv, int ld, int H, int G, int d, int dv, const float* __restrict__ qk_table,
                     int rot_dims, int interleaved, int v_norm, float v_eps, const float* __restrict__ v_table, int v_interleaved,
                     T* __restrict__ q_out, T* __restrict__ k_pages, long long k_page_stride, T* __restrict__ v_pages,
-                    long long v_page_stride, const int* __restrict__ slot_mapping, int page_size, int v_from_k) {
+                    long long v_page_stride, const int* __restrict__ slot_mapping, int page_size, int v_from_k, int qk_norm, float qk_eps) {
   ifb_pdl_wait();
   ifb_pdl_trigger();
   const int n = blockIdx.x;
@@ -48,7 +49,18 @@ rotary_store_kernel(const float* __restrict__ qkv, int ld, int H, int G, int d, 
   const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
   const float* qt = qk_table ? qk_table + (size_t)n * rot_dims : nullptr;
   const int dims = qt ? rot_dims : 0;
-  for (int idx = threadIdx.x; idx < (H + G) * d; idx += blockDim.x) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  for (int head = warp; qk_norm && head < H + G; head += warps) {          // a warp per head
+    const float* x = row + (size_t)head * d;
+    float ss = 0.f;
+    for (int j = lane; j < d; j += 32) { const float y = as_rotated(x, j, dims, interleaved, qt, 1.f, 1.f); ss = fmaf(y, y, ss); }
+    const float gain = 1.f / sqrtf(warp_sum(ss) / (float)d + qk_eps);
+    if (head >= H && slot < 0) continue;
+    T* dst = head < H ? q_out + (size_t)n * H * d + (size_t)head * d
+                      : k_pages + (size_t)page * k_page_stride + ((size_t)(head - H) * page_size + off) * d;
+    for (int j = lane; j < d; j += 32) dst[j] = from_f32<T>(as_rotated(x, j, dims, interleaved, qt, 1.f, 1.f) * gain);
+  }
+  for (int idx = threadIdx.x; !qk_norm && idx < (H + G) * d; idx += blockDim.x) {
     const int head = idx / d, j = idx % d;
     const float y = as_rotated(row + (size_t)head * d, j, dims, interleaved, qt, 1.f, 1.f);
     if (head < H) q_out[(size_t)n * H * d + idx] = from_f32<T>(y);
@@ -56,7 +68,6 @@ rotary_store_kernel(const float* __restrict__ qkv, int ld, int H, int G, int d, 
       k_pages[(size_t)page * k_page_stride + ((size_t)(head - H) * page_size + off) * d + j] = from_f32<T>(y);
   }
   if (slot < 0) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const float* vt = v_table ? v_table + (size_t)n * dv : nullptr;
   for (int g = warp; g < G; g += warps) {
     // v_from_k: the row holds no values; a value head is the key head as projected, before its rotation (dv == d)
@@ -75,18 +86,19 @@ rotary_store_kernel(const float* __restrict__ qkv, int ld, int H, int G, int d, 
 IFB_EXPORT int ifb_rotary_store(const float* qkv, int ld, int H, int G, int d, int dv, const float* qk_table, int rot_dims,
                                 int interleaved, int v_norm, float v_eps, const float* v_table, int v_interleaved, void* q_out,
                                 int dtype, void* k_pages, long long k_page_stride, void* v_pages, long long v_page_stride,
-                                const int* slot_mapping, int page_size, int n, int v_from_k, cudaStream_t stream) {
+                                const int* slot_mapping, int page_size, int n, int v_from_k, int qk_norm, float qk_eps,
+                                cudaStream_t stream) {
   if (n <= 0) return IFB_OK;
   if (H < 1 || G < 1 || d < 1 || dv < 1 || page_size < 1 || (v_from_k && dv != d)) return IFB_ERR_SIZE;
   if ((qk_table && (rot_dims < 2 || rot_dims % 2 || rot_dims > d)) || (v_table && dv % 2)) return IFB_ERR_ARG;
   if (dtype == IFB_BF16)
     return ifb_launch(rotary_store_kernel<__nv_bfloat16>, dim3(n), dim3(128), 0, stream, qkv, ld, H, G, d, dv, qk_table, rot_dims,
                       interleaved, v_norm, v_eps, v_table, v_interleaved, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pages,
-                      k_page_stride, (__nv_bfloat16*)v_pages, v_page_stride, slot_mapping, page_size, v_from_k);
+                      k_page_stride, (__nv_bfloat16*)v_pages, v_page_stride, slot_mapping, page_size, v_from_k, qk_norm, qk_eps);
   if (dtype != IFB_F32) return IFB_ERR_DTYPE;
   return ifb_launch(rotary_store_kernel<float>, dim3(n), dim3(128), 0, stream, qkv, ld, H, G, d, dv, qk_table, rot_dims, interleaved,
                     v_norm, v_eps, v_table, v_interleaved, (float*)q_out, (float*)k_pages, k_page_stride, (float*)v_pages,
-                    v_page_stride, slot_mapping, page_size, v_from_k);
+                    v_page_stride, slot_mapping, page_size, v_from_k, qk_norm, qk_eps);
 }
 
 // rows[n][head][:] are rotated in place by the token's angles, forward (sign 1) or back (sign -1), over `dims` entries

@@ -7,7 +7,7 @@
 //     with a bonus u[i]  o[c] = sum_i (S[i][c] + u[i] k[i] v[c]) q[i];   then S[i][c] = d[i] S[i][c] + k[i] v[c]
 // (the output is read BEFORE the update and the token's own k v^T enters it through the bonus only).  The decay is
 // either one constant per head (retention) or exp(-exp(w[i] + bias[i])) from a raw per-token row (RWKV-style time
-// mixing); keys are multiplied by key_scale.  Then out[c] = o[c] / sqrt(mean_c(o^2) + eps) (* norm_w[head][c])
+// mixing); keys are multiplied by key_scale; q, k and v may pass silu first.  Then (unless the caller takes o itself) out[c] = o[c] / sqrt(mean_c(o^2) + eps) (* norm_w[head][c])
 // (* silu(gate[c])).  The sum with the bonus splits into sum_i S[i][c] q[i] + v[c] * (sum_i u[i] k[i] q[i]); the
 // second factor is one number per token and head, formed when the token is staged.
 //
@@ -50,11 +50,15 @@ struct LinearScanArgs {
   void* out;                             // [tokens][heads * vdim], T
   float* raw;                            // [tokens][heads * vdim]: outputs before the finish, when a head has several slabs
   int heads, dim, vdim, slabs;
+  int silu;                              // q, k and v pass silu as they are read
+  int plain;                             // the outputs are o itself, float32, written to raw (= out)
   int mode;                              // 0: a request per block row, from and to its slot.  1: launch A.  2: launch C.
   int requests;
   float* z;                              // [blocks][heads][dim][vdim]
   float* dprod;                          // [blocks][heads][dim]
 };
+
+__device__ __forceinline__ float ls_in(const LinearScanArgs& a, float x) { return a.silu ? x / (1.f + expf(-x)) : x; }
 
 __device__ __forceinline__ bool ls_find_block(const LinearScanArgs& a, int row, int& r, int& t0, int& t1) {
   for (int i = 0; i < a.requests; ++i) {
@@ -137,8 +141,8 @@ linear_scan_kernel(LinearScanArgs a) {
       float qv = 0.f, kv = 0.f, dv = 1.f;
       if (i < dim) {
         const size_t tok = (size_t)(g0 + t);
-        qv = a.q[tok * a.ldq + h * dim + i];
-        kv = a.k[tok * a.ldk + h * dim + i] * a.key_scale;
+        qv = ls_in(a, a.q[tok * a.ldq + h * dim + i]);
+        kv = ls_in(a, a.k[tok * a.ldk + h * dim + i]) * a.key_scale;
         dv = a.decay ? head_decay
                      : expf(-expf(a.w[tok * a.ldw + h * dim + i] + load_as_f32(a.w_bias, a.p_dtype, (size_t)h * dim + i)));
       }
@@ -148,7 +152,7 @@ linear_scan_kernel(LinearScanArgs a) {
     }
     for (int idx = threadIdx.x; idx < cnt * width; idx += blockDim.x) {
       const int t = idx / width, e = idx % width;
-      vs[t * blockDim.x + e] = a.v[(size_t)(g0 + t) * a.ldv + h * vdim + c0 + e];
+      vs[t * blockDim.x + e] = ls_in(a, a.v[(size_t)(g0 + t) * a.ldv + h * vdim + c0 + e]);
     }
     __syncthreads();
     if (BONUS)                                   // b_t = sum_i u[i] k[i] q[i], a warp per token
@@ -262,8 +266,8 @@ linear_scan_split_kernel(LinearScanArgs a) {
       float qv = 0.f, kv = 0.f, dv = 1.f;
       if (i < dim) {
         const size_t tok = (size_t)(g0 + t);
-        qv = a.q[tok * a.ldq + h * dim + i];
-        kv = a.k[tok * a.ldk + h * dim + i] * a.key_scale;
+        qv = ls_in(a, a.q[tok * a.ldq + h * dim + i]);
+        kv = ls_in(a, a.k[tok * a.ldk + h * dim + i]) * a.key_scale;
         dv = a.decay ? head_decay
                      : expf(-expf(a.w[tok * a.ldw + h * dim + i] + load_as_f32(a.w_bias, a.p_dtype, (size_t)h * dim + i)));
       }
@@ -273,7 +277,7 @@ linear_scan_split_kernel(LinearScanArgs a) {
     }
     for (int idx = threadIdx.x; idx < cnt * width; idx += blockDim.x) {
       const int t = idx / width, e = idx % width;
-      vs[t * cols + e] = a.v[(size_t)(g0 + t) * a.ldv + h * vdim + c0 + e];
+      vs[t * cols + e] = ls_in(a, a.v[(size_t)(g0 + t) * a.ldv + h * vdim + c0 + e]);
     }
     __syncthreads();
     if (BONUS)                                   // b_t = sum_i u[i] k[i] q[i], a warp per token
@@ -402,15 +406,15 @@ linear_scan_wide_kernel(LinearScanArgs a) {
   for (int t = a.cu_q[r]; t < a.cu_q[r + 1]; ++t) {
     float bpart = 0.f;
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-      qs[i] = a.q[(size_t)t * a.ldq + h * dim + i];
-      ks[i] = a.k[(size_t)t * a.ldk + h * dim + i] * a.key_scale;
+      qs[i] = ls_in(a, a.q[(size_t)t * a.ldq + h * dim + i]);
+      ks[i] = ls_in(a, a.k[(size_t)t * a.ldk + h * dim + i]) * a.key_scale;
       ds[i] = a.decay ? a.decay[h]
                       : expf(-expf(a.w[(size_t)t * a.ldw + h * dim + i] + load_as_f32(a.w_bias, a.p_dtype, (size_t)h * dim + i)));
       if (a.bonus) bpart += load_as_f32(a.bonus, a.p_dtype, (size_t)h * dim + i) * ks[i] * qs[i];
     }
     const float b = block_sum(bpart, scratch);       // also orders the staging before the walk
     for (int c = threadIdx.x; c < vdim; c += blockDim.x) {
-      const float v = a.v[(size_t)t * a.ldv + h * vdim + c];
+      const float v = ls_in(a, a.v[(size_t)t * a.ldv + h * vdim + c]);
       float o = 0.f;
       for (int i = 0; i < dim; ++i) {
         const float old = S[(size_t)i * vdim + c];
@@ -421,7 +425,8 @@ linear_scan_wide_kernel(LinearScanArgs a) {
       os[c] = a.bonus ? fmaf(v, b, o) : o;
     }
     __syncthreads();
-    if (threadIdx.x < 32) ls_finish<T>(a, os, t, h, lane);
+    if (a.plain) for (int c = threadIdx.x; c < vdim; c += blockDim.x) a.raw[((size_t)t * a.heads + h) * vdim + c] = os[c];
+    else if (threadIdx.x < 32) ls_finish<T>(a, os, t, h, lane);
     __syncthreads();
   }
 }
@@ -461,7 +466,7 @@ static int ls_launch(LinearScanArgs a, int requests, int tokens, cudaStream_t s)
   const bool split = ls_row_split(a.dim, a.vdim) == 2;
   a.slabs = (a.vdim + threads - 1) / threads;
   if (a.slabs > 1 && !a.raw) return IFB_ERR_ARG;
-  if (a.slabs == 1) a.raw = nullptr;
+  if (a.slabs == 1 && !a.plain) a.raw = nullptr;
   dim3 grid(a.heads * a.slabs, a.mode == 0 ? requests : (tokens + LS_BLOCK - 1) / LS_BLOCK + requests);
   int st = IFB_ERR_SIZE;
   bool done = false;
@@ -492,7 +497,7 @@ static int ls_launch(LinearScanArgs a, int requests, int tokens, cudaStream_t s)
   LS_CASE(16) LS_CASE(32) LS_SPLIT(64) LS_CASE(64) LS_SPLIT(128) LS_CASE(128)
 #undef LS_CASE
 #undef LS_SPLIT
-  if (st != IFB_OK || a.slabs == 1 || a.mode == 1) return st;
+  if (st != IFB_OK || a.slabs == 1 || a.mode == 1 || a.plain) return st;
   const long long items = (long long)tokens * a.heads;
   return ifb_launch(linear_scan_finish_kernel<T>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, s, a, items);
 }
@@ -529,18 +534,21 @@ static int ls_run(LinearScanArgs a, int requests, int tokens, float* scratch, cu
 // q, k, v, w, gate: float32 rows with their own leading dimensions.  Exactly one of decay (with w and w_bias null) and
 // (w, w_bias) is given.  bonus, norm_w and gate may be null; w_bias, bonus and norm_w share one dtype.  raw: float32
 // [tokens][heads * vdim] scratch, needed when ifb_linear_scan_slabs(dim, vdim) > 1.  scratch: null for the one-launch
-// walk; else ifb_linear_scan_scratch_floats(...) floats for the three-launch form.
+// walk; else ifb_linear_scan_scratch_floats(...) floats for the three-launch form.  silu: q, k and v pass it first.  plain: out
+// (float32) is o itself, and there is no norm and no gate.
 IFB_EXPORT int ifb_linear_scan(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* w, int ldw,
                                const float* gate, int ldg, const float* decay, const void* w_bias, const void* bonus,
                                const void* norm_w, int p_dtype, float key_scale, float eps, float* state, const int* state_slots,
                                const int* cu_q, const int* seq_lens, void* out, int out_dtype, float* raw, float* scratch,
-                               int requests, int tokens, int heads, int dim, int vdim, cudaStream_t stream) {
+                               int requests, int tokens, int heads, int dim, int vdim, int silu, int plain, cudaStream_t stream) {
   if (requests <= 0 || tokens <= 0) return IFB_OK;
   if (heads < 1 || dim < 1 || vdim < 1 || requests > 65535) return IFB_ERR_SIZE;
+  if (plain && (out_dtype != IFB_F32 || norm_w || gate)) return IFB_ERR_ARG;
+  if (plain) raw = (float*)out;
   if (p_dtype != IFB_F32 && p_dtype != IFB_BF16) return IFB_ERR_DTYPE;
   if ((decay != nullptr) == (w != nullptr) || (w != nullptr) != (w_bias != nullptr)) return IFB_ERR_ARG;
   LinearScanArgs a{q, k, v, w, gate, ldq, ldk, ldv, ldw, ldg, decay, w_bias, bonus, norm_w, p_dtype, key_scale, eps, state,
-                   state_slots, cu_q, seq_lens, out, raw, heads, dim, vdim, 1, 0, requests, nullptr, nullptr};
+                   state_slots, cu_q, seq_lens, out, raw, heads, dim, vdim, 1, silu, plain, 0, requests, nullptr, nullptr};
   if (out_dtype == IFB_F32)
     return bonus ? ls_run<float, true>(a, requests, tokens, scratch, stream) : ls_run<float, false>(a, requests, tokens, scratch, stream);
   if (out_dtype == IFB_BF16)

@@ -119,6 +119,9 @@ class CudaKernels:
         self.gated_unit_chunked_calls = 0
         self._rg_scratch = None
         self.rglru_chunked_calls = 0
+        self._dr_scratch = None
+        self.delta_chunked_calls = 0
+        self.delta_chunk_min = int(os.environ.get("INFURNACE_DELTA_CHUNK_MIN", "33"))      # tokens of the longest request from
         self.moe_tensor_cores = os.environ.get("INFURNACE_MOE_MMA", "1") != "0"
         self.moe_tcgen05 = os.environ.get("INFURNACE_MOE_TCGEN05", "1") != "0"     # prompts' expert products on tcgen05
         self.moe_tcgen05_calls = 0
@@ -941,14 +944,27 @@ class CudaKernels:
             m.ifb_linear_scan.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
                                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p,
                                           c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                          c_int, c_void_p]
+                                          c_int, c_int, c_int, c_void_p]
+            m.ifb_delta_prepare.argtypes = [c_void_p, c_longlong, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p,
+                                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                            c_int, c_int, c_int, c_void_p]
+            m.ifb_delta_rule_slabs.argtypes = [c_int, c_int]
+            m.ifb_delta_rule_scratch_floats.restype = c_longlong
+            m.ifb_delta_rule_scratch_floats.argtypes = [c_int, c_int, c_int, c_int, c_int]
+            m.ifb_delta_rule.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+                                         c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                         c_int, c_int, c_int, c_void_p]
+            m.ifb_embed_bigram.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                           c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]
+            m.ifb_norm_gate_rows.argtypes = [c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_float, c_void_p, c_longlong, c_int,
+                                             c_float, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p]
             m.ifb_gated_unit_scan.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                               c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
             m.ifb_gated_unit_scratch_floats.restype = c_longlong
             m.ifb_gated_unit_scratch_floats.argtypes = [c_int, c_int, c_int]
             m.ifb_rotary_store.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float,
                                            c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p,
-                                           c_int, c_int, c_int, c_void_p]
+                                           c_int, c_int, c_int, c_int, c_float, c_void_p]
             m.ifb_rotate_rows.argtypes = [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
             m.ifb_paged_attention_streams.argtypes = [c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int,
                                                       c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -1061,12 +1077,13 @@ class CudaKernels:
         return t.data_ptr(), t.stride(0)
 
     def linear_scan(self, q, k, v, w, heads, dim, vdim, state, state_slots, cu_q, seq_lens, out, eps, decay=None, w_bias=None,
-                    key_scale=1.0, bonus=None, norm_weight=None, gate=None, max_q_len=1):
+                    key_scale=1.0, bonus=None, norm_weight=None, gate=None, max_q_len=1, activation=None, finish=True):
         """The recurrence of a matrix state per head over this step's tokens of every request (csrc/linear_scan.cu).
         q, k, w [n, heads * dim], v, gate [n, heads * vdim]: float32, may be column slices.  ``decay`` float32 [heads]:
         a constant decay per head; else the decay is exp(-exp(w + w_bias)).  ``bonus`` [heads * dim]: the output is read
         before the token's update, the token's own k v^T weighted by the bonus.  out = o / rms(o) per head
-        (* norm_weight [heads * vdim]) (* silu(gate)).  From ``scan_block_min`` tokens on the requests are cut into blocks
+        (* norm_weight [heads * vdim]) (* silu(gate)); ``finish`` False: out (float32) is o itself.  ``activation`` "silu": q, k
+        and v pass it first.  From ``scan_block_min`` tokens on the requests are cut into blocks
         of 64 tokens that run side by side (three launches)."""
         n = out.shape[0]
         r = seq_lens.numel()
@@ -1078,6 +1095,8 @@ class CudaKernels:
         pg = self._rows_f32(gate, "gate", n, hv) if gate is not None else (0, 0)
         if (decay is None) == (w is None) or (w is None) != (w_bias is None):
             raise KernelError("linear_scan: give either decay, or w with w_bias")
+        if activation not in (None, "silu") or (not finish and (norm_weight is not None or gate is not None or out.dtype != torch.float32)):
+            raise KernelError("linear_scan: the activation is silu or none; outputs without finish are float32, without norm and gate")
         if decay is not None and _dense(decay, "decay", torch.float32).numel() != heads:
             raise KernelError("linear_scan: decay has one number per head")
         pdt = None
@@ -1093,7 +1112,7 @@ class CudaKernels:
         lib = self._hyb_lib()
         raw = None
         slabs = int(lib.ifb_linear_scan_slabs(dim, vdim))
-        need = n * hv if slabs > 1 else 0
+        need = n * hv if slabs > 1 and finish else 0
         scratch = 0
         blocked = max_q_len >= self.scan_block_min and dim <= 128
         if blocked:
@@ -1104,12 +1123,115 @@ class CudaKernels:
                 self._ls_scratch = torch.empty(need + scratch, dtype=torch.float32, device="cuda")
                 self.scratch_generation += 1
             raw = self._ls_scratch[:need] if need else None
-        self.launches += (3 if blocked else 1) + (1 if slabs > 1 else 0)
+        self.launches += (3 if blocked else 1) + (1 if need else 0)
         _check(lib.ifb_linear_scan(
             pq[0], pq[1], pk[0], pk[1], pv[0], pv[1], pw[0], pw[1], pg[0], pg[1], _ptr(decay), _ptr(w_bias), _ptr(bonus),
             _ptr(norm_weight), _CODES[pdt] if pdt is not None else 0, float(key_scale), float(eps), state.data_ptr(),
             state_slots.data_ptr(), cu_q.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), _code(out), _ptr(raw),
-            self._ls_scratch[need:].data_ptr() if blocked else 0, r, n, heads, dim, vdim, self._stream()), "linear_scan")
+            self._ls_scratch[need:].data_ptr() if blocked else 0, r, n, heads, dim, vdim, 1 if activation == "silu" else 0,
+            0 if finish else 1, self._stream()), "linear_scan")
+
+    def norm_gate_rows(self, x, out, groups=1, weight=None, eps=None, gate=None, activation="sigmoid", scale=1.0):
+        """out = scale * norm(x) * act(gate), row by row in float32 (csrc/rows.cu).  The norm (``eps`` None: none) divides each of
+        ``groups`` equal parts of a row by its own root mean square and multiplies by ``weight`` (float32, of the row's length or,
+        shared by the parts, of a part's).  ``gate`` float32; ``activation`` "sigmoid" or "silu".  Rows of x, gate and out may be
+        slices of wider rows."""
+        n, width = x.shape
+        for t, name in ((x, "x"), (out, "out"), (gate, "gate")):
+            if t is not None and (not t.is_cuda or t.shape != (n, width) or (width > 1 and t.stride(1) != 1)):
+                raise KernelError(f"norm_gate_rows: {name} has x's shape and unit stride along the row")
+        if gate is not None and gate.dtype != torch.float32 or activation not in ("sigmoid", "silu"):
+            raise KernelError("norm_gate_rows: gate is float32, its function sigmoid or silu")
+        if groups < 1 or width % groups:
+            raise KernelError("norm_gate_rows: groups divides the row")
+        if weight is not None and _dense(weight, "weight", torch.float32).numel() not in (width, width // groups):
+            raise KernelError("norm_gate_rows: weight has the length of a row or of a part")
+        shared = weight is not None and weight.numel() != width
+        self.launches += 1
+        _check(self._hyb_lib().ifb_norm_gate_rows(
+            x.data_ptr(), _code(x), x.stride(0), _ptr(weight), int(shared), 0 if eps is None else 1, float(eps or 0.0), _ptr(gate),
+            gate.stride(0) if gate is not None else 0, int(activation == "silu"), float(scale), out.data_ptr(), _code(out), out.stride(0),
+            n, width, int(groups), self._stream()), "norm_gate_rows")
+
+    def embed_bigram(self, table, pairs, ids, positions, req_index, cu_q, seq_lens, state_slots, state, buckets, mul_prev, mul_cur, out):
+        """out[t] = table[ids[t]] + pairs[(prev * mul_prev + ids[t] * mul_cur) mod buckets], the row ``buckets`` at position 0
+        (csrc/rows.cu); prev is the request's token before t, state[slot] for its first of the step, which then takes its last."""
+        _dense(table, "table"), _dense(pairs, "pairs", table.dtype), _dense(out, "out", torch.float32), _dense(state, "state", torch.float32)
+        for t, name in ((ids, "ids"), (positions, "positions"), (req_index, "req_index"), (cu_q, "cu_q"), (seq_lens, "seq_lens"),
+                        (state_slots, "state_slots")):
+            _dense(t, name, torch.int32)
+        n, hidden = out.shape
+        if table.shape[1] != hidden or pairs.shape != (buckets + 1, hidden) or ids.numel() != n or positions.numel() != n \
+                or req_index.numel() != n or cu_q.numel() != seq_lens.numel() + 1 or state_slots.numel() < seq_lens.numel():
+            raise KernelError("embed_bigram: sizes of the tables, ids, request arrays and out do not match")
+        self.launches += 1
+        self._err_armed = True
+        _check(self._hyb_lib().ifb_embed_bigram(
+            table.data_ptr(), pairs.data_ptr(), _code(table), ids.data_ptr(), positions.data_ptr(), req_index.data_ptr(), cu_q.data_ptr(),
+            seq_lens.data_ptr(), state_slots.data_ptr(), state.data_ptr(), int(buckets), int(mul_prev) % int(buckets),
+            int(mul_cur) % int(buckets), out.data_ptr(), n, hidden, table.shape[0], self._dev_err.data_ptr(), self._stream()),
+            "embed_bigram")
+
+    def delta_prepare(self, proj, kv_heads, heads, dim, vdim, taps_weight, unit_eps, state, state_slots, cu_q, seq_lens, req_index, qkv,
+                      beta, low, low_width):
+        """From the input product's rows q | k | v | beta | bottlenecks (proj, float32): the short causal convolutions with silu,
+        q and k heads as unit vectors, q times dim^(-1/2) -> qkv [n, channels] float32; sigmoid -> beta [n, heads]; the
+        bottlenecks in the products' dtype, zeros beyond ``low_width``, -> low (csrc/delta_rule.cu).  taps_weight
+        [channels, taps] float32; state [slots, max(taps - 1, 1), channels]: the inputs before a portion, then its last ones."""
+        _dense(proj, "proj", torch.float32), _dense(taps_weight, "taps_weight", torch.float32), _dense(state, "state", torch.float32)
+        _dense(qkv, "qkv", torch.float32), _dense(beta, "beta", torch.float32), _dense(low, "low")
+        for t, name in ((state_slots, "state_slots"), (cu_q, "cu_q"), (seq_lens, "seq_lens"), (req_index, "req_index")):
+            _dense(t, name, torch.int32)
+        n = proj.shape[0]
+        C, taps = taps_weight.shape
+        if C != 2 * kv_heads * dim + heads * vdim or proj.shape[1] != C + heads + low_width or qkv.shape != (n, C) \
+                or beta.shape != (n, heads) or low.shape[0] != n or low.shape[1] < low_width or state.shape[1:] != (max(taps - 1, 1), C) \
+                or req_index.numel() != n or cu_q.numel() != seq_lens.numel() + 1 or state_slots.numel() < seq_lens.numel():
+            raise KernelError("delta_prepare: sizes of proj, taps_weight, state, qkv, beta and low do not match")
+        self.launches += 1
+        _check(self._hyb_lib().ifb_delta_prepare(
+            proj.data_ptr(), proj.shape[1], taps_weight.data_ptr(), taps, float(unit_eps), float(dim) ** -0.5, state.data_ptr(),
+            state_slots.data_ptr(), cu_q.data_ptr(), seq_lens.data_ptr(), req_index.data_ptr(), qkv.data_ptr(), beta.data_ptr(),
+            low.data_ptr(), _code(low), int(low_width), low.shape[1], n, kv_heads, heads, dim, vdim, self._stream()), "delta_prepare")
+
+    def delta_rule(self, qkv, up, beta, kv_heads, heads, dim, vdim, rate, decay_bias, norm_weight, eps, state, state_slots, cu_q, seq_lens,
+                   out, max_q_len=1):
+        """The gated delta rule with a decay per key channel over this step's tokens of every request (csrc/delta_rule.cu).
+        qkv: rows q | k | v as :meth:`delta_prepare` leaves them; up [n, heads * (dim + vdim)] float32: raw decays | gates;
+        g = exp(-rate_h softplus(raw + decay_bias)); out = o / rms(o) per head * norm_weight [vdim] * sigmoid(gate).  state
+        [slots, heads, dim, vdim] float32.  From ``delta_chunk_min`` tokens on the requests are run in chunks of 16 tokens, which
+        differs by rounding only (three launches)."""
+        _dense(qkv, "qkv", torch.float32), _dense(up, "up", torch.float32), _dense(beta, "beta", torch.float32)
+        _dense(state, "state", torch.float32), _dense(out, "out")
+        for t, size, name in ((rate, heads, "rate"), (decay_bias, heads * dim, "decay_bias"), (norm_weight, vdim, "norm_weight")):
+            if _dense(t, name, torch.float32).numel() != size:
+                raise KernelError(f"delta_rule: {name} has {size} numbers")
+        for t, name in ((state_slots, "state_slots"), (cu_q, "cu_q"), (seq_lens, "seq_lens")):
+            _dense(t, name, torch.int32)
+        n, r = out.shape[0], seq_lens.numel()
+        if heads % kv_heads or qkv.shape != (n, 2 * kv_heads * dim + heads * vdim) or up.shape != (n, heads * (dim + vdim)) \
+                or beta.shape != (n, heads) or out.shape != (n, heads * vdim) or state.shape[1:] != (heads, dim, vdim) \
+                or cu_q.numel() != r + 1 or state_slots.numel() < r:
+            raise KernelError("delta_rule: sizes of qkv, up, beta, state, out and the request arrays do not match")
+        lib = self._hyb_lib()
+        chunked = max_q_len >= self.delta_chunk_min and dim <= 256
+        slabs = int(lib.ifb_delta_rule_slabs(dim, vdim))
+        scratch = int(lib.ifb_delta_rule_scratch_floats(n, r, heads, dim, vdim)) if chunked else 0
+        need = n * heads * vdim if chunked or slabs > 1 else 0
+        if need + scratch:
+            if self._dr_scratch is None or self._dr_scratch.numel() < need + scratch:
+                self._dr_scratch = torch.empty(need + scratch, dtype=torch.float32, device="cuda")
+                self.scratch_generation += 1
+        raw = self._dr_scratch[scratch:].data_ptr() if need else 0
+        # two columns per thread halve the reads of shared memory per product, where the blocks still cover the device
+        columns = 2 if r * heads * (-(-vdim // 32)) >= self.sm_count else 1
+        self.delta_chunked_calls += chunked
+        self.launches += 3 if chunked else 2 if need else 1
+        _check(lib.ifb_delta_rule(
+            qkv.data_ptr(), qkv.shape[1], up.data_ptr(), up.shape[1], beta.data_ptr(), rate.data_ptr(), decay_bias.data_ptr(),
+            norm_weight.data_ptr(), float(eps), state.data_ptr(), state_slots.data_ptr(), cu_q.data_ptr(), seq_lens.data_ptr(),
+            out.data_ptr(), _code(out), raw, self._dr_scratch.data_ptr() if chunked else 0, columns, r, n, kv_heads, heads, dim, vdim,
+            self._stream()), "delta_rule")
 
     def gated_unit_scan(self, proj, z_bias, x_bias, state, state_slots, cu_q, seq_lens, out, max_q_len=1):
         """minGRU over this step's tokens of every request: proj [n, 3 width] float32 holds z_raw | x_raw | g
@@ -1209,12 +1331,12 @@ class CudaKernels:
         return t.data_ptr(), t.stride(0), t.shape[2]
 
     def rotary_store(self, qkv, num_heads, num_kv_heads, head_dim, value_head_dim, qk_table, rotary_dim, interleaved, value_eps,
-                     v_table, v_interleaved, q_out, k_pages, v_pages, slot_mapping, values_are_keys=False):
-        """Rotation of q and k, norm and rotation of v, q row and page stores in one launch (csrc/attention_streams.cu).
-        qkv float32 [n, H d + G d + G dv]; tables float32 (cos, sin) pairs per token; value_eps None: no value norm.
+                     v_table, v_interleaved, q_out, k_pages, v_pages, slot_mapping, values_are_keys=False, qk_eps=None):
+        """Rotation of q and k (and, with ``qk_eps``, their division by each head's root mean square after it), norm and rotation of v, q row and page stores in one launch (csrc/attention_streams.cu).
+        qkv float32 [n, H d + G d + G dv], maybe a slice of wider rows; tables float32 (cos, sin) pairs per token; value_eps None: no value norm.
         ``values_are_keys``: qkv is [n, H d + G d] and a value head is its key head before the rotation."""
-        _dense(qkv, "qkv", torch.float32), _dense(q_out, "q_out")
         n = qkv.shape[0]
+        self._rows_f32(qkv, "qkv", n, qkv.shape[1]), _dense(q_out, "q_out")
         H, G, d, dv = num_heads, num_kv_heads, head_dim, value_head_dim
         if qkv.shape[1] != H * d + G * (d + (0 if values_are_keys else dv)) or q_out.shape != (n, H * d) or (values_are_keys and dv != d):
             raise KernelError("rotary_store: widths of qkv and q_out do not match the heads")
@@ -1231,10 +1353,10 @@ class CudaKernels:
                 raise KernelError("rotary_store: the streams differ in page size, or slot_mapping in length")
         self.launches += 1
         _check(self._hyb_lib().ifb_rotary_store(
-            qkv.data_ptr(), qkv.shape[1], H, G, d, dv, _ptr(qk_table), int(rotary_dim), int(bool(interleaved)),
+            qkv.data_ptr(), qkv.stride(0), H, G, d, dv, _ptr(qk_table), int(rotary_dim), int(bool(interleaved)),
             0 if value_eps is None else 1, float(value_eps or 0.0), _ptr(v_table), int(bool(v_interleaved)), q_out.data_ptr(),
-            _code(q_out), pk[0], pk[1], pv[0], pv[1], _ptr(slot_mapping), ps, n, 1 if values_are_keys else 0, self._stream()),
-            "rotary_store")
+            _code(q_out), pk[0], pk[1], pv[0], pv[1], _ptr(slot_mapping), ps, n, 1 if values_are_keys else 0, 0 if qk_eps is None else 1,
+            float(qk_eps or 0.0), self._stream()), "rotary_store")
 
     def rotate_rows(self, rows, table, heads, width, dims, interleaved, back=False):
         """rows [n, heads * width] in place: every head's first ``dims`` entries turned by the token's angles of
