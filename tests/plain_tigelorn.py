@@ -240,3 +240,11 @@ def forward(cfg, weights, tokens, return_layers=False):
         streams.append(x)
     logits = layer_norm(x, w64(weights, "final.norm"), eps) @ w64(weights, "embed").T
     return (logits, torch.stack(streams)) if return_layers else logits
+
+
+def greedy(cfg, weights, prompt, n):
+    """The n tokens that follow ``prompt``, the largest logit each time (the lowest id among equals)."""
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(torch.argmax(forward(cfg, weights, toks)[-1])))
+    return toks[len(prompt):]
