@@ -710,6 +710,37 @@ def parallel_config(size):
             "norm": {"eps": 1e-6}, "vocab": 32768, "width": W}
 
 
+def delta_config(size):
+    """A Tigelorn config.json mapping at the width, depth, head sizes and ACTIVE parameter count of design_configs(size):
+    layers delta rule, latent attention, attention beside linear attention, delta rule, and again; delta-rule heads of
+    128 x 128, four taps, bottlenecks of 128; latent attention as recurrent_config's without its window; attention of the
+    design's heads under a window, rotated whole, beside linear attention with heads of the Kafunex recurrence's shape; a gated
+    dense feed-forward of two thirds of the width (gate, up and down against up and down); 2^16 - 1 pairs of tokens."""
+    W, layers, H, G, d, rh, rd, rv, ff, window = {
+        "s": (1024, 8, 16, 4, 64, 8, 64, 128, 3072, 512),
+        "m": (2048, 8, 16, 4, 128, 16, 64, 128, 6144, 1024),
+        "l": (4096, 8, 32, 8, 128, 32, 64, 128, 12288, 1024),
+    }[size]
+    mlp = {"kind": "dense", "ff": ff * 2 // 3}
+    entries = []
+    for i in range(layers):
+        if i % 4 in (0, 3):
+            entries.append({"type": "channel_delta", "mlp": mlp, "mixer": {
+                "heads": W // 128, "kv_heads": W // 128, "dim": 128, "vdim": 128, "conv": 4, "rank": 128}})
+        elif i % 4 == 1:
+            entries.append({"type": "latent_attention", "mlp": mlp, "mixer": {
+                "heads": H, "dim": d, "rot_dim": d // 4, "vdim": d, "kv_rank": 2 * d, "q_rank": W // 2, "scale": (d + d // 4) ** -0.5,
+                "rot": {"base": 1e6, "dims": d // 4, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}})
+        else:
+            entries.append({"type": "parallel", "mlp": mlp, "mixer": {
+                "left": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": window},
+                         "rot": {"base": 1e6, "dims": d}},
+                "right": {"heads": rh, "dim": rd, "vdim": rv, "decay": [1.0 - 2.0 ** (-3 - 4 * j / max(1, rh - 1)) for j in range(rh)]},
+                "left_scale": 0.7, "right_scale": 0.7}})
+    return {"architecture": "Tigelorn", "embedding": {"bigram": {"buckets": 65535, "mul_prev": 8191, "mul_cur": 31}}, "layers": entries,
+            "norm": {"eps": 1e-6}, "vocab": 32768, "width": W}
+
+
 def window_pairs(window, positions):
     """Sum over query positions of the keys each sees under a sliding window."""
     return sum(min(p + 1, window) for p in positions)
@@ -744,7 +775,8 @@ class DesignTimer(KernelClassTimer):
                                           "rotate_rows", "paged_attention_streams", "moe_route", "moe_plan", "moe_linear",
                                           "moe_combine", "moe_plan_padded", "moe_gather", "moe_linear_grouped", "moe_route_plan",
                                           "group_rmsnorm", "depth_average", "causal_conv", "latent_prepare", "latent_attention",
-                                          "gate_heads", "rglru_conv", "rglru_scan", "moe_gather_scaled", "moe_combine_update")
+                                          "gate_heads", "rglru_conv", "rglru_scan", "moe_gather_scaled", "moe_combine_update",
+                                          "embed_bigram", "norm_gate_rows", "delta_prepare", "delta_rule")
 
     def __init__(self, kernels, vocab, pairs, key_bytes, positions=(), head_weights=()):
         super().__init__(kernels, vocab)
@@ -781,6 +813,14 @@ class DesignTimer(KernelClassTimer):
             # the least: the gates' two numbers, u and the gelu branch's input read once, the result written; per element
             # two sigmoids, two exponentials, a root, a tanh and a dozen products and sums
             cls, ff, by = "recurrence", 40 * out.numel(), out.numel() * (4 * 4 + out.element_size())
+        elif name == "delta_rule":
+            up, heads, dim, vdim, state, out = a[1], a[4], a[5], a[6], a[11], a[15]
+            n = up.shape[0]
+            # the state decays, gives u, takes k u^T and is read: seven operations an entry and token
+            cls, ff = "delta rule", 7 * n * heads * dim * vdim
+            by = (a[0].numel() + up.numel() + a[2].numel()) * 4 + out.numel() * out.element_size() + 2 * a[14].numel() * heads * dim * vdim * 4
+        elif name == "delta_prepare":
+            cls, by = "delta convolutions", (a[0].numel() + a[12].numel()) * 4
         elif name == "latent_attention":
             q_lat, lat_pages, rot_pages, window = a[0], a[2], a[3], a[11]
             H, _, R = q_lat.shape
@@ -864,6 +904,8 @@ def run_designs(args):
             pair = (("golonex", recurrent_config(size)), ("lunelorn", hybrid_config(size)))
         if args.parallel:            # the closest in attention and dense products, and the closest in experts
             pair = (("mubutar", parallel_config(size)), ("qwen3", qwen), ("lunelorn", hybrid_config(size)))
+        if args.delta:               # the closest in latent attention, and the closest in recurrences beside attention
+            pair = (("tigelorn", delta_config(size)), ("golonex", recurrent_config(size)), ("lunelorn", hybrid_config(size)))
         for design, conf in pair:
             pool = batch * (context + 64) + PREFILL_TOKENS + 64
             opts = EngineOptions(dtype="bfloat16", page_size=16, num_pages=pool // 16, max_num_seqs=batch,
@@ -891,6 +933,8 @@ def run_designs(args):
                                                              getattr(m, "w_gates", None)) if w is not None]
             window = next((layer["mixer"]["mask"]["size"] for layer in conf.get("layers", ()) if design == "golonex"
                            and layer["type"] == "attention" and layer["mixer"].get("mask")), None)
+            if design == "tigelorn":
+                window = next(layer["mixer"]["left"]["mask"]["size"] for layer in conf["layers"] if layer["type"] == "parallel")
             pairs_of = (lambda positions: window_pairs(window, positions)) if window else (lambda positions: visible_pairs(chunk, positions))
             toks = torch.randint(0, vocab, (PREFILL_TOKENS,), generator=torch.Generator().manual_seed(2)).tolist()
             runner.cache.add_request("kp")
@@ -1249,6 +1293,117 @@ def time_recurrent_kernels(args):
     return 0
 
 
+def time_delta_kernels(args):
+    """The delta rule's kernels each alone (its convolutions, the recurrence), beside RWKV-style time mixing (the framework's
+    other matrix state with a decay per key channel) and the real-gated recurrence's convolution at the same width; linear
+    attention with silu inputs and its joint norm and gate, beside retention with its norm per head; attention over unit
+    queries with two-term weights under a window, beside plain attention of the same heads and window: a 2,048-token prompt
+    and a decode step of 8 requests (2,040 tokens in), CUDA events, the median of 20 repetitions with L2 flushed between
+    them, against the slowest of tensor flops, float32 flops and bytes; one JSON line.  (Also a profiler's small case.)"""
+    import torch
+    from infurnace_b200.kernels import load_cuda_kernels
+    K = load_cuda_kernels()
+    hbm_peak, tc_peak, peak_src = read_peaks()
+    fp32_peak = torch.cuda.get_device_properties(0).multi_processor_count * FP32_LANES_PER_SM * 2 * 1.965 / 1e3
+    g = torch.Generator(device="cuda").manual_seed(1)
+    rnd = lambda *shape, dtype=torch.float32: torch.randn(*shape, generator=g, device="cuda").to(dtype)      # noqa: E731
+    flush = torch.empty(160 << 20, dtype=torch.uint8, device="cuda")                # larger than L2
+
+    def timed(f, reps=20):
+        times = []
+        for i in range(reps + 3):
+            flush.zero_()
+            s, e = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            s.record()
+            f()
+            e.record()
+            torch.cuda.synchronize()
+            times.append(s.elapsed_time(e) * 1e3)
+        return statistics.median(times[3:])
+
+    def entry(us, tf=0.0, ff=0.0, by=0.0):
+        bound = max(tf / (tc_peak * 1e12), ff / (fp32_peak * 1e12), by / (hbm_peak * 1e9)) * 1e6
+        return {"us": round(us, 1), "of_bound": round(bound / us, 4)}
+
+    sizes = {}
+    for size in args.design_sizes.split(","):
+        conf = delta_config(size)
+        W = conf["width"]
+        m = next(l["mixer"] for l in conf["layers"] if l["type"] == "channel_delta")
+        par = next(l["mixer"] for l in conf["layers"] if l["type"] == "parallel")
+        H, D, V, taps, low_w = m["heads"], m["dim"], m["vdim"], m["conv"], 2 * m["rank"]
+        C = 2 * H * D + H * V
+        r = {}
+        for label, lens in (("prompt_2048", [PREFILL_TOKENS]), ("decode_8", [1] * 8)):
+            n, R, longest = sum(lens), len(lens), max(lens)
+            cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device="cuda")
+            past = 0 if R == 1 else 2040
+            seq = torch.tensor([x + past for x in lens], dtype=torch.int32, device="cuda")
+            slots = torch.arange(R, dtype=torch.int32, device="cuda")
+            req = torch.repeat_interleave(torch.arange(R, device="cuda"), torch.tensor(lens, device="cuda")).to(torch.int32)
+            arrays = (slots, cu, seq)
+            proj, qkv, beta = rnd(n, C + H + low_w), torch.zeros(n, C, device="cuda"), torch.zeros(n, H, device="cuda")
+            low, tw = torch.zeros(n, low_w, dtype=torch.bfloat16, device="cuda"), rnd(C, taps) / 2
+            cst, st = torch.zeros(8, max(taps - 1, 1), C, device="cuda"), torch.zeros(8, H, D, V, device="cuda")
+            up, rate, bias, nw = rnd(n, H * (D + V)), torch.exp(rnd(H)), rnd(H * D) - 3, torch.ones(V, device="cuda")
+            out = torch.zeros(n, H * V, dtype=torch.bfloat16, device="cuda")
+            r["convolutions_" + label] = entry(timed(lambda: K.delta_prepare(proj, H, H, D, V, tw, 1e-6, cst, *arrays, req, qkv, beta, low, low_w)),
+                                               by=n * C * 8)
+            r["delta_rule_" + label] = entry(timed(lambda: K.delta_rule(qkv, up, beta, H, H, D, V, rate, bias, nw, 1e-6, st, *arrays, out,
+                                                                        max_q_len=longest)),
+                                             ff=7.0 * n * H * D * V, by=n * (C + H * (D + V)) * 4 + n * H * V * 2 + 2 * R * H * D * V * 4)
+            mh = W // 64
+            q, k, v, gate, wraw = (rnd(n, W) for _ in range(5))
+            w0, u, mw, mst = rnd(W) - 1.5, rnd(W) / 2, 1 + rnd(W) / 5, torch.zeros(8, mh, 64, 64, device="cuda")
+            mo = torch.zeros(n, W, dtype=torch.bfloat16, device="cuda")
+            r["time_mixing_" + label] = entry(timed(lambda: K.linear_scan(q, k, v, wraw, mh, 64, 64, mst, *arrays, mo, 1e-6, w_bias=w0, bonus=u,
+                                                                          norm_weight=mw, gate=gate, max_q_len=longest)),
+                                              ff=6.0 * n * W * 64, by=n * W * 22 + 2 * R * W * 64 * 4)
+            # the other convolution at as many channels
+            xb, cw, cb = rnd(C), rnd(C, taps), rnd(C)
+            proj2, uo, cst2 = rnd(n, 2 * C), torch.zeros(n, C, device="cuda"), torch.zeros(8, max(taps - 1, 1), C, device="cuda")
+            ub, off = torch.zeros(C // 128, n, 128, dtype=torch.bfloat16, device="cuda"), torch.zeros(C // 128 + 1, dtype=torch.int32, device="cuda")
+            r["gated_unit_convolution_" + label] = entry(timed(lambda: K.rglru_conv(proj2, C, xb, cw, cb, cst2, *arrays, req, uo, ub, off)), by=n * C * 10)
+            # linear attention beside retention
+            rt = par["right"]
+            h2, d2, v2 = rt["heads"], rt["dim"], rt["vdim"]
+            rows, raw = rnd(n, h2 * (2 * d2 + 2 * v2)), torch.zeros(n, h2 * v2, device="cuda")
+            dec, st2, w2 = torch.tensor(rt["decay"], device="cuda"), torch.zeros(8, h2, d2, v2, device="cuda"), torch.ones(h2 * v2, device="cuda")
+            o2 = torch.zeros(n, h2 * v2, dtype=torch.bfloat16, device="cuda")
+            qs, ks, vs, gs = rows[:, :h2 * d2], rows[:, h2 * d2:2 * h2 * d2], rows[:, 2 * h2 * d2:h2 * (2 * d2 + v2)], rows[:, h2 * (2 * d2 + v2):]
+
+            def linear_attention():
+                K.linear_scan(qs, ks, vs, None, h2, d2, v2, st2, *arrays, raw, 1e-6, decay=dec, activation="silu", finish=False, max_q_len=longest)
+                K.norm_gate_rows(raw, o2, weight=w2, eps=1e-6, gate=gs, scale=0.7)
+            work = {"ff": 6.0 * n * h2 * d2 * v2, "by": n * h2 * (2 * d2 + 2 * v2) * 4 + n * h2 * v2 * 2 + 2 * R * h2 * d2 * v2 * 4}
+            r["linear_attention_" + label] = entry(timed(linear_attention), **work)
+            r["retention_" + label] = entry(timed(lambda: K.linear_scan(qs, ks, vs, None, h2, d2, v2, st2, *arrays, o2, 1e-6, decay=dec, gate=gs,
+                                                                        max_q_len=longest)), **work)
+            # attention
+            lf = par["left"]
+            h3, g3, d3, window, ps = lf["heads"], lf["kv_heads"], lf["dim"], lf["mask"]["size"], 16
+            total = longest + past
+            maxp = -(-total // ps)
+            pages = rnd(R * maxp + 1, 2, g3, ps, d3, dtype=torch.bfloat16)
+            bt = torch.arange(R * maxp, dtype=torch.int32, device="cuda").view(R, maxp).contiguous()
+            aq, ao = rnd(n, h3 * d3, dtype=torch.bfloat16), torch.zeros(n, h3 * d3, dtype=torch.bfloat16, device="cuda")
+            aq = aq / aq.float().view(n, h3, d3).pow(2).mean(-1).sqrt().repeat_interleave(d3, dim=1).to(torch.bfloat16)
+            pages[:, 0] /= pages[:, 0].float().pow(2).mean(-1, keepdim=True).sqrt().to(torch.bfloat16)
+            pairs = R * window_pairs(window, range(past, total))
+            work = {"tf": 4.0 * h3 * d3 * pairs, "by": 4 * R * min(total, window + longest) * g3 * d3}
+            bounded = {"score_bound": lf["scale"] * d3} if "score_bound" in K.paged_attention.__code__.co_varnames else {}
+            for name, terms, extra in (("unit_attention_", 2, bounded), ("plain_attention_", 1, {})):
+                r[name + label] = entry(timed(lambda: K.paged_attention(aq, h3, g3, d3, pages, bt, cu, seq, ao, lf["scale"], window, longest, total,
+                                                                        min_q_len=longest, weight_terms=terms, **extra)), **work)
+        sizes[size] = r
+    K.check_device_errors()
+    print(json.dumps({"metric": "delta_kernels_alone", "dtype": "bfloat16 operands, float32 recurrences", "unit": "us",
+                      "config": "L2 flushed between repetitions", "peaks": {"hbm_gbs": hbm_peak, "tensor_tflops": tc_peak,
+                                                                            "fp32_tflops_nominal": round(fp32_peak, 1), "source": peak_src},
+                      "sizes": sizes}))
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1274,6 +1429,8 @@ def main():
                     help="with --designs: the Golonex design beside Lunelorn (equal width, depth and active parameters)")
     ap.add_argument("--parallel", action="store_true",
                     help="with --designs: the Mubutar design beside Qwen3 and Lunelorn (equal width, depth and active parameters)")
+    ap.add_argument("--delta", action="store_true",
+                    help="with --designs: the Tigelorn design beside Golonex and Lunelorn (equal width, depth and active parameters)")
     ap.add_argument("--design-sizes", default="s,m", help="with --designs: which of the sizes s, m, l (commas between)")
     ap.add_argument("--kernels-alone", action="store_true",
                     help="with --designs: only the talking attention and the gated recurrence, each alone (a small case)")
@@ -1289,6 +1446,8 @@ def main():
     args.warmup = max(3, args.warmup)
     if args.designs:
         if args.kernels_alone:
+            if args.delta:
+                return time_delta_kernels(args)
             if args.parallel:
                 return time_parallel_kernels(args)
             if args.recurrent:
