@@ -37,6 +37,8 @@
 // maximum (the caller gives c of at most TC_MAX_CAP: 2^(c log2 e), summed over any context, is a float32 number): weights are
 // 2^z itself, nothing is ever rescaled.  tanh is a polynomial in two-number FMA instructions where every score of a warp's half
 // is small (|s| <= 0.7 c; absolute error 2e-7), else 1 - 2 / (1 + e^(2 s / c)).
+// -DSOFTCAP=2: scaled scores lie in [-c, c] as they are (queries and keys of unit size, say): no cap is applied, and the
+// exponentials again need no running maximum.
 // A sink z (an argument; -inf: none) joins the denominator as exp(z).
 //
 // Requests are routed as in attention_mma.cu: this kernel takes those with more than 16 score rows,
@@ -242,7 +244,7 @@ __device__ __forceinline__ void tc_pack_terms(float e0, float e1, uint32_t& firs
   second = 0u;
 #endif
 }
-// the exponent of a weight: capped scores are exponents already
+// the exponent of a weight: capped and bounded scores are exponents already
 #if SOFTCAP
 #define TC_EXPONENT(v) __uint_as_float(v)
 #else
@@ -549,7 +551,20 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
         for (int cc = 0; cc < 2; ++cc) tc_ld32(s_addr + cc * 32, v[cc]);
         tc_wait_ld();
         bool o_waited = false;                 // whether this step has waited for the previous half's P V
-#if SOFTCAP
+#if SOFTCAP == 2
+        // bounded scores: into the base-2 domain, in place
+        {
+          const f32x2 sl = tc_pair(score.scale_log2, score.scale_log2);
+#pragma unroll
+          for (int cc = 0; cc < 2; ++cc)
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+              float z0, z1;
+              tc_unpair(tc_mul2(tc_pair(__uint_as_float(v[cc][i]), __uint_as_float(v[cc][i + 1])), sl), z0, z1);
+              v[cc][i] = __float_as_uint(z0); v[cc][i + 1] = __float_as_uint(z1);
+            }
+        }
+#elif SOFTCAP
         // the capped scores in the base-2 domain, in place
         {
           float am[4] = {0.f, 0.f, 0.f, 0.f};
@@ -754,7 +769,7 @@ attn_tile_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
 // k_page_stride / v_page_stride elements apart, num_pages of them, each [kv heads][page_size][d or dv]; out [n_tokens, nq * dv].
 // nkv: groups of query heads (at most 128 each), `share` of which read one key/value head.  Takes the requests with
 // q_len * (nq / nkv) > 16.  page_size must be 16, 32 or 64.  softcap: 0 none (a library compiled with SOFTCAP takes a positive
-// one of at most 60 and no other takes one).  has_sink: exp(sink) joins the denominators (with SOFTCAP, sink at most 60).
+// one, or with SOFTCAP=2 the scores' bound, of at most 60 and no other takes one).  has_sink: exp(sink) joins the denominators (with SOFTCAP, sink at most 60).
 // err: a device int that stays 0 unless a bounded wait gave up.
 IFB_EXPORT int ifb_attention_tc(const void* qkv, int row_stride, const void* k_pages, long long k_page_stride, const void* v_pages,
                                 long long v_page_stride, long long num_pages, const int* block_tables, int bt_stride, const int* cu_q,

@@ -32,7 +32,7 @@
 
 constexpr int DR_C = 16;            // tokens of a chunk
 constexpr int DR_GROUP = 16;        // tokens that the walk stages at a time
-constexpr int DR_TOK = 8;           // neighbouring tokens that a warp of delta_prepare does
+constexpr int DR_TOK = 8;           // neighbouring tokens that a warp of delta_prepare does in a large step (one in a small one)
 constexpr float DR_LOG2E = 1.4426950408889634f;
 // A decay is at least 2^-32: what is left of the state is then below the rounding of anything that is added to it, and the
 // running sums of logarithms stay short enough for their differences to be exact to float32.
@@ -49,7 +49,7 @@ struct DeltaPrepareArgs {
   float* qkv;                        // [tokens][channels]
   float* beta;                       // [tokens][heads]
   void* low; int low_dtype, low_width, low_cols;
-  int tokens, kv_heads, heads, dim, vdim, channels;
+  int tokens, kv_heads, heads, dim, vdim, channels, tok;
 };
 
 // The conv output (before silu) of channel c for token t, the i-th of its request's tokens of this step.
@@ -98,6 +98,25 @@ __device__ __forceinline__ void dp_token(const DeltaPrepareArgs& a, int t, int i
   for (int e = lane; e < width; e += 32) dst[e] *= f;               // each lane its own elements
 }
 
+// The slot's inputs of `width` channels from c0 on after a portion of len tokens that starts at row t.
+__device__ __forceinline__ void dp_keep(const DeltaPrepareArgs& a, float* slot, int t, int len, int c0, int width, int lane) {
+  const int past = a.taps - 1;
+  for (int e = lane; e < width; e += 32) {               // rows in ascending order: a row reads a later one or the portion
+    const int c = c0 + e;
+    for (int p = 0; p < past; ++p)
+      slot[(size_t)p * a.channels + c] = len + p < past ? slot[(size_t)(len + p) * a.channels + c]
+                                                        : a.proj[(size_t)(t + len + p - past) * a.ld + c];
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ void dp_rest(const DeltaPrepareArgs& a, int t, int lane) {       // beta and the bottlenecks
+  const float* row = a.proj + (size_t)t * a.ld + a.channels;
+  for (int e = lane; e < a.heads; e += 32) a.beta[(size_t)t * a.heads + e] = 1.f / (1.f + expf(-row[e]));
+  T* dst = (T*)a.low + (size_t)t * a.low_cols;
+  for (int e = lane; e < a.low_cols; e += 32) dst[e] = from_f32<T>(e < a.low_width ? row[a.heads + e] : 0.f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 delta_prepare_kernel(DeltaPrepareArgs a) {
@@ -107,14 +126,9 @@ delta_prepare_kernel(DeltaPrepareArgs a) {
   const int unit = blockIdx.x * 8 + (threadIdx.x >> 5);
   const int G = a.kv_heads, units = 2 * G + a.heads;
   if (unit > units) return;
-  const int ta = blockIdx.y * DR_TOK, tb = min(ta + DR_TOK, a.tokens);
-  if (unit == units) {                                  // beta and the bottlenecks
-    for (int t = ta; t < tb; ++t) {
-      const float* row = a.proj + (size_t)t * a.ld + a.channels;
-      for (int e = lane; e < a.heads; e += 32) a.beta[(size_t)t * a.heads + e] = 1.f / (1.f + expf(-row[e]));
-      T* dst = (T*)a.low + (size_t)t * a.low_cols;
-      for (int e = lane; e < a.low_cols; e += 32) dst[e] = from_f32<T>(e < a.low_width ? row[a.heads + e] : 0.f);
-    }
+  const int ta = blockIdx.y * a.tok, tb = min(ta + a.tok, a.tokens);
+  if (unit == units) {
+    for (int t = ta; t < tb; ++t) dp_rest<T>(a, t, lane);
     return;
   }
   const bool is_v = unit >= 2 * G;
@@ -133,13 +147,113 @@ delta_prepare_kernel(DeltaPrepareArgs a) {
     }
     const int first = min(len, max(past, 1));
     for (int j = 0; j < first; ++j) dp_token(a, t + j, j, c0, width, !is_v, gain, slot, lane);
-    for (int e = lane; e < width; e += 32) {             // rows in ascending order: a row reads a later one or the portion
-      const int c = c0 + e;
-      for (int p = 0; p < past; ++p)
-        slot[(size_t)p * a.channels + c] = len + p < past ? slot[(size_t)(len + p) * a.channels + c]
-                                                          : a.proj[(size_t)(t + len + p - past) * a.ld + c];
-    }
+    dp_keep(a, slot, t, len, c0, width, lane);
   }
+}
+
+// The same for heads of up to 128 channels, multiples of 4, and two to four taps: a lane has four neighbouring channels, their
+// taps and their last inputs in registers, so that a token costs one 16-byte load.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+delta_prepare_rolling_kernel(DeltaPrepareArgs a) {
+  ifb_pdl_wait();
+  ifb_pdl_trigger();
+  constexpr int PAST = TAPS - 1;
+  const int lane = threadIdx.x & 31;
+  const int unit = blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int G = a.kv_heads, units = 2 * G + a.heads;
+  if (unit > units) return;
+  const int ta = blockIdx.y * a.tok, tb = min(ta + a.tok, a.tokens);
+  if (unit == units) {
+    for (int t = ta; t < tb; ++t) dp_rest<T>(a, t, lane);
+    return;
+  }
+  const bool is_v = unit >= 2 * G;
+  const int width = is_v ? a.vdim : a.dim;
+  const int c = (is_v ? 2 * G * a.dim + (unit - 2 * G) * a.vdim : unit * a.dim) + lane * 4;
+  const float gain = unit < G ? a.q_scale : 1.f;
+  const bool on = lane * 4 < width;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float w[4][TAPS];
+#pragma unroll
+  for (int x = 0; x < 4; ++x)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[x][j] = on ? a.taps_w[(size_t)(c + x) * TAPS + j] : 0.f;
+  auto input = [&](int t) { return on ? *reinterpret_cast<const float4*>(a.proj + (size_t)t * a.ld + c) : zero; };
+  auto emit = [&](int t, const float4* last, const float4 now) {       // last[PAST - 1]: the input before this one
+    float4 y = make_float4(now.x * w[0][PAST], now.y * w[1][PAST], now.z * w[2][PAST], now.w * w[3][PAST]);
+#pragma unroll
+    for (int j = 0; j < PAST; ++j) {
+      y.x = fmaf(last[j].x, w[0][j], y.x); y.y = fmaf(last[j].y, w[1][j], y.y);
+      y.z = fmaf(last[j].z, w[2][j], y.z); y.w = fmaf(last[j].w, w[3][j], y.w);
+    }
+    y.x = y.x / (1.f + expf(-y.x)); y.y = y.y / (1.f + expf(-y.y)); y.z = y.z / (1.f + expf(-y.z)); y.w = y.w / (1.f + expf(-y.w));
+    if (!is_v) {
+      const float f = gain / sqrtf(warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w) + a.unit_eps);
+      y.x *= f; y.y *= f; y.z *= f; y.w *= f;
+    }
+    if (on) *reinterpret_cast<float4*>(a.qkv + (size_t)t * a.channels + c) = y;
+  };
+  float4 last[PAST];
+  int have = -1;                                         // `last` holds the inputs before this token
+  for (int t = ta; t < tb; ++t) {
+    const int r = a.req_index[t];
+    if (a.seq_lens[r] <= 0) continue;
+    const int i = t - a.cu_q[r], len = a.cu_q[r + 1] - a.cu_q[r];
+    if (i > 0 && i < PAST) continue;                     // done by the warp of the request's first token
+    if (i > 0) {
+      if (have != t) {
+#pragma unroll
+        for (int j = 0; j < PAST; ++j) last[j] = input(t - PAST + j);
+      }
+      const float4 now = input(t);
+      emit(t, last, now);
+#pragma unroll
+      for (int j = 0; j + 1 < PAST; ++j) last[j] = last[j + 1];
+      last[PAST - 1] = now;
+      have = t + 1;
+      continue;
+    }
+    float* slot = a.state + (size_t)a.state_slots[r] * PAST * a.channels + c;
+    float4 held[PAST];
+#pragma unroll
+    for (int j = 0; j < PAST; ++j) held[j] = last[j] = on ? *reinterpret_cast<const float4*>(slot + (size_t)j * a.channels) : zero;
+#pragma unroll
+    for (int k = 0; k < PAST; ++k) {                     // the tokens that read the slot
+      if (k >= len) break;
+      const float4 now = input(t + k);
+      emit(t + k, last, now);
+#pragma unroll
+      for (int j = 0; j + 1 < PAST; ++j) last[j] = last[j + 1];
+      last[PAST - 1] = now;
+    }
+    if (on) {
+#pragma unroll
+      for (int p = 0; p < PAST; ++p) {                   // entry len + p of [held inputs | portion]
+        float4 v = zero;
+        if (len + p >= PAST) v = input(t + len + p - PAST);
+#pragma unroll
+        for (int j = 0; j < PAST; ++j)
+          if (len + p == j) v = held[j];
+        *reinterpret_cast<float4*>(slot + (size_t)p * a.channels) = v;
+      }
+    }
+    have = t + PAST;
+  }
+}
+
+template <typename T>
+static int dp_launch(DeltaPrepareArgs a, cudaStream_t stream) {
+  a.tok = a.tokens <= 512 ? 1 : DR_TOK;
+  const int chunks = (a.tokens + a.tok - 1) / a.tok;
+  if (chunks > 65535) return IFB_ERR_SIZE;
+  dim3 grid((2 * a.kv_heads + a.heads + 1 + 7) / 8, chunks);
+  const bool rolling = a.dim <= 128 && a.vdim <= 128 && a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ld % 4 == 0 &&
+                       (((uintptr_t)a.proj | (uintptr_t)a.qkv | (uintptr_t)a.state) & 15) == 0;
+  if (rolling && a.taps == 2) return ifb_launch(delta_prepare_rolling_kernel<T, 2>, grid, dim3(256), 0, stream, a);
+  if (rolling && a.taps == 3) return ifb_launch(delta_prepare_rolling_kernel<T, 3>, grid, dim3(256), 0, stream, a);
+  if (rolling && a.taps == 4) return ifb_launch(delta_prepare_rolling_kernel<T, 4>, grid, dim3(256), 0, stream, a);
+  return ifb_launch(delta_prepare_kernel<T>, grid, dim3(256), 0, stream, a);
 }
 
 IFB_EXPORT int ifb_delta_prepare(const float* proj, long long ld, const float* taps_w, int taps, float unit_eps, float q_scale,
@@ -149,14 +263,11 @@ IFB_EXPORT int ifb_delta_prepare(const float* proj, long long ld, const float* t
   if (tokens <= 0) return IFB_OK;
   if (kv_heads < 1 || heads < 1 || dim < 1 || vdim < 1 || taps < 1 || low_cols < low_width) return IFB_ERR_SIZE;
   const int channels = 2 * kv_heads * dim + heads * vdim;
-  const int chunks = (tokens + DR_TOK - 1) / DR_TOK;
-  if (chunks > 65535) return IFB_ERR_SIZE;
   DeltaPrepareArgs a{proj, ld, taps_w, taps, unit_eps, q_scale, state, state_slots, cu_q, seq_lens, req_index, qkv, beta, low, low_dtype,
-                     low_width, low_cols, tokens, kv_heads, heads, dim, vdim, channels};
-  dim3 grid((2 * kv_heads + heads + 1 + 7) / 8, chunks);
-  if (low_dtype == IFB_BF16) return ifb_launch(delta_prepare_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, a);
+                     low_width, low_cols, tokens, kv_heads, heads, dim, vdim, channels, 1};
+  if (low_dtype == IFB_BF16) return dp_launch<__nv_bfloat16>(a, stream);
   if (low_dtype != IFB_F32) return IFB_ERR_DTYPE;
-  return ifb_launch(delta_prepare_kernel<float>, grid, dim3(256), 0, stream, a);
+  return dp_launch<float>(a, stream);
 }
 
 // ------------------------------------------------------------------------------------------ (2) delta_rule
@@ -337,11 +448,12 @@ delta_wide_kernel(DeltaRuleArgs a) {
 }
 
 // ---- the chunked form
-// One (chunk, head) of the scratch: W, Q, K [DR_C][dp] each, P [DR_C][DR_C], decay [dp], U [DR_C][vp]
+constexpr int DR_PP = DR_C + 4;     // pitch of a row of P, so that neighbouring rows start in different banks
+// One (chunk, head) of the scratch: W, Q, K [DR_C][dp] each, P [DR_C][DR_PP], decay [dp], U [DR_C][vp]
 __host__ __device__ __forceinline__ int dr_dp(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
 __host__ __device__ __forceinline__ int dr_vp(int vdim) { return (vdim + 31) / 32 * 32; }
 __host__ __device__ __forceinline__ size_t dr_chunk_floats(int dim, int vdim) {
-  return (size_t)3 * DR_C * dr_dp(dim) + DR_C * DR_C + dr_dp(dim) + (size_t)DR_C * dr_vp(vdim);
+  return (size_t)3 * DR_C * dr_dp(dim) + DR_C * DR_PP + dr_dp(dim) + (size_t)DR_C * dr_vp(vdim);
 }
 
 // The chunk that row `row` of the grid is; false: beyond the last
@@ -359,28 +471,37 @@ __device__ __forceinline__ bool dr_find_chunk(const DeltaRuleArgs& a, int row, i
   return false;
 }
 
-constexpr int DA_THREADS = 288;                        // 2 threads for each of the 136 pairs s <= t, and 16 more
+// 2^x for x at most 0 (what underflows is 0)
+__device__ __forceinline__ float dr_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
 
+constexpr int DA_THREADS = 320;                        // 8 threads for each of the 40 (t, four neighbouring s <= t) items
+
+template <int DP>
 __global__ void __launch_bounds__(DA_THREADS)
 delta_chunk_kernel(DeltaRuleArgs a) {
   extern __shared__ float sm[];
   ifb_pdl_wait();
   ifb_pdl_trigger();
+  constexpr int PITCH = DP + 1;
   int t0, cnt;
   if (!dr_find_chunk(a, blockIdx.y, t0, cnt)) return;
-  const int h = blockIdx.x, dim = a.dim, vdim = a.vdim, dp = dr_dp(dim), vp = dr_vp(vdim), pitch = dp + 1;
+  const int h = blockIdx.x, dim = a.dim, vdim = a.vdim, vp = dr_vp(vdim);
   const int hk = h / (a.heads / a.kv_heads), tid = threadIdx.x;
-  float* qs = sm;                                      // [DR_C][pitch]
-  float* ks = qs + DR_C * pitch;
-  float* ls = ks + DR_C * pitch;                       // log2 of the decays, then their running sums
-  float* As = ls + DR_C * pitch;                       // [DR_C][DR_C + 1]
+  float* qs = sm;                                      // [DR_C][PITCH]
+  float* ks = qs + DR_C * PITCH;
+  float* ls = ks + DR_C * PITCH;                       // log2 of the decays, then their running sums
+  float* As = ls + DR_C * PITCH;                       // [DR_C][DR_C + 1]
   float* Ts = As + DR_C * (DR_C + 1);                  // [DR_C][DR_C + 1]
   float* bs = Ts + DR_C * (DR_C + 1);                  // [DR_C]
   float* base = a.chunks + ((size_t)blockIdx.y * a.heads + h) * dr_chunk_floats(dim, vdim);
-  float *gW = base, *gQ = gW + DR_C * dp, *gK = gQ + DR_C * dp, *gP = gK + DR_C * dp, *gG = gP + DR_C * DR_C, *gU = gG + dp;
+  float *gW = base, *gQ = gW + DR_C * DP, *gK = gQ + DR_C * DP, *gP = gK + DR_C * DP, *gG = gP + DR_C * DR_PP, *gU = gG + DP;
   const float rate = a.rate[h];
-  for (int idx = tid; idx < DR_C * dp; idx += DA_THREADS) {
-    const int t = idx / dp, i = idx % dp;
+  for (int idx = tid; idx < DR_C * DP; idx += DA_THREADS) {
+    const int t = idx / DP, i = idx % DP;
     float qv = 0.f, kv = 0.f, lv = 0.f;
     if (t < cnt && i < dim) {
       const float* row = a.qkv + (size_t)(t0 + t) * a.ldc;
@@ -388,35 +509,49 @@ delta_chunk_kernel(DeltaRuleArgs a) {
       kv = row[(a.kv_heads + hk) * dim + i];
       lv = dr_log2_decay(a.up[(size_t)(t0 + t) * a.ldu + h * dim + i] + a.bias[h * dim + i], rate);
     }
-    qs[t * pitch + i] = qv; ks[t * pitch + i] = kv; ls[t * pitch + i] = lv;
+    qs[t * PITCH + i] = qv; ks[t * PITCH + i] = kv; ls[t * PITCH + i] = lv;
   }
   if (tid < DR_C) bs[tid] = tid < cnt ? a.beta[(size_t)(t0 + tid) * a.heads + h] : 0.f;
   __syncthreads();
-  if (tid < dp) {
+  if (tid < DP) {
     float s = 0.f;
 #pragma unroll
-    for (int t = 0; t < DR_C; ++t) { s += ls[t * pitch + tid]; ls[t * pitch + tid] = s; }
+    for (int t = 0; t < DR_C; ++t) { s += ls[t * PITCH + tid]; ls[t * PITCH + tid] = s; }
   }
   __syncthreads();
   {
-    // pair p = t (t + 1) / 2 + s; two neighbouring threads share its channels.  The last 16 threads repeat pair 0.
-    const int p = min(tid >> 1, DR_C * (DR_C + 1) / 2 - 1), half = tid & 1;
-    int t = 0;
-    while ((t + 1) * (t + 2) / 2 <= p) ++t;
-    const int s = p - t * (t + 1) / 2;
-    float ak = 0.f, aq = 0.f;
-    for (int i = half; i < dp; i += 2) {
-      const float ke = ks[s * pitch + i] * exp2f(ls[t * pitch + i] - ls[s * pitch + i]);
-      ak = fmaf(ks[t * pitch + i], ke, ak);
-      aq = fmaf(qs[t * pitch + i], ke, aq);
+    // item (t, g): the pairs of t with s = 4 g .. 4 g + 3 (those beyond t count for nothing); its 8 neighbouring threads share
+    // the channels
+    const int item = tid >> 3, lane8 = tid & 7;
+    const int band = item < 4 ? 0 : item < 12 ? 1 : item < 24 ? 2 : 3;             // t / 4: bands of 4, 8, 12 and 16 items
+    const int in = item - 2 * band * (band + 1), t = 4 * band + in / (band + 1), s0 = 4 * (in % (band + 1));
+    float ak[4] = {0.f, 0.f, 0.f, 0.f}, aq[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+    for (int i = lane8; i < DP; i += 8) {
+      const float kt = ks[t * PITCH + i], qt = qs[t * PITCH + i], lt = ls[t * PITCH + i];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const float ke = ks[(s0 + x) * PITCH + i] * dr_exp2(fminf(lt - ls[(s0 + x) * PITCH + i], 0.f));
+        ak[x] = fmaf(kt, ke, ak[x]);
+        aq[x] = fmaf(qt, ke, aq[x]);
+      }
     }
-    ak += __shfl_xor_sync(0xffffffffu, ak, 1);
-    aq += __shfl_xor_sync(0xffffffffu, aq, 1);
-    if (half == 0 && tid < DR_C * (DR_C + 1)) {
-      As[t * (DR_C + 1) + s] = s < t ? bs[t] * ak : 0.f;
-      gP[t * DR_C + s] = aq;
-      if (s < t) gP[s * DR_C + t] = 0.f;
-    }
+#pragma unroll
+    for (int x = 0; x < 4; ++x)
+#pragma unroll
+      for (int m = 1; m < 8; m <<= 1) {
+        ak[x] += __shfl_xor_sync(0xffffffffu, ak[x], m);
+        aq[x] += __shfl_xor_sync(0xffffffffu, aq[x], m);
+      }
+    if (lane8 == 0)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int s = s0 + x;
+        if (s > t) continue;
+        As[t * (DR_C + 1) + s] = s < t ? bs[t] * ak[x] : 0.f;
+        gP[t * DR_PP + s] = aq[x];
+        if (s < t) gP[s * DR_PP + t] = 0.f;
+      }
   }
   __syncthreads();
   if (tid < 32) {
@@ -424,34 +559,37 @@ delta_chunk_kernel(DeltaRuleArgs a) {
       float x[DR_C];
 #pragma unroll
       for (int t = 0; t < DR_C; ++t) {
-        float v = t == tid ? 1.f : 0.f;
+        float v0 = t == tid ? 1.f : 0.f, v1 = 0.f;
 #pragma unroll
-        for (int s = 0; s < t; ++s) v = fmaf(-As[t * (DR_C + 1) + s], x[s], v);
-        x[t] = v;
+        for (int s = 0; s < t; ++s) {
+          if (s & 1) v1 = fmaf(-As[t * (DR_C + 1) + s], x[s], v1);
+          else v0 = fmaf(-As[t * (DR_C + 1) + s], x[s], v0);
+        }
+        x[t] = v0 + v1;
       }
 #pragma unroll
       for (int t = 0; t < DR_C; ++t) Ts[t * (DR_C + 1) + tid] = x[t] * bs[tid];
     }
   } else {
-    for (int idx = tid - 32; idx < DR_C * dp; idx += DA_THREADS - 32) {
-      const int t = idx / dp, i = idx % dp;
-      const float l = ls[t * pitch + i], end = ls[(DR_C - 1) * pitch + i];
-      gQ[idx] = qs[t * pitch + i] * exp2f(l);
-      gK[idx] = ks[t * pitch + i] * exp2f(end - l);
-      if (t == 0) gG[i] = exp2f(end);
+    for (int idx = tid - 32; idx < DR_C * DP; idx += DA_THREADS - 32) {
+      const int t = idx / DP, i = idx % DP;
+      const float l = ls[t * PITCH + i], end = ls[(DR_C - 1) * PITCH + i];
+      gQ[idx] = qs[t * PITCH + i] * dr_exp2(l);
+      gK[idx] = ks[t * PITCH + i] * dr_exp2(end - l);
+      if (t == 0) gG[i] = dr_exp2(end);
     }
   }
   __syncthreads();
-  for (int j = tid; j < dp + vp; j += DA_THREADS) {    // W: a thread per channel; U: a thread per column
+  for (int j = tid; j < DP + vp; j += DA_THREADS) {    // W: a thread per channel; U: a thread per column
     float x[DR_C];
     float* dst;
     int step;
-    if (j < dp) {
+    if (j < DP) {
 #pragma unroll
-      for (int t = 0; t < DR_C; ++t) x[t] = ks[t * pitch + j] * exp2f(ls[t * pitch + j]);
-      dst = gW + j; step = dp;
+      for (int t = 0; t < DR_C; ++t) x[t] = ks[t * PITCH + j] * dr_exp2(ls[t * PITCH + j]);
+      dst = gW + j; step = DP;
     } else {
-      const int c = j - dp;
+      const int c = j - DP;
 #pragma unroll
       for (int t = 0; t < DR_C; ++t)
         x[t] = (t < cnt && c < vdim) ? a.qkv[(size_t)(t0 + t) * a.ldc + 2 * a.kv_heads * dim + h * vdim + c] : 0.f;
@@ -471,34 +609,35 @@ __device__ __forceinline__ void dr_copy16(float* dst, const float* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
 
-// Each of 16 neighbouring lanes holds 16 numbers; lane i is left with the sum over the lanes of the i-th.
-__device__ __forceinline__ float dr_reduce16(float* x, int i) {
+// Each of 8 neighbouring lanes holds 16 numbers; lane i is left with the sums over the lanes of numbers 2 i and 2 i + 1.
+__device__ __forceinline__ float2 dr_reduce16(float* x, int i) {
 #pragma unroll
-  for (int half = 8; half >= 1; half >>= 1) {
-    const bool up = i & half;
+  for (int half = 8; half >= 2; half >>= 1) {
+    const bool up = i & (half >> 1);
 #pragma unroll
     for (int j = 0; j < half; ++j) {
       const float send = up ? x[j] : x[j + half], keep = up ? x[j + half] : x[j];
-      x[j] = keep + __shfl_xor_sync(0xffffffffu, send, half);
+      x[j] = keep + __shfl_xor_sync(0xffffffffu, send, half >> 1);
     }
   }
-  return x[0];
+  return make_float2(x[0], x[1]);
 }
 
-// A block per (head, slab of 16 CPT columns) and request: thread (column, part), 16 parts of a column in neighbouring lanes,
-// part p with rows (j / V) 16 V + p V + j % V, j = 0 .. DP / 16 - 1, V = min(4, DP / 16), of CPT columns 16 apart.
+// A block per (head, slab of 16 CPT columns) and request: thread (column, part), 8 parts of a column in neighbouring lanes,
+// part p with rows 32 b + 4 p + i, b = 0 .. DP / 32 - 1, i = 0 .. 3, of CPT columns 16 apart.
+constexpr int DC_THREADS = 128;
 template <int DP, int CPT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(DC_THREADS)
 delta_carry_kernel(DeltaRuleArgs a) {
-  constexpr int RPT = DP / 16, V = RPT < 4 ? RPT : 4, NC = 16 * CPT;
-  constexpr int OPER = 3 * DR_C * DP + DR_C * DR_C + DP;              // W, Q, K, P, decay: contiguous in the scratch
+  constexpr int NB = DP / 32, NC = 16 * CPT;
+  constexpr int OPER = 3 * DR_C * DP + DR_C * DR_PP + DP;             // W, Q, K, P, decay: contiguous in the scratch
   constexpr int STAGE = OPER + DR_C * NC;
   extern __shared__ __align__(16) float sm[];
   ifb_pdl_wait();
   ifb_pdl_trigger();
   const int r = blockIdx.y, h = blockIdx.x / a.slabs, c0 = (blockIdx.x % a.slabs) * NC;
   if (a.seq_lens[r] <= 0) return;
-  const int dim = a.dim, vdim = a.vdim, vp = dr_vp(vdim), tid = threadIdx.x, p = tid & 15, cl = tid >> 4;
+  const int dim = a.dim, vdim = a.vdim, vp = dr_vp(vdim), tid = threadIdx.x, p = tid & 7, cl = tid >> 3;
   int first = 0;                                        // the request's first chunk among all
   for (int i = 0; i < r; ++i) first += a.seq_lens[i] > 0 ? (a.cu_q[i + 1] - a.cu_q[i] + DR_C - 1) / DR_C : 0;
   const int ta = a.cu_q[r], tb = a.cu_q[r + 1], n = (tb - ta + DR_C - 1) / DR_C;
@@ -507,26 +646,26 @@ delta_carry_kernel(DeltaRuleArgs a) {
   float* us = sm + 2 * STAGE;                           // [NC][DR_C + 4]: u of a column, read as float4
   float* os = us + NC * (DR_C + 4);                     // [2][DR_C][NC]
   float* sp = a.state + (((size_t)a.state_slots[r] * a.heads + h) * dim) * vdim;
-  float S[CPT][RPT];
-  int row[RPT];
-#pragma unroll
-  for (int i = 0; i < RPT; ++i) row[i] = (i / V) * 16 * V + p * V + i % V;
+  float S[CPT][NB * 4];
 #pragma unroll
   for (int x = 0; x < CPT; ++x) {
     const int c = c0 + x * 16 + cl;
 #pragma unroll
-    for (int i = 0; i < RPT; ++i) S[x][i] = (c < vdim && row[i] < dim) ? sp[(size_t)row[i] * vdim + c] : 0.f;
+    for (int i = 0; i < NB * 4; ++i) {
+      const int row = (i >> 2) * 32 + p * 4 + (i & 3);
+      S[x][i] = (c < vdim && row < dim) ? sp[(size_t)row * vdim + c] : 0.f;
+    }
   }
   auto ask = [&](int j) {
     const float* g = src + (size_t)j * a.heads * per;
     float* s = sm + (j & 1) * STAGE;
-    for (int i = tid * 4; i < OPER; i += 1024) dr_copy16(s + i, g + i);
-    for (int i = tid * 4; i < DR_C * NC; i += 1024) dr_copy16(s + OPER + i, g + OPER + (size_t)(i / NC) * vp + c0 + i % NC);
+    for (int i = tid * 4; i < OPER; i += DC_THREADS * 4) dr_copy16(s + i, g + i);
+    for (int i = tid * 4; i < DR_C * NC; i += DC_THREADS * 4) dr_copy16(s + OPER + i, g + OPER + (size_t)(i / NC) * vp + c0 + i % NC);
     asm volatile("cp.async.commit_group;\n" ::);
   };
   auto give = [&](int j) {                              // outputs of chunk j from shared memory, whole row segments
     const float* o = os + (j & 1) * DR_C * NC;
-    for (int i = tid; i < DR_C * NC; i += 256) {
+    for (int i = tid; i < DR_C * NC; i += DC_THREADS) {
       const int t = ta + j * DR_C + i / NC, c = c0 + i % NC;
       if (t < tb && c < vdim) a.raw[((size_t)t * a.heads + h) * vdim + c] = o[i];
     }
@@ -538,37 +677,51 @@ delta_carry_kernel(DeltaRuleArgs a) {
     if (j + 1 < n) ask(j + 1);
     if (j > 0) give(j - 1);
     const float* s = sm + (j & 1) * STAGE;
-    const float *Ws = s, *Qs = Ws + DR_C * DP, *Ks = Qs + DR_C * DP, *Ps = Ks + DR_C * DP, *Gs = Ps + DR_C * DR_C, *Us = Gs + DP;
-    float w[CPT][DR_C], o[CPT][DR_C];
+    const float *Ws = s, *Qs = Ws + DR_C * DP, *Ks = Qs + DR_C * DP, *Ps = Ks + DR_C * DP, *Gs = Ps + DR_C * DR_PP, *Us = Gs + DP;
+    {
+      float w[CPT][DR_C];
 #pragma unroll
-    for (int t = 0; t < DR_C; ++t) {
+      for (int t = 0; t < DR_C; ++t) {
 #pragma unroll
-      for (int x = 0; x < CPT; ++x) w[x][t] = o[x][t] = 0.f;
+        for (int x = 0; x < CPT; ++x) w[x][t] = 0.f;
 #pragma unroll
-      for (int b = 0; b < RPT / V; ++b) {
-        float wv[V], qv[V];
-        if (V == 4) {
-          *reinterpret_cast<float4*>(wv) = *reinterpret_cast<const float4*>(Ws + t * DP + b * 64 + p * 4);
-          *reinterpret_cast<float4*>(qv) = *reinterpret_cast<const float4*>(Qs + t * DP + b * 64 + p * 4);
-        } else {
-          *reinterpret_cast<float2*>(wv) = *reinterpret_cast<const float2*>(Ws + t * DP + p * 2);
-          *reinterpret_cast<float2*>(qv) = *reinterpret_cast<const float2*>(Qs + t * DP + p * 2);
+        for (int b = 0; b < NB; ++b) {
+          const float4 wv = *reinterpret_cast<const float4*>(Ws + t * DP + b * 32 + p * 4);
+#pragma unroll
+          for (int x = 0; x < CPT; ++x)
+            w[x][t] = fmaf(wv.w, S[x][4 * b + 3], fmaf(wv.z, S[x][4 * b + 2], fmaf(wv.y, S[x][4 * b + 1], fmaf(wv.x, S[x][4 * b], w[x][t]))));
         }
+      }
 #pragma unroll
-        for (int x = 0; x < CPT; ++x)
-#pragma unroll
-          for (int i = 0; i < V; ++i) {
-            w[x][t] = fmaf(wv[i], S[x][b * V + i], w[x][t]);
-            o[x][t] = fmaf(qv[i], S[x][b * V + i], o[x][t]);
-          }
+      for (int x = 0; x < CPT; ++x) {
+        const float2 ws = dr_reduce16(w[x], p);
+        const int col = x * 16 + cl;
+        *reinterpret_cast<float2*>(us + col * (DR_C + 4) + 2 * p) =
+            make_float2(Us[2 * p * NC + col] - ws.x, Us[(2 * p + 1) * NC + col] - ws.y);
       }
     }
+    __syncwarp();                                       // the 8 lanes of a column are in one warp
+    float y[CPT][2];                                    // outputs of tokens 2 p and 2 p + 1: what the state before the chunk gives
+    {
+      float o[CPT][DR_C];
 #pragma unroll
-    for (int x = 0; x < CPT; ++x) {
-      const float ws = dr_reduce16(w[x], p);
-      us[(x * 16 + cl) * (DR_C + 4) + p] = Us[p * NC + x * 16 + cl] - ws;
+      for (int t = 0; t < DR_C; ++t) {
+#pragma unroll
+        for (int x = 0; x < CPT; ++x) o[x][t] = 0.f;
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+          const float4 qv = *reinterpret_cast<const float4*>(Qs + t * DP + b * 32 + p * 4);
+#pragma unroll
+          for (int x = 0; x < CPT; ++x)
+            o[x][t] = fmaf(qv.w, S[x][4 * b + 3], fmaf(qv.z, S[x][4 * b + 2], fmaf(qv.y, S[x][4 * b + 1], fmaf(qv.x, S[x][4 * b], o[x][t]))));
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < CPT; ++x) {
+        const float2 v = dr_reduce16(o[x], p);
+        y[x][0] = v.x; y[x][1] = v.y;
+      }
     }
-    __syncwarp();                                       // the 16 lanes of a column are in one warp
     float u[CPT][DR_C];
 #pragma unroll
     for (int x = 0; x < CPT; ++x)
@@ -576,34 +729,34 @@ delta_carry_kernel(DeltaRuleArgs a) {
       for (int t = 0; t < DR_C; t += 4)
         *reinterpret_cast<float4*>(&u[x][t]) = *reinterpret_cast<const float4*>(us + (x * 16 + cl) * (DR_C + 4) + t);
 #pragma unroll
-    for (int x = 0; x < CPT; ++x) {
-      float y = dr_reduce16(o[x], p);
+    for (int m = 0; m < 2; ++m)
 #pragma unroll
       for (int t = 0; t < DR_C; t += 4) {
-        const float4 pv = *reinterpret_cast<const float4*>(Ps + p * DR_C + t);
-        y = fmaf(pv.x, u[x][t], y); y = fmaf(pv.y, u[x][t + 1], y); y = fmaf(pv.z, u[x][t + 2], y); y = fmaf(pv.w, u[x][t + 3], y);
+        const float4 pv = *reinterpret_cast<const float4*>(Ps + (2 * p + m) * DR_PP + t);
+#pragma unroll
+        for (int x = 0; x < CPT; ++x)
+          y[x][m] = fmaf(pv.w, u[x][t + 3], fmaf(pv.z, u[x][t + 2], fmaf(pv.y, u[x][t + 1], fmaf(pv.x, u[x][t], y[x][m]))));
       }
-      os[(j & 1) * DR_C * NC + p * NC + x * 16 + cl] = y;
+#pragma unroll
+    for (int x = 0; x < CPT; ++x) {
+      float* o = os + (j & 1) * DR_C * NC + x * 16 + cl;
+      o[2 * p * NC] = y[x][0];
+      o[(2 * p + 1) * NC] = y[x][1];
     }
     __syncwarp();                                       // u was read by all its lanes before the next chunk writes it
 #pragma unroll
-    for (int b = 0; b < RPT / V; ++b) {
-      float gv[V];
+    for (int b = 0; b < NB; ++b) {
+      const float4 gv = *reinterpret_cast<const float4*>(Gs + b * 32 + p * 4);
 #pragma unroll
-      for (int i = 0; i < V; ++i) gv[i] = Gs[b * 16 * V + p * V + i];
-#pragma unroll
-      for (int x = 0; x < CPT; ++x)
-#pragma unroll
-        for (int i = 0; i < V; ++i) S[x][b * V + i] *= gv[i];
+      for (int x = 0; x < CPT; ++x) { S[x][4 * b] *= gv.x; S[x][4 * b + 1] *= gv.y; S[x][4 * b + 2] *= gv.z; S[x][4 * b + 3] *= gv.w; }
 #pragma unroll
       for (int t = 0; t < DR_C; ++t) {
-        float kv[V];
-        if (V == 4) *reinterpret_cast<float4*>(kv) = *reinterpret_cast<const float4*>(Ks + t * DP + b * 64 + p * 4);
-        else *reinterpret_cast<float2*>(kv) = *reinterpret_cast<const float2*>(Ks + t * DP + p * 2);
+        const float4 kv = *reinterpret_cast<const float4*>(Ks + t * DP + b * 32 + p * 4);
 #pragma unroll
-        for (int x = 0; x < CPT; ++x)
-#pragma unroll
-          for (int i = 0; i < V; ++i) S[x][b * V + i] = fmaf(kv[i], u[x][t], S[x][b * V + i]);
+        for (int x = 0; x < CPT; ++x) {
+          S[x][4 * b] = fmaf(kv.x, u[x][t], S[x][4 * b]); S[x][4 * b + 1] = fmaf(kv.y, u[x][t], S[x][4 * b + 1]);
+          S[x][4 * b + 2] = fmaf(kv.z, u[x][t], S[x][4 * b + 2]); S[x][4 * b + 3] = fmaf(kv.w, u[x][t], S[x][4 * b + 3]);
+        }
       }
     }
   }
@@ -613,8 +766,10 @@ delta_carry_kernel(DeltaRuleArgs a) {
   for (int x = 0; x < CPT; ++x) {
     const int c = c0 + x * 16 + cl;
 #pragma unroll
-    for (int i = 0; i < RPT; ++i)
-      if (c < vdim && row[i] < dim) sp[(size_t)row[i] * vdim + c] = S[x][i];
+    for (int i = 0; i < NB * 4; ++i) {
+      const int row = (i >> 2) * 32 + p * 4 + (i & 3);
+      if (c < vdim && row < dim) sp[(size_t)row * vdim + c] = S[x][i];
+    }
   }
 }
 
@@ -634,11 +789,23 @@ static int dr_walk(DeltaRuleArgs a, cudaStream_t s) {
 
 template <int DP, int CPT>
 static int dr_carry(DeltaRuleArgs a, cudaStream_t s) {
-  constexpr int NC = 16 * CPT, STAGE = 3 * DR_C * DP + DR_C * DR_C + DP + DR_C * NC;
+  constexpr int NC = 16 * CPT, STAGE = 3 * DR_C * DP + DR_C * DR_PP + DP + DR_C * NC;
   const size_t smem = (size_t)(2 * STAGE + NC * (DR_C + 4) + 2 * DR_C * NC) * sizeof(float);
   a.slabs = (a.vdim + NC - 1) / NC;
   IFB_ALLOW_SMEM((delta_carry_kernel<DP, CPT>), smem);
-  return ifb_launch(delta_carry_kernel<DP, CPT>, dim3(a.heads * a.slabs, a.requests), dim3(256), smem, s, a);
+  // not early: blocks placed while the chunks' launch still fills the device crowd on the SMs that are free first
+  return ifb_launch_opt(false, delta_carry_kernel<DP, CPT>, dim3(a.heads * a.slabs, a.requests), dim3(DC_THREADS), smem, s, a);
+}
+
+template <int DP>
+static int dr_chunked(DeltaRuleArgs a, int rows, bool two, cudaStream_t s) {
+  const size_t smem = (size_t)(3 * DR_C * (DP + 1) + 2 * DR_C * (DR_C + 1) + DR_C) * sizeof(float);
+  IFB_ALLOW_SMEM(delta_chunk_kernel<DP>, smem);
+  const int st = ifb_launch(delta_chunk_kernel<DP>, dim3(a.heads, rows), dim3(DA_THREADS), smem, s, a);
+  if (st != IFB_OK) return st;
+  if constexpr (DP <= 128)
+    if (two) return dr_carry<DP, 2>(a, s);
+  return dr_carry<DP, 1>(a, s);
 }
 
 template <typename T>
@@ -653,16 +820,12 @@ static int dr_run(DeltaRuleArgs a, int tokens, int columns, cudaStream_t s) {
   if (a.chunks) {
     const long long rows = (tokens + DR_C - 1) / DR_C + a.requests;
     if (rows > 65535 || !a.raw) return IFB_ERR_SIZE;
-    const size_t smem = (size_t)(3 * DR_C * (dr_dp(a.dim) + 1) + 2 * DR_C * (DR_C + 1) + DR_C) * sizeof(float);
-    IFB_ALLOW_SMEM(delta_chunk_kernel, smem);
-    st = ifb_launch(delta_chunk_kernel, dim3(a.heads, (unsigned)rows), dim3(DA_THREADS), smem, s, a);
-    if (st != IFB_OK) return st;
     const bool two = columns == 2;
     switch (dr_dp(a.dim)) {
-      case 32: st = two ? dr_carry<32, 2>(a, s) : dr_carry<32, 1>(a, s); break;
-      case 64: st = two ? dr_carry<64, 2>(a, s) : dr_carry<64, 1>(a, s); break;
-      case 128: st = two ? dr_carry<128, 2>(a, s) : dr_carry<128, 1>(a, s); break;
-      default: st = dr_carry<256, 1>(a, s);
+      case 32: st = dr_chunked<32>(a, (int)rows, two, s); break;
+      case 64: st = dr_chunked<64>(a, (int)rows, two, s); break;
+      case 128: st = dr_chunked<128>(a, (int)rows, two, s); break;
+      default: st = dr_chunked<256>(a, (int)rows, two, s);
     }
   } else {
     const int cols = dr_walk_cols(a.dim, a.vdim);

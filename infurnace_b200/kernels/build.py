@@ -54,6 +54,8 @@ LIBRARIES: Dict[str, tuple] = {
 DEFAULT_VARIANTS = [("attention_mma", {"HEAD_DIM": d}) for d in (128, 16, 32, 48)]
 # capped scores with two-term weights, heads of 128: decoding and prompts
 DEFAULT_VARIANTS += [(name, {"HEAD_DIM": 128, "WEIGHT_TERMS": 2, "SOFTCAP": 1}) for name in ("attention_mma", "attention_tc")]
+# bounded scores of unit queries and keys with two-term weights, heads of 128: prompts, and decoding
+DEFAULT_VARIANTS += [("attention_tc", {"HEAD_DIM": 128, "WEIGHT_TERMS": 2, "SOFTCAP": 2}), ("attention_mma", {"HEAD_DIM": 128, "WEIGHT_TERMS": 2})]
 
 def register_library(name: str, sources: Sequence[str], flags: Sequence[str] = (), *, replace: bool = False) -> None:
     """Make a library of CUDA sources from outside the package known to :func:`load_library`, so that a

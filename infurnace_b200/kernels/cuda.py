@@ -562,10 +562,11 @@ class CudaKernels:
 
     # ------------------------------------------------------------------ attention
     def paged_attention(self, qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q, seq_lens, out,
-                        scale, window, max_q_len, max_seq_len, min_q_len=1, weight_terms=1):
+                        scale, window, max_q_len, max_seq_len, min_q_len=1, weight_terms=1, score_bound=None):
         """``weight_terms`` 2 (tensor-core route only): a softmax weight enters the weighted sum as two bfloat16 terms, its
-        rounding and what the rounding left out, so that 16 bits of the float32 weight count; the tcgen05 prompt kernel, which
-        has one term, is then not taken."""
+        rounding and what the rounding left out, so that 16 bits of the float32 weight count; the tcgen05 prompt kernel for
+        plain scores, which has one term, is then not taken.  ``score_bound``: what no scaled score exceeds in size, if the
+        caller knows it; up to ``TC_CAP_LIMIT`` prompts then run on the tcgen05 kernel for bounded scores."""
         _dense(qkv, "qkv"), _dense(kv_pages, "kv_pages", qkv.dtype), _dense(out, "out", qkv.dtype)
         _dense(cu_q, "cu_q", torch.int32), _dense(seq_lens, "seq_lens", torch.int32)
         if block_tables.dtype != torch.int32 or block_tables.stride(1) != 1:
@@ -582,7 +583,7 @@ class CudaKernels:
                 and num_heads % num_kv_heads == 0:
             return self._paged_attention_mma(qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q,
                                              seq_lens, out, scale, window, max_q_len, max_seq_len, n, r,
-                                             min_q_len=min_q_len, weight_terms=weight_terms)      # keys and values in one tensor
+                                             min_q_len=min_q_len, weight_terms=weight_terms, score_bound=score_bound)      # keys and values in one tensor
         self.launches += 1
         _check(self.core.ifb_paged_attention_simt(
             qkv.data_ptr(), _code(qkv), qkv.stride(0), kv_pages.data_ptr(), block_tables.data_ptr(),
@@ -606,7 +607,7 @@ class CudaKernels:
 
     def _attention_tc_fits(self, head_dim, value_head_dim, page_size, group, weight_terms, softcap, sink, one_tensor):
         """Whether prompts of these sizes run on the tcgen05 attention kernel: plain attention with heads of 128 in one tensor
-        and one-term weights, or capped scores over streams of any widths that its tiles hold."""
+        and one-term weights, or capped or bounded scores over streams of any widths that its tiles hold."""
         if not self.attention_tc or page_size not in (16, 32, 64):
             return False
         if softcap:
@@ -616,11 +617,12 @@ class CudaKernels:
                 and one_tensor.data_ptr() % 128 == 0)
 
     def _attention_tc_streams(self, qkv, num_heads, num_kv_heads, share, head_dim, value_head_dim, k, v, num_pages, block_tables, cu_q,
-                              seq_lens, out, scale, window, max_q_len, n, r, weight_terms, softcap, sink):
+                              seq_lens, out, scale, window, max_q_len, n, r, weight_terms, softcap, sink, kind):
+        """``kind``: 0 plain scores, 1 capped at ``softcap``, 2 no larger than ``softcap`` as they are."""
         self._err_armed = True
         self.launches += 1
         self.tc_attention_calls += 1
-        lib = self._attention_tc_library(head_dim, weight_terms, value_head_dim, bool(softcap))
+        lib = self._attention_tc_library(head_dim, weight_terms, value_head_dim, kind)
         _check(lib.ifb_attention_tc(
             qkv.data_ptr(), qkv.stride(0), k[0], k[1], v[0], v[1], num_pages, block_tables.data_ptr(), block_tables.stride(0),
             cu_q.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), self._dev_err.data_ptr(), n, r, num_heads, num_kv_heads, share,
@@ -636,7 +638,7 @@ class CudaKernels:
         if value_head_dim not in (None, head_dim):
             defines["VALUE_DIM"] = value_head_dim
         if softcap:
-            defines["SOFTCAP"] = 1
+            defines["SOFTCAP"] = int(softcap)           # 1: a cap, 2 (prompts on tcgen05 only): bounded scores
         return defines
 
     def attention_library(self, head_dim, weight_terms=1, value_head_dim=None, softcap=False):
@@ -672,14 +674,15 @@ class CudaKernels:
         return self._attn_scratch
 
     def _paged_attention_mma(self, qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q, seq_lens, out,
-                             scale, window, max_q_len, max_seq_len, n, r, num_splits=None, min_q_len=1, weight_terms=1):
+                             scale, window, max_q_len, max_seq_len, n, r, num_splits=None, min_q_len=1, weight_terms=1,
+                             score_bound=None):
         """Keys and values of one width in one tensor [pages, 2, kv_heads, page_size, head_dim]: two streams of a common stride."""
         esize, ps = kv_pages.element_size(), kv_pages.shape[3]
         k = (kv_pages.data_ptr(), kv_pages.stride(0), ps)
         v = (kv_pages.data_ptr() + esize * num_kv_heads * ps * head_dim, kv_pages.stride(0), ps)
         self._attention_mma_streams(qkv, num_heads, num_kv_heads, head_dim, head_dim, k, v, kv_pages.shape[0], block_tables, cu_q, seq_lens,
                                     out, scale, window, max_q_len, max_seq_len, n, r, num_splits, min_q_len, weight_terms,
-                                    one_tensor=kv_pages)
+                                    one_tensor=kv_pages, score_bound=score_bound)
 
     ATTENTION_GROUP = 16      # query heads that share a key/value head's rows in one CTA of the small-q kernel
 
@@ -690,7 +693,7 @@ class CudaKernels:
 
     def _attention_mma_streams(self, qkv, num_heads, num_kv_heads, head_dim, value_head_dim, k, v, num_pages, block_tables, cu_q,
                                seq_lens, out, scale, window, max_q_len, max_seq_len, n, r, num_splits=None, min_q_len=1,
-                               weight_terms=1, softcap=None, sink=None, one_tensor=None):
+                               weight_terms=1, softcap=None, sink=None, one_tensor=None, score_bound=None):
         """The tensor-core attention kernels over key and value streams ``k`` and ``v`` = (address, elements between pages, page
         size).  ``one_tensor``: the tensor that holds both, where there is one (what the tcgen05 kernel for plain attention takes)."""
         share = self.attention_share(num_heads // num_kv_heads)
@@ -711,9 +714,13 @@ class CudaKernels:
                 self._attn_counters = torch.zeros(max(r * num_kv_heads, 4096), dtype=torch.int32, device="cuda")
                 self.scratch_generation += 1
             counters = self._attn_counters
-        if not only_small and self._attention_tc_fits(head_dim, value_head_dim, page_size, group, weight_terms, softcap, sink, one_tensor):
+        if softcap or score_bound is None or not 0.0 < score_bound <= self.TC_CAP_LIMIT:
+            score_bound = None
+        if not only_small and self._attention_tc_fits(head_dim, value_head_dim, page_size, group, weight_terms, softcap or score_bound, sink,
+                                                      one_tensor):
             self._attention_tc_streams(qkv, num_heads, num_kv_heads, share, head_dim, value_head_dim, k, v, num_pages, block_tables, cu_q,
-                                       seq_lens, out, scale, window, max_q_len, n, r, weight_terms, softcap, sink)
+                                       seq_lens, out, scale, window, max_q_len, n, r, weight_terms, softcap or score_bound, sink,
+                                       kind=2 if score_bound else 1 if softcap else 0)
             if min_q_len * group > 16:
                 return                 # no request of this step is left for the small-q kernel
             only_small = True          # the tile kernel's requests are done; the small-q kernel takes the rest
@@ -1371,7 +1378,7 @@ class CudaKernels:
 
     def paged_attention_streams(self, q, num_heads, num_kv_heads, head_dim, value_head_dim, k_pages, v_pages, block_tables, cu_q,
                                 seq_lens, out, scale, window, out_table, out_interleaved, max_q_len=0, max_seq_len=0, min_q_len=1,
-                                softcap=None, sink=None, weight_terms=1, exact=True):
+                                softcap=None, sink=None, weight_terms=1, exact=True, score_bound=None):
         """Causal softmax attention of q [n, H d] over key and value page streams (csrc/attention_streams.cu), float32
         scores, weights and sums; each head's output is rotated back by the query token's angles of ``out_table``
         ([n, dv] (cos, sin) pairs; None: not).  ``softcap`` c: a scaled score s becomes c tanh(s / c).  ``sink`` z: exp(z) joins the
@@ -1379,7 +1386,7 @@ class CudaKernels:
 
         ``exact`` False: bfloat16 streams whose widths are multiples of 16 (at most 256), without ``out_table``, run the
         tensor-core kernels (csrc/attention_mma.cu): float32 scores, softmax and sums, a softmax weight entering the weighted
-        sum as ``weight_terms`` bfloat16 numbers."""
+        sum as ``weight_terms`` bfloat16 numbers; ``score_bound`` as :meth:`paged_attention`'s."""
         _dense(q, "q"), _dense(out, "out", q.dtype), _dense(cu_q, "cu_q", torch.int32), _dense(seq_lens, "seq_lens", torch.int32)
         if block_tables.dtype != torch.int32 or block_tables.stride(1) != 1:
             raise KernelError("paged_attention_streams: block_tables must be int32 with unit stride along pages")
@@ -1397,7 +1404,7 @@ class CudaKernels:
         if not exact and q.dtype == torch.bfloat16 and out_table is None and d % 16 == 0 and dv % 16 == 0 and d <= 256 and dv <= 256 \
                 and max_q_len and max_seq_len:
             return self._attention_mma_streams(q, H, G, d, dv, pk, pv, k_pages.shape[0], block_tables, cu_q, seq_lens, out, scale, window,
-                                               max_q_len, max_seq_len, n, r, None, min_q_len, weight_terms, softcap, sink)
+                                               max_q_len, max_seq_len, n, r, None, min_q_len, weight_terms, softcap, sink, score_bound=score_bound)
         self.launches += 1
         self.stream_attention_calls += 1
         _check(self._hyb_lib().ifb_paged_attention_streams(

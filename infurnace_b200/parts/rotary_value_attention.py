@@ -61,6 +61,8 @@ class RotaryValueAttention:
         self.extra = {key: value for key, value in (("softcap", spec.softcap), ("sink", spec.sink_score)) if value is not None}
         if spec.weight_terms != 1:
             self.extra["weight_terms"] = spec.weight_terms
+        if spec.unit_qk:                              # |q . k| is at most head_dim
+            self.extra["score_bound"] = abs(spec.scale) * spec.head_dim
 
     can_fold_output = True
 
@@ -156,7 +158,7 @@ class RotaryValueAttention:
             # the framework's tensor-core attention over the entry's one tensor of keys and values, then the turn back
             k.paged_attention(q, s.num_heads, s.num_kv_heads, s.head_dim, kv.pages, kv.block_tables, ctx.cu_q, ctx.seq_lens, attn,
                               s.scale, s.window or 0, ctx.max_q_len, ctx.max_seq_len, min_q_len=ctx.min_q_len,
-                              **({"weight_terms": s.weight_terms} if s.weight_terms != 1 else {}))
+                              **{key: self.extra[key] for key in ("weight_terms", "score_bound") if key in self.extra})
             if v_table is not None:
                 k.rotate_rows(attn, v_table, s.num_heads, s.value_head_dim, s.value_head_dim, bool(s.value_position.interleaved),
                               back=True)

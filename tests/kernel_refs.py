@@ -185,7 +185,7 @@ class ReferenceKernels:
 
     # ------------------------------------------------------------------ attention over pages
     def paged_attention(self, qkv, num_heads, num_kv_heads, head_dim, kv_pages, block_tables, cu_q,
-                        seq_lens, out, scale, window, max_q_len, max_seq_len, min_q_len=1, weight_terms=1):
+                        seq_lens, out, scale, window, max_q_len, max_seq_len, min_q_len=1, weight_terms=1, score_bound=None):
         """For request r the query tokens are rows cu_q[r] .. cu_q[r+1]-1 of qkv (their q
         heads are the first nq*d columns); the last of them stands at position
         seq_lens[r]-1.  A query at position p attends to the keys at positions
@@ -620,7 +620,7 @@ class ReferenceKernels:
 
     def paged_attention_streams(self, q, num_heads, num_kv_heads, head_dim, value_head_dim, k_pages, v_pages, block_tables, cu_q,
                                 seq_lens, out, scale, window, out_table, out_interleaved, max_q_len=0, max_seq_len=0, min_q_len=1,
-                                softcap=None, sink=None, weight_terms=1, exact=True):
+                                softcap=None, sink=None, weight_terms=1, exact=True, score_bound=None):
         """Causal softmax attention of q [n, H d] over the keys and values of the request's pages (streams
         [pages, G, page_size, width]); a scaled score s becomes softcap * tanh(s / softcap), exp(sink) joins the denominator;
         the output of every head is then rotated BACK by the angles of out_table (the

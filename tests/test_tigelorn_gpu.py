@@ -311,9 +311,13 @@ def test_a_far_key_and_the_windows_edges(K, dtype, d, dv, window, dist):
         cu, seq, _, _ = requests(lens_new, lens_old)
         want, got = torch.zeros(q.shape[0], H * dv, dtype=torch.float64), torch.zeros(q.shape[0], H * dv, device="cuda", dtype=dtype)
         REF.paged_attention_streams(q.double(), H, G, d, dv, pk.double(), pv.double(), bt, cu, seq, want, scale, window, None, False)
+        before = K.tc_attention_calls
         K.paged_attention_streams(*cuda(q), H, G, d, dv, *cuda(pk, pv, bt, cu, seq), got, scale, window, None, False,
-                                  max_q_len=max(lens_new), max_seq_len=max(total), min_q_len=min(lens_new), weight_terms=2, exact=False)
+                                  max_q_len=max(lens_new), max_seq_len=max(total), min_q_len=min(lens_new), weight_terms=2, exact=False,
+                                  score_bound=scale * d)
         close(got, want, (2e-5 if dtype == torch.float32 else 0.03) * max(1.0, float(want.abs().max())), f"window {window}, distance {dist}, {lens_new}")
+        if dtype == torch.bfloat16 and d % 16 == 0 and max(lens_new) > 1:
+            assert K.tc_attention_calls > before                                       # the tcgen05 kernel for bounded scores
         planted = pv[int(bt[0, pos // ps]), :, pos % ps].double().repeat_interleave(H // G, dim=0).reshape(-1)
         inside = window == 0 or dist < window
         if d >= 64:
@@ -365,15 +369,15 @@ def test_cutting_modes(models, name, mode, dtype):
 
 
 def test_the_fast_routes_ran(models):
-    """The wider model's bfloat16 steps take the tensor-core attention kernels and the chunked delta rule and scan; its layers
+    """The wider model's bfloat16 steps take the tensor-core attention kernels (bounded scores on tcgen05) and the chunked delta rule and scan; its layers
     would otherwise pass on the plain kernels alone."""
     d, cfg, w, reqs, ref = models["T3"]
     runner = _runner(d, "T3", "bfloat16", 640)
     k = runner.rt.kernels
-    before = (k.latent_mma_calls, k.delta_chunked_calls, k.linear_scan_blocked_calls, k.stream_attention_calls)
+    before = (k.latent_mma_calls, k.delta_chunked_calls, k.linear_scan_blocked_calls, k.stream_attention_calls, k.tc_attention_calls)
     tiny.run_inprocess(runner, tiny.schedule_whole({"a": reqs["r9"]}))
     assert k.latent_mma_calls > before[0] and k.delta_chunked_calls > before[1] and k.linear_scan_blocked_calls > before[2]
-    assert k.stream_attention_calls == before[3]
+    assert k.stream_attention_calls == before[3] and k.tc_attention_calls > before[4]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
