@@ -609,27 +609,30 @@ __device__ __forceinline__ void dr_copy16(float* dst, const float* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
 
-// Each of 8 neighbouring lanes holds 16 numbers; lane i is left with the sums over the lanes of numbers 2 i and 2 i + 1.
-__device__ __forceinline__ float2 dr_reduce16(float* x, int i) {
+// Each of LP neighbouring lanes holds 16 numbers; lane i is left with the sums over the lanes of numbers i TK .. i TK + TK - 1,
+// TK = 16 / LP, in x[0 .. TK - 1].
+template <int LP>
+__device__ __forceinline__ void dr_reduce16(float* x, int i) {
 #pragma unroll
-  for (int half = 8; half >= 2; half >>= 1) {
-    const bool up = i & (half >> 1);
+  for (int half = 8; half >= 16 / LP; half >>= 1) {
+    const int mask = half * LP / 16;
+    const bool up = i & mask;
 #pragma unroll
     for (int j = 0; j < half; ++j) {
       const float send = up ? x[j] : x[j + half], keep = up ? x[j + half] : x[j];
-      x[j] = keep + __shfl_xor_sync(0xffffffffu, send, half >> 1);
+      x[j] = keep + __shfl_xor_sync(0xffffffffu, send, mask);
     }
   }
-  return make_float2(x[0], x[1]);
 }
 
-// A block per (head, slab of 16 CPT columns) and request: thread (column, part), 8 parts of a column in neighbouring lanes,
-// part p with rows 32 b + 4 p + i, b = 0 .. DP / 32 - 1, i = 0 .. 3, of CPT columns 16 apart.
+// A block per (head, slab of columns) and request: thread (column, part), LP parts of a column in neighbouring lanes, part p
+// with rows b 4 LP + 4 p + i, b = 0 .. DP / (4 LP) - 1, i = 0 .. 3, of CPT columns.
 constexpr int DC_THREADS = 128;
-template <int DP, int CPT>
+template <int DP, int LP, int CPT>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_carry_kernel(DeltaRuleArgs a) {
-  constexpr int NB = DP / 32, NC = 16 * CPT;
+  constexpr int CB = DC_THREADS / LP, NC = CB * CPT;                  // columns side by side, columns of the block
+  constexpr int NB = DP / (4 * LP), TK = 16 / LP;
   constexpr int OPER = 3 * DR_C * DP + DR_C * DR_PP + DP;             // W, Q, K, P, decay: contiguous in the scratch
   constexpr int STAGE = OPER + DR_C * NC;
   extern __shared__ __align__(16) float sm[];
@@ -637,7 +640,7 @@ delta_carry_kernel(DeltaRuleArgs a) {
   ifb_pdl_trigger();
   const int r = blockIdx.y, h = blockIdx.x / a.slabs, c0 = (blockIdx.x % a.slabs) * NC;
   if (a.seq_lens[r] <= 0) return;
-  const int dim = a.dim, vdim = a.vdim, vp = dr_vp(vdim), tid = threadIdx.x, p = tid & 7, cl = tid >> 3;
+  const int dim = a.dim, vdim = a.vdim, vp = dr_vp(vdim), tid = threadIdx.x, p = tid % LP, cl = tid / LP;
   int first = 0;                                        // the request's first chunk among all
   for (int i = 0; i < r; ++i) first += a.seq_lens[i] > 0 ? (a.cu_q[i + 1] - a.cu_q[i] + DR_C - 1) / DR_C : 0;
   const int ta = a.cu_q[r], tb = a.cu_q[r + 1], n = (tb - ta + DR_C - 1) / DR_C;
@@ -649,10 +652,10 @@ delta_carry_kernel(DeltaRuleArgs a) {
   float S[CPT][NB * 4];
 #pragma unroll
   for (int x = 0; x < CPT; ++x) {
-    const int c = c0 + x * 16 + cl;
+    const int c = c0 + x * CB + cl;
 #pragma unroll
     for (int i = 0; i < NB * 4; ++i) {
-      const int row = (i >> 2) * 32 + p * 4 + (i & 3);
+      const int row = (i >> 2) * 4 * LP + p * 4 + (i & 3);
       S[x][i] = (c < vdim && row < dim) ? sp[(size_t)row * vdim + c] : 0.f;
     }
   }
@@ -670,6 +673,32 @@ delta_carry_kernel(DeltaRuleArgs a) {
       if (t < tb && c < vdim) a.raw[((size_t)t * a.heads + h) * vdim + c] = o[i];
     }
   };
+  // acc[x][t] = this part's share of sum_rows M[t][row] S[x][row]; eight tokens' chains side by side
+  auto times_state = [&](const float* M, float (&acc)[CPT][DR_C]) {
+#pragma unroll
+    for (int x = 0; x < CPT; ++x)
+#pragma unroll
+      for (int t = 0; t < DR_C; ++t) acc[x][t] = 0.f;
+#pragma unroll
+    for (int b = 0; b < NB; ++b)
+#pragma unroll
+      for (int tg = 0; tg < DR_C; tg += 8) {
+        float4 m[8];
+#pragma unroll
+        for (int t = 0; t < 8; ++t) m[t] = *reinterpret_cast<const float4*>(M + (tg + t) * DP + b * 4 * LP + p * 4);
+#pragma unroll
+        for (int x = 0; x < CPT; ++x) {
+#pragma unroll
+          for (int t = 0; t < 8; ++t) acc[x][tg + t] = fmaf(m[t].x, S[x][4 * b], acc[x][tg + t]);
+#pragma unroll
+          for (int t = 0; t < 8; ++t) acc[x][tg + t] = fmaf(m[t].y, S[x][4 * b + 1], acc[x][tg + t]);
+#pragma unroll
+          for (int t = 0; t < 8; ++t) acc[x][tg + t] = fmaf(m[t].z, S[x][4 * b + 2], acc[x][tg + t]);
+#pragma unroll
+          for (int t = 0; t < 8; ++t) acc[x][tg + t] = fmaf(m[t].w, S[x][4 * b + 3], acc[x][tg + t]);
+        }
+      }
+  };
   ask(0);
   for (int j = 0; j < n; ++j) {
     asm volatile("cp.async.wait_group 0;\n" ::);
@@ -678,96 +707,66 @@ delta_carry_kernel(DeltaRuleArgs a) {
     if (j > 0) give(j - 1);
     const float* s = sm + (j & 1) * STAGE;
     const float *Ws = s, *Qs = Ws + DR_C * DP, *Ks = Qs + DR_C * DP, *Ps = Ks + DR_C * DP, *Gs = Ps + DR_C * DR_PP, *Us = Gs + DP;
-    {
-      float w[CPT][DR_C];
+    float acc[CPT][DR_C];
+    times_state(Ws, acc);
 #pragma unroll
-      for (int t = 0; t < DR_C; ++t) {
+    for (int x = 0; x < CPT; ++x) {
+      dr_reduce16<LP>(acc[x], p);
 #pragma unroll
-        for (int x = 0; x < CPT; ++x) w[x][t] = 0.f;
-#pragma unroll
-        for (int b = 0; b < NB; ++b) {
-          const float4 wv = *reinterpret_cast<const float4*>(Ws + t * DP + b * 32 + p * 4);
-#pragma unroll
-          for (int x = 0; x < CPT; ++x)
-            w[x][t] = fmaf(wv.w, S[x][4 * b + 3], fmaf(wv.z, S[x][4 * b + 2], fmaf(wv.y, S[x][4 * b + 1], fmaf(wv.x, S[x][4 * b], w[x][t]))));
-        }
-      }
-#pragma unroll
-      for (int x = 0; x < CPT; ++x) {
-        const float2 ws = dr_reduce16(w[x], p);
-        const int col = x * 16 + cl;
-        *reinterpret_cast<float2*>(us + col * (DR_C + 4) + 2 * p) =
-            make_float2(Us[2 * p * NC + col] - ws.x, Us[(2 * p + 1) * NC + col] - ws.y);
-      }
+      for (int m = 0; m < TK; ++m)
+        us[(x * CB + cl) * (DR_C + 4) + TK * p + m] = Us[(TK * p + m) * NC + x * CB + cl] - acc[x][m];
     }
-    __syncwarp();                                       // the 8 lanes of a column are in one warp
-    float y[CPT][2];                                    // outputs of tokens 2 p and 2 p + 1: what the state before the chunk gives
-    {
-      float o[CPT][DR_C];
+    __syncwarp();                                       // the lanes of a column are in one warp
+    times_state(Qs, acc);                               // what the state before the chunk gives to the outputs
 #pragma unroll
-      for (int t = 0; t < DR_C; ++t) {
-#pragma unroll
-        for (int x = 0; x < CPT; ++x) o[x][t] = 0.f;
-#pragma unroll
-        for (int b = 0; b < NB; ++b) {
-          const float4 qv = *reinterpret_cast<const float4*>(Qs + t * DP + b * 32 + p * 4);
-#pragma unroll
-          for (int x = 0; x < CPT; ++x)
-            o[x][t] = fmaf(qv.w, S[x][4 * b + 3], fmaf(qv.z, S[x][4 * b + 2], fmaf(qv.y, S[x][4 * b + 1], fmaf(qv.x, S[x][4 * b], o[x][t]))));
-        }
-      }
-#pragma unroll
-      for (int x = 0; x < CPT; ++x) {
-        const float2 v = dr_reduce16(o[x], p);
-        y[x][0] = v.x; y[x][1] = v.y;
-      }
-    }
+    for (int x = 0; x < CPT; ++x) dr_reduce16<LP>(acc[x], p);
     float u[CPT][DR_C];
 #pragma unroll
     for (int x = 0; x < CPT; ++x)
 #pragma unroll
       for (int t = 0; t < DR_C; t += 4)
-        *reinterpret_cast<float4*>(&u[x][t]) = *reinterpret_cast<const float4*>(us + (x * 16 + cl) * (DR_C + 4) + t);
-#pragma unroll
-    for (int m = 0; m < 2; ++m)
-#pragma unroll
-      for (int t = 0; t < DR_C; t += 4) {
-        const float4 pv = *reinterpret_cast<const float4*>(Ps + (2 * p + m) * DR_PP + t);
-#pragma unroll
-        for (int x = 0; x < CPT; ++x)
-          y[x][m] = fmaf(pv.w, u[x][t + 3], fmaf(pv.z, u[x][t + 2], fmaf(pv.y, u[x][t + 1], fmaf(pv.x, u[x][t], y[x][m]))));
-      }
-#pragma unroll
-    for (int x = 0; x < CPT; ++x) {
-      float* o = os + (j & 1) * DR_C * NC + x * 16 + cl;
-      o[2 * p * NC] = y[x][0];
-      o[(2 * p + 1) * NC] = y[x][1];
-    }
-    __syncwarp();                                       // u was read by all its lanes before the next chunk writes it
+        *reinterpret_cast<float4*>(&u[x][t]) = *reinterpret_cast<const float4*>(us + (x * CB + cl) * (DR_C + 4) + t);
 #pragma unroll
     for (int b = 0; b < NB; ++b) {
-      const float4 gv = *reinterpret_cast<const float4*>(Gs + b * 32 + p * 4);
+      const float4 gv = *reinterpret_cast<const float4*>(Gs + b * 4 * LP + p * 4);
 #pragma unroll
       for (int x = 0; x < CPT; ++x) { S[x][4 * b] *= gv.x; S[x][4 * b + 1] *= gv.y; S[x][4 * b + 2] *= gv.z; S[x][4 * b + 3] *= gv.w; }
+    }
 #pragma unroll
-      for (int t = 0; t < DR_C; ++t) {
-        const float4 kv = *reinterpret_cast<const float4*>(Ks + t * DP + b * 32 + p * 4);
+    for (int t = 0; t < DR_C; ++t)
+#pragma unroll
+      for (int b = 0; b < NB; ++b) {
+        const float4 kv = *reinterpret_cast<const float4*>(Ks + t * DP + b * 4 * LP + p * 4);
 #pragma unroll
         for (int x = 0; x < CPT; ++x) {
           S[x][4 * b] = fmaf(kv.x, u[x][t], S[x][4 * b]); S[x][4 * b + 1] = fmaf(kv.y, u[x][t], S[x][4 * b + 1]);
           S[x][4 * b + 2] = fmaf(kv.z, u[x][t], S[x][4 * b + 2]); S[x][4 * b + 3] = fmaf(kv.w, u[x][t], S[x][4 * b + 3]);
         }
       }
+#pragma unroll
+    for (int m = 0; m < TK; ++m) {
+      float4 pv[4];
+#pragma unroll
+      for (int t = 0; t < 4; ++t) pv[t] = *reinterpret_cast<const float4*>(Ps + (TK * p + m) * DR_PP + 4 * t);
+#pragma unroll
+      for (int x = 0; x < CPT; ++x) {
+        float y[4];
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+          y[t] = fmaf(pv[t].w, u[x][4 * t + 3], fmaf(pv[t].z, u[x][4 * t + 2], fmaf(pv[t].y, u[x][4 * t + 1], pv[t].x * u[x][4 * t])));
+        os[(j & 1) * DR_C * NC + (TK * p + m) * NC + x * CB + cl] = acc[x][m] + ((y[0] + y[1]) + (y[2] + y[3]));
+      }
     }
+    __syncwarp();                                       // u was read by all its lanes before the next chunk writes it
   }
   __syncthreads();
   give(n - 1);
 #pragma unroll
   for (int x = 0; x < CPT; ++x) {
-    const int c = c0 + x * 16 + cl;
+    const int c = c0 + x * CB + cl;
 #pragma unroll
     for (int i = 0; i < NB * 4; ++i) {
-      const int row = (i >> 2) * 32 + p * 4 + (i & 3);
+      const int row = (i >> 2) * 4 * LP + p * 4 + (i & 3);
       if (c < vdim && row < dim) sp[(size_t)row * vdim + c] = S[x][i];
     }
   }
@@ -787,25 +786,28 @@ static int dr_walk(DeltaRuleArgs a, cudaStream_t s) {
   return ifb_launch(delta_walk_kernel<T, RS, RPT>, dim3(a.heads * a.slabs, a.requests), dim3(cols * RS), smem, s, a);
 }
 
-template <int DP, int CPT>
+template <int DP, int LP, int CPT>
 static int dr_carry(DeltaRuleArgs a, cudaStream_t s) {
-  constexpr int NC = 16 * CPT, STAGE = 3 * DR_C * DP + DR_C * DR_PP + DP + DR_C * NC;
+  constexpr int NC = DC_THREADS / LP * CPT, STAGE = 3 * DR_C * DP + DR_C * DR_PP + DP + DR_C * NC;
   const size_t smem = (size_t)(2 * STAGE + NC * (DR_C + 4) + 2 * DR_C * NC) * sizeof(float);
   a.slabs = (a.vdim + NC - 1) / NC;
-  IFB_ALLOW_SMEM((delta_carry_kernel<DP, CPT>), smem);
+  IFB_ALLOW_SMEM((delta_carry_kernel<DP, LP, CPT>), smem);
   // not early: blocks placed while the chunks' launch still fills the device crowd on the SMs that are free first
-  return ifb_launch_opt(false, delta_carry_kernel<DP, CPT>, dim3(a.heads * a.slabs, a.requests), dim3(DC_THREADS), smem, s, a);
+  return ifb_launch_opt(false, delta_carry_kernel<DP, LP, CPT>, dim3(a.heads * a.slabs, a.requests), dim3(DC_THREADS), smem, s, a);
 }
 
 template <int DP>
-static int dr_chunked(DeltaRuleArgs a, int rows, bool two, cudaStream_t s) {
+static int dr_chunked(DeltaRuleArgs a, int rows, int columns, cudaStream_t s) {
   const size_t smem = (size_t)(3 * DR_C * (DP + 1) + 2 * DR_C * (DR_C + 1) + DR_C) * sizeof(float);
   IFB_ALLOW_SMEM(delta_chunk_kernel<DP>, smem);
   const int st = ifb_launch(delta_chunk_kernel<DP>, dim3(a.heads, rows), dim3(DA_THREADS), smem, s, a);
   if (st != IFB_OK) return st;
+  // columns per block: 8 (16 lanes a column), 16 (8 lanes), 32 (8 lanes, two columns each)
+  if constexpr (DP >= 64)
+    if (columns == 8) return dr_carry<DP, 16, 1>(a, s);
   if constexpr (DP <= 128)
-    if (two) return dr_carry<DP, 2>(a, s);
-  return dr_carry<DP, 1>(a, s);
+    if (columns == 32) return dr_carry<DP, 8, 2>(a, s);
+  return dr_carry<DP, 8, 1>(a, s);
 }
 
 template <typename T>
@@ -820,12 +822,11 @@ static int dr_run(DeltaRuleArgs a, int tokens, int columns, cudaStream_t s) {
   if (a.chunks) {
     const long long rows = (tokens + DR_C - 1) / DR_C + a.requests;
     if (rows > 65535 || !a.raw) return IFB_ERR_SIZE;
-    const bool two = columns == 2;
     switch (dr_dp(a.dim)) {
-      case 32: st = dr_chunked<32>(a, (int)rows, two, s); break;
-      case 64: st = dr_chunked<64>(a, (int)rows, two, s); break;
-      case 128: st = dr_chunked<128>(a, (int)rows, two, s); break;
-      default: st = dr_chunked<256>(a, (int)rows, two, s);
+      case 32: st = dr_chunked<32>(a, (int)rows, columns, s); break;
+      case 64: st = dr_chunked<64>(a, (int)rows, columns, s); break;
+      case 128: st = dr_chunked<128>(a, (int)rows, columns, s); break;
+      default: st = dr_chunked<256>(a, (int)rows, columns, s);
     }
   } else {
     const int cols = dr_walk_cols(a.dim, a.vdim);
@@ -854,14 +855,15 @@ IFB_EXPORT long long ifb_delta_rule_scratch_floats(int tokens, int requests, int
 }
 
 // chunks: null for the token walk, else ifb_delta_rule_scratch_floats(...) floats, 16-byte aligned, for the chunked form (heads of
-// up to 256 rows), which needs `raw` too.  columns: 1 or 2, the columns of a thread of the chunked form.
+// up to 256 rows), which needs `raw` too.  columns: 8, 16 or 32, the columns of a block of the chunked form: few for a
+// small grid, many where the blocks cover the device anyway (fewer reads of shared memory per product).
 IFB_EXPORT int ifb_delta_rule(const float* qkv, int ldc, const float* up, int ldu, const float* beta, const float* rate,
                               const float* bias, const float* norm_w, float eps, float* state, const int* state_slots,
                               const int* cu_q, const int* seq_lens, void* out, int out_dtype, float* raw, float* chunks, int columns,
                               int requests, int tokens, int kv_heads, int heads, int dim, int vdim, cudaStream_t stream) {
   if (requests <= 0 || tokens <= 0) return IFB_OK;
   if (kv_heads < 1 || heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || requests > 65535) return IFB_ERR_SIZE;
-  if (chunks && (((uintptr_t)chunks & 15) || columns < 1 || columns > 2)) return IFB_ERR_ARG;
+  if (chunks && (((uintptr_t)chunks & 15) || (columns != 8 && columns != 16 && columns != 32))) return IFB_ERR_ARG;
   DeltaRuleArgs a{qkv, ldc, up, ldu, beta, rate, bias, norm_w, eps, state, state_slots, cu_q, seq_lens, out, raw, chunks, kv_heads, heads,
                   dim, vdim, 1, requests};
   if (out_dtype == IFB_F32) return dr_run<float>(a, tokens, columns, stream);

@@ -121,6 +121,7 @@ class CudaKernels:
         self.rglru_chunked_calls = 0
         self._dr_scratch = None
         self.delta_chunked_calls = 0
+        self.delta_columns = int(os.environ.get("INFURNACE_DELTA_COLUMNS", "0"))      # of a block of the chunked form; 0: by the grid
         self.delta_chunk_min = int(os.environ.get("INFURNACE_DELTA_CHUNK_MIN", "33"))      # tokens of the longest request from
         self.moe_tensor_cores = os.environ.get("INFURNACE_MOE_MMA", "1") != "0"
         self.moe_tcgen05 = os.environ.get("INFURNACE_MOE_TCGEN05", "1") != "0"     # prompts' expert products on tcgen05
@@ -1230,8 +1231,8 @@ class CudaKernels:
                 self._dr_scratch = torch.empty(need + scratch, dtype=torch.float32, device="cuda")
                 self.scratch_generation += 1
         raw = self._dr_scratch[scratch:].data_ptr() if need else 0
-        # two columns per thread halve the reads of shared memory per product, where the blocks still cover the device
-        columns = 2 if r * heads * (-(-vdim // 32)) >= self.sm_count else 1
+        # the more columns a block has, the fewer reads of shared memory per product; the fewer, the more blocks
+        columns = self.delta_columns or next((c for c in (32, 16) if 5 * r * heads * -(-vdim // c) >= 4 * self.sm_count), 8)
         self.delta_chunked_calls += chunked
         self.launches += 3 if chunked else 2 if need else 1
         _check(lib.ifb_delta_rule(
