@@ -754,6 +754,9 @@ def attention_shape(conf):
         for layer in conf["layers"]:
             if layer["type"] == "attention":
                 return layer["mixer"]["kv_heads"], layer["mixer"]["dim"], None
+    if conf.get("architecture") == "Tigelorn":            # likewise; its latent layers are counted by their own rule
+        left = next(layer["mixer"]["left"] for layer in conf["layers"] if layer["type"] == "parallel")
+        return left["kv_heads"], left["dim"], None
     for layer in conf["layers"]:
         m = layer["mixer"]
         if layer["type"] == "attention":
